@@ -18,6 +18,7 @@ LIB_PATH = os.path.join(HERE, "libemelb.so")
 
 # dtype codes (src/emel/kernel/events.hpp:78-123)
 F32, F16, Q4_0, Q8_0, Q4_K, Q6_K, Q8_K, I32 = 0, 1, 2, 8, 12, 14, 15, 26
+BF16 = 30   # weights of layered decoder sessions
 BLOCK_ELEMS = {Q4_0: 32, Q8_0: 32, Q4_K: 256, Q6_K: 256, Q8_K: 256}
 BLOCK_BYTES = {Q4_0: 18, Q8_0: 34, Q4_K: 144, Q6_K: 210, Q8_K: 292}
 # error bitmask (src/emel/kernel/errors.hpp:7-13)

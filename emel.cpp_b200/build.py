@@ -6,6 +6,7 @@ from __future__ import annotations
 import os
 import subprocess
 import sys
+from concurrent.futures import ThreadPoolExecutor
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
@@ -29,6 +30,12 @@ SOURCES = {
     "gemm_q8_mma.cu": [],
     "gemm_q4k_mma.cu": [],
     "gemm_q6k_mma.cu": [],
+    "linear.cu": [],
+    "gemm_bf16.cu": [],
+    "mixer_ops.cu": [],
+    "mixed_attention.cu": [],
+    "lightning.cu": [],
+    "layered.cu": [],
     "llama.cu": [],
     "comm.cu": [],
     "noalloc.cu": [],
@@ -68,6 +75,22 @@ def build(verbose: bool = False, force: bool = False) -> str:
     headers = [h for h in headers if os.path.exists(h)]
     nccl_inc, nccl_lib = _nccl_paths()
     objs = []
+
+    def compile_one(name, extra):
+        # written beside the object and moved into place, so that an interrupted build leaves none that looks finished
+        src, obj = os.path.join(CSRC, name), os.path.join(CSRC, name.replace(".cu", ".o"))
+        cmd = [nvcc] + ARCH + COMMON + extra + (["-Xptxas", "-v"] if verbose else [])
+        if nccl_inc:
+            cmd += ["-I", nccl_inc, "-DEMELB_HAVE_NCCL=1"]
+        tmp = f"{obj}.{os.getpid()}.tmp"
+        r = subprocess.run(cmd + ["-c", src, "-o", tmp], capture_output=True, text=True)
+        if verbose or r.returncode != 0:
+            sys.stderr.write(r.stdout + r.stderr)
+        if r.returncode != 0:
+            raise RuntimeError(f"nvcc failed for {name}")
+        os.replace(tmp, obj)
+
+    stale = []
     for name, extra in SOURCES.items():
         src = os.path.join(CSRC, name)
         if not os.path.exists(src):
@@ -75,17 +98,13 @@ def build(verbose: bool = False, force: bool = False) -> str:
         obj = os.path.join(CSRC, name.replace(".cu", ".o"))
         objs.append(obj)
         if force or _newer([src] + headers, obj):
-            cmd = [nvcc] + ARCH + COMMON + extra + (["-Xptxas", "-v"] if verbose else [])
-            if nccl_inc:
-                cmd += ["-I", nccl_inc, "-DEMELB_HAVE_NCCL=1"]
-            cmd += ["-c", src, "-o", obj]
-            r = subprocess.run(cmd, capture_output=True, text=True)
-            if verbose or r.returncode != 0:
-                sys.stderr.write(r.stdout + r.stderr)
-            if r.returncode != 0:
-                raise RuntimeError(f"nvcc failed for {name}")
+            stale.append((name, extra))
+    with ThreadPoolExecutor(max_workers=max(1, min(os.cpu_count() or 1, 16))) as pool:
+        for f in [pool.submit(compile_one, *job) for job in stale]:
+            f.result()
     if force or _newer(objs, OUT):
-        cmd = [nvcc] + ARCH + ["-shared", "-o", OUT] + objs
+        tmp = f"{OUT}.{os.getpid()}.tmp"
+        cmd = [nvcc] + ARCH + ["-shared", "-o", tmp] + objs
         if nccl_lib:
             # linked by soname; resolved at run time from the same wheel
             cmd += ["-L", nccl_lib, "-l:libnccl.so.2", "-Xlinker", f"-rpath={nccl_lib}"]
@@ -93,6 +112,7 @@ def build(verbose: bool = False, force: bool = False) -> str:
         if r.returncode != 0:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
+        os.replace(tmp, OUT)
     return OUT
 
 

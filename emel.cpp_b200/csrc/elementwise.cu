@@ -748,6 +748,34 @@ cudaError_t launch_argmax_columns(const float* x, int rows, int B, float* part_v
   return cudaGetLastError();
 }
 
+namespace {
+__global__ void gather_columns_kernel(const float* __restrict__ x, int B, const int* __restrict__ index, int n, float* __restrict__ out, int64_t total) {
+  const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (i < total) out[i] = x[i / n * B + index[i % n]];
+}
+__global__ void transpose_kernel(const float* __restrict__ x, int rows, int cols, float* __restrict__ out) {
+  __shared__ float tile[32][33];
+  const int c = blockIdx.x * 32 + threadIdx.x, r0 = blockIdx.y * 32;
+  for (int i = threadIdx.y; i < 32; i += 8)
+    if (r0 + i < rows && c < cols) tile[i][threadIdx.x] = x[(int64_t)(r0 + i) * cols + c];
+  __syncthreads();
+  const int r = r0 + threadIdx.x, c0 = blockIdx.x * 32;
+  for (int i = threadIdx.y; i < 32; i += 8)
+    if (r < rows && c0 + i < cols) out[(int64_t)(c0 + i) * rows + r] = tile[threadIdx.x][i];
+}
+}  // namespace
+
+cudaError_t launch_gather_columns(const float* x, int K, int B, const int* index, int n, float* out, cudaStream_t st) {
+  const int64_t total = (int64_t)K * n;
+  gather_columns_kernel<<<(unsigned)((total + 255) / 256), 256, 0, st>>>(x, B, index, n, out, total);
+  return cudaGetLastError();
+}
+
+cudaError_t launch_transpose(const float* x, int rows, int cols, float* out, cudaStream_t st) {
+  transpose_kernel<<<dim3((cols + 31) / 32, (rows + 31) / 32), dim3(32, 8), 0, st>>>(x, rows, cols, out);
+  return cudaGetLastError();
+}
+
 cudaError_t launch_add_inplace(float* acc, const float* y, int64_t n, cudaStream_t st) {
   add_inplace_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(acc, y, n);
   return cudaGetLastError();

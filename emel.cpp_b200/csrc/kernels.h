@@ -177,6 +177,9 @@ int rms_norm_batch_partials(int B);
 cudaError_t launch_rope_store_batch(float* q, const float* k, const float* v, const float* cos_t, const float* sin_t, int pos0,
                                     int B, int n_head, int n_head_kv, int head_dim, int rot_dim, int neox, __half* kcache,
                                     __half* vcache, int64_t cache_head_stride, cudaStream_t st);
+// columns index[0..n) of x {K, B} -> out {K, n};  x {rows, cols} -> out {cols, rows}
+cudaError_t launch_gather_columns(const float* x, int K, int B, const int* index, int n, float* out, cudaStream_t st);
+cudaError_t launch_transpose(const float* x, int rows, int cols, float* out, cudaStream_t st);
 cudaError_t launch_add_inplace(float* acc, const float* y, int64_t n, cudaStream_t st);
 // ---- one decode step of B sequences together (activations {features, B}, sequence index fastest)
 // state: three rows of `stride` ints {token, position, kv token count} per sequence, then {step}

@@ -1,0 +1,254 @@
+// Products with bf16 weights on the CUDA cores: the one-row kernel of the decode step (streams the weights once, with
+// the step before it fused into its input and the activation into its output) and a plain f32 tile kernel for many
+// rows in full f32.  f32 activations and accumulation in both.
+#include <cstdlib>
+
+#include "common.cuh"
+#include "layered.h"
+
+namespace emelb {
+namespace {
+
+constexpr int kVecThreads = 256;
+constexpr int kVecWarps = kVecThreads / 32;
+
+__device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float siluf_(float z) { return z / (1.0f + expf(-z)); }
+
+__device__ __forceinline__ float block_sum(float v, float* scratch) {
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.0f;
+#pragma unroll
+  for (int w = 0; w < kVecWarps; ++w) t += scratch[w];
+  return t;
+}
+
+__device__ __forceinline__ uint4 load_stream(const uint4* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+
+// Input vector in shared memory, split so that a warp's reads of one half chunk are contiguous: elements 8c..8c+3 at
+// lo[c], 8c+4..8c+7 at hi[c].
+struct SplitVec {
+  float* lo;
+  float* hi;
+  __device__ __forceinline__ float& at(int i) const { return ((i & 4) ? hi : lo)[(i >> 3) * 4 + (i & 3)]; }
+};
+
+// A warp owns RW rows at a time (for ACT_GLU a gate row and its up row) and walks them in 16-byte chunks, U per lane
+// in flight; the first chunks are requested before the wait for the kernel in front.
+template <int RW, int U>
+__global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArgs a, const VecArgs v) {
+  extern __shared__ __align__(16) float xs_raw[];
+  __shared__ float scratch[kVecWarps];
+  pdl_trigger();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int K = a.w.K, chunks = (K + 7) / 8;
+  const SplitVec xs{xs_raw, xs_raw + 4 * chunks};
+  const bool glu = a.act == ACT_GLU;
+  const int outs = glu ? a.w.M / 2 : a.w.M;
+  const int per_task = glu ? 1 : RW;
+  const int tasks = (outs + per_task - 1) / per_task;
+  const int stride = gridDim.x * kVecWarps;
+  int task = blockIdx.x * kVecWarps + warp;
+
+  auto row_of = [&](int t, int r) { return glu ? t + r * outs : min(t * RW + r, outs - 1); };
+  uint4 w[RW][U];
+  auto load = [&](int t, int c0) {
+#pragma unroll
+    for (int r = 0; r < RW; ++r) {
+      const uint4* p = reinterpret_cast<const uint4*>(a.w.w + (int64_t)row_of(t, r) * a.w.ld);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int c = c0 + lane + 32 * u;
+        w[r][u] = c < chunks ? load_stream(p + c) : make_uint4(0, 0, 0, 0);
+      }
+    }
+  };
+  if (task < tasks) load(task, 0);
+  pdl_wait();
+
+  // ---- the input vector
+  for (int i = K + tid; i < 8 * chunks; i += kVecThreads) xs.at(i) = 0.0f;
+  if (v.pro == PRO_PLAIN) {
+    for (int i = tid; i < K; i += kVecThreads) xs.at(i) = v.x[i];
+  } else if (v.pro == PRO_EMBED) {
+    const __nv_bfloat16* row = v.table + (int64_t)*v.token * v.table_ld;
+    for (int i = tid; i < K; i += kVecThreads) {
+      const float x = __bfloat162float(row[i]);
+      xs.at(i) = x;
+      if (blockIdx.x == 0) v.x_out[i] = x;
+    }
+  } else if (v.pro == PRO_RMS_GATE) {
+    float ss = 0.0f;
+    for (int i = tid; i < K; i += kVecThreads) {
+      const float x = v.x[i];
+      xs.at(i) = x;
+      ss = fmaf(x, x, ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / K + v.eps);
+    for (int i = tid; i < K; i += kVecThreads) xs.at(i) = xs.at(i) * inv * v.norm_w[i] * v.gate[i];
+  } else {
+    float s = 0.0f;
+    for (int i = tid; i < K; i += kVecThreads) {
+      const float y = v.y[i];
+      xs.at(i) = y;
+      s += y;
+    }
+    const float mean = block_sum(s, scratch) / K;
+    float ss = 0.0f;
+    for (int i = tid; i < K; i += kVecThreads) {
+      const float d = xs.at(i) - mean;
+      ss = fmaf(d, d, ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / K + v.eps);
+    s = 0.0f;
+    for (int i = tid; i < K; i += kVecThreads) {
+      const float x = v.x[i] + (xs.at(i) - mean) * inv * v.norm_w[i];
+      xs.at(i) = x;
+      s += x;
+      if (v.x_out && blockIdx.x == 0) v.x_out[i] = x;
+    }
+    if (v.pro == PRO_RESIDUAL_NORM) {
+      const float mean2 = block_sum(s, scratch) / K;
+      ss = 0.0f;
+      for (int i = tid; i < K; i += kVecThreads) {
+        const float d = xs.at(i) - mean2;
+        ss = fmaf(d, d, ss);
+      }
+      const float inv2 = 1.0f / sqrtf(block_sum(ss, scratch) / K + v.eps);
+      for (int i = tid; i < K; i += kVecThreads) xs.at(i) = (xs.at(i) - mean2) * inv2 * v.norm2_w[i];
+    }
+  }
+  __syncthreads();
+
+  for (; task < tasks; task += stride) {
+    float acc[RW];
+#pragma unroll
+    for (int r = 0; r < RW; ++r) acc[r] = 0.0f;
+    for (int c0 = 0; c0 < chunks; c0 += 32 * U) {
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int c = c0 + lane + 32 * u;
+        if (c < chunks) {
+          const float4 xl = *reinterpret_cast<const float4*>(xs.lo + 4 * c), xh = *reinterpret_cast<const float4*>(xs.hi + 4 * c);
+          const float x[8] = {xl.x, xl.y, xl.z, xl.w, xh.x, xh.y, xh.z, xh.w};
+#pragma unroll
+          for (int r = 0; r < RW; ++r) {
+            const uint32_t q[4] = {w[r][u].x, w[r][u].y, w[r][u].z, w[r][u].w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              acc[r] = fmaf(__uint_as_float(q[i] << 16), x[2 * i], acc[r]);
+              acc[r] = fmaf(__uint_as_float(q[i] & 0xffff0000u), x[2 * i + 1], acc[r]);
+            }
+          }
+        }
+      }
+      // the next chunks of this task, or the first of the next one
+      if (c0 + 32 * U < chunks) load(task, c0 + 32 * U);
+      else if (task + stride < tasks) load(task + stride, 0);
+    }
+#pragma unroll
+    for (int r = 0; r < RW; ++r) acc[r] = warp_sum(acc[r]);
+    if (glu) {
+      if (lane == 0) {
+        float g = acc[0], u = acc[RW - 1];
+        if (a.bias) {
+          g += a.bias[task];
+          u += a.bias[task + outs];
+        }
+        v.out[task] = siluf_(g) * u;
+      }
+    } else {
+#pragma unroll
+      for (int r = 0; r < RW; ++r) {
+        const int row = task * RW + r;
+        if (lane == r && row < outs) {
+          float y = acc[r];
+          if (a.bias) y += a.bias[row];
+          if (a.act == ACT_SILU_SIGMOID) y = row < a.act_split ? siluf_(y) : sigmoidf_(y);
+          v.out[row] = y;
+        }
+      }
+    }
+  }
+}
+
+constexpr int kTile = 64, kTileK = 16;
+// 64 rows x 64 features per block of 256 threads, 4 x 4 outputs per thread
+__global__ void __launch_bounds__(256) linear_f32_kernel(const LinearArgs a, const float* __restrict__ x, int64_t ldx, float* __restrict__ y,
+                                                         int64_t ldy) {
+  __shared__ float xt[kTileK][kTile + 4], wt[kTileK][kTile + 4];
+  const int tid = threadIdx.x, r0 = blockIdx.y * kTile, f0 = blockIdx.x * kTile;
+  const int tr = (tid / 16) * 4, tf = (tid % 16) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < a.w.K; k0 += kTileK) {
+    for (int i = tid; i < kTile * kTileK; i += 256) {
+      const int row = i / kTileK, k = k0 + i % kTileK;
+      xt[i % kTileK][row] = r0 + row < a.rows && k < a.w.K ? x[(int64_t)(r0 + row) * ldx + k] : 0.0f;
+      wt[i % kTileK][row] = f0 + row < a.w.M && k < a.w.K ? __bfloat162float(a.w.w[(int64_t)(f0 + row) * a.w.ld + k]) : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kTileK; ++k) {
+      float xr[4], wr[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        xr[i] = xt[k][tr + i];
+        wr[i] = wt[k][tf + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xr[i], wr[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int row = r0 + tr + i, f = f0 + tf + j;
+      if (row >= a.rows || f >= a.w.M) continue;
+      float o = acc[i][j];
+      if (a.bias) o += a.bias[f];
+      if (a.act == ACT_SILU_SIGMOID) o = f < a.act_split ? siluf_(o) : sigmoidf_(o);
+      y[(int64_t)row * ldy + f] = o;
+    }
+}
+
+}  // namespace
+
+cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_count, bool pdl, cudaStream_t st) {
+  const int chunks = (a.w.K + 7) / 8, smem = 32 * chunks;
+  if (smem > 200 * 1024) return cudaErrorInvalidValue;
+  const bool glu = a.act == ACT_GLU;
+  const int outs = glu ? a.w.M / 2 : a.w.M;
+  // two rows per warp unless that leaves SMs without work
+  const bool pair = glu || outs >= sm_count * kVecWarps * 2;
+  auto kern = pair ? linear_vec_kernel<2, 4> : linear_vec_kernel<1, 8>;
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+  }
+  const int tasks = pair && !glu ? (outs + 1) / 2 : outs;
+  int per_sm = (200 * 1024) / (smem + 1024);
+  per_sm = per_sm > 4 ? 4 : per_sm;
+  int grid = (tasks + kVecWarps - 1) / kVecWarps;
+  if (grid > sm_count * per_sm) grid = sm_count * per_sm;
+  return launch_kernel(kern, dim3(grid), dim3(kVecThreads), (size_t)smem, st, pdl, a, v);
+}
+
+cudaError_t launch_linear_f32(const LinearArgs& a, const float* x, int64_t ldx, float* y, int64_t ldy, cudaStream_t st) {
+  if (a.act == ACT_GLU) return cudaErrorInvalidValue;
+  const dim3 grid((a.w.M + kTile - 1) / kTile, (a.rows + kTile - 1) / kTile);
+  linear_f32_kernel<<<grid, 256, 0, st>>>(a, x, ldx, y, ldy);
+  return cudaGetLastError();
+}
+
+}  // namespace emelb

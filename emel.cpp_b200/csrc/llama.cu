@@ -27,6 +27,7 @@
 #include "../../include/emelb_llama.h"
 #include "../../include/emelb_window.h"
 #include "ctx.h"
+#include "layered.h"
 #include "window.h"
 
 using namespace emelb;
@@ -125,12 +126,19 @@ struct emelb_llama {
   // from the slot the window hands out for the layer; steps then run as plain launches, not as replayed graphs
   emelb_window* window = nullptr;
   bool streamed = false;
+  // a session described layer by layer (emelb_llama_create_layers): its layers, caches and recurrent state.  The rest
+  // of the session -- token and position state, step graphs, sequences, sampling -- is the same for both kinds
+  Layered* layered = nullptr;
+  std::vector<int> seq_len;   // layered: tokens each sequence has taken (-1: unknown after a failed call)
+  int* want_idx = nullptr;    // rows whose logits a prompt call asks for, and their logits
+  float* want_logits = nullptr;
   std::vector<void*> owned;
 };
 
 namespace {
 
 constexpr int kMaxSeqs = 64;
+constexpr int kWantRows = 64;   // rows per output product of emelb_llama_prefill_logits
 
 // offset (halves) of sequence seq's planes of layer l inside the K or V cache
 int64_t cache_off(const emelb_llama* s, int l, int seq) {
@@ -157,6 +165,7 @@ int streamed_tensors(const emelb_llama* s) {
 }
 
 bool all_bound(const emelb_llama* s) {
+  if (s->layered) return layered_bound(s->layered);
   if (!bound(s->tok_embd) || !bound(s->out_norm) || !bound(s->output)) return false;
   for (const Layer& l : s->layers)
     if (!(bound(l.attn_norm) && bound(l.wq) && bound(l.wk) && bound(l.wv) && bound(l.wo) && bound(l.ffn_norm) &&
@@ -614,6 +623,15 @@ struct Enqueue {
   }
 
   void prefill_chunk(int B, int pos0) {
+    if (s->layered) {
+      // the position is read on the device; state holds it for the batch's first token
+      check(launch_step_begin(s->state, 0, pos0, st));
+      LayeredRun run{st};
+      layered_rows(s->layered, run, s->batch_tokens, Rows{B, true, s->cur_seq, s->state + 1}, pos0);
+      launches += run.launches + 1;
+      ok = ok && run.ok;
+      return;
+    }
     const emelb_llama_config& c = s->cfg;
     const int G = s->G, r = s->rank;
     const int heads_l = c.n_head / G, kv_l = c.n_head_kv / G;
@@ -658,12 +676,41 @@ struct Enqueue {
     }
   }
 
+  // logits of n batch rows (indices into the last prefill batch, in s->want_idx) -> s->want_logits {n, n_vocab}
+  void prefill_logits(int n, int B) {
+    const emelb_llama_config& c = s->cfg;
+    if (s->layered) {
+      LayeredRun run{st};
+      layered_rows_logits(s->layered, run, s->want_idx, n, s->want_logits);
+      launches += run.launches;
+      ok = ok && run.ok;
+      return;
+    }
+    // feature-major: gather the columns, norm, output product, and turn {n_vocab, n} into rows
+    check(launch_gather_columns(s->b_hidden, c.n_embd, B, s->want_idx, n, s->b_y, st));
+    check(launch_rms_norm_batch(s->b_y, reinterpret_cast<const float*>(s->out_norm.dev), c.rms_eps, c.n_embd, n, s->b_norm, s->b_partial, st));
+    float* cols = s->want_logits + (size_t)kWantRows * c.n_vocab;
+    batch_matmul(s->output, s->b_norm, cols, n);
+    check(launch_transpose(cols, c.n_vocab, n, s->want_logits, st));
+    launches += 4;
+  }
+
   // One decode step of sequences 0 .. B-1 together: column j of every activation tensor {features, B} is sequence
   // j's token (ids, positions and token counts in s->bstate).  Per column the arithmetic is token_step's: the
   // same products, the same rotation, the split-KV attention with the session's split count, so a sequence
   // decodes to the tokens it decodes to alone.  Ends with the per-column argmax (and the logits left in
   // s->b_logits, {n_vocab, B}).
   void batch_step(int B) {
+    if (s->layered) {
+      LayeredRun run{st};
+      layered_rows(s->layered, run, s->bstate, Rows{B, false, 0, s->bstate + kMaxSeqs}, 0);
+      layered_rows_logits(s->layered, run, nullptr, B, s->want_logits);
+      launches += run.launches + 3;
+      ok = ok && run.ok;
+      check(launch_transpose(s->want_logits, B, s->cfg.n_vocab, s->b_logits, st));
+      check(launch_argmax_columns(s->b_logits, s->cfg.n_vocab, B, s->b_amax_val, s->b_amax_idx, s->b_idx, st));
+      return;
+    }
     const emelb_llama_config& c = s->cfg;
     const int G = s->G, r = s->rank;
     const int heads_l = c.n_head / G, kv_l = c.n_head_kv / G;
@@ -777,7 +824,23 @@ struct Enqueue {
     launches += 2;
   }
 
+  // a layered session's step: the same modes, state words and follow-ups
+  void layered_token_step(Mode mode) {
+    LayeredRun run{st};
+    layered_step(s->layered, run, s->cur_seq, s->state, mode == MODE_PREFILL ? nullptr : s->logits);
+    launches += run.launches;
+    ok = ok && run.ok;
+    if (mode != MODE_ARGMAX || !ok) return;
+    check(launch_argmax_columns(s->logits, s->cfg.n_vocab, 1, s->c->part_val, s->c->part_idx, s->c->best_idx, st));
+    check(launch_step_advance(s->state, s->c->best_idx, s->tokens_dev, st));
+    launches += 3;
+  }
+
   void token_step(Mode mode) {
+    if (s->layered) {
+      layered_token_step(mode);
+      return;
+    }
     const emelb_llama_config& c = s->cfg;
     // which launches of the step carry the programmatic-serialization attribute (bit mask: 1 mat-vecs,
     // 2 RoPE/KV store, 4 attention, 8 SwiGLU, 16 the rest); the flag is read by EMELB_LAUNCH
@@ -895,12 +958,15 @@ cudaGraphExec_t step_graph(emelb_llama* s, Mode mode, int token, int position) {
     cudaGraphExecDestroy(s->graphs[mode]);
     s->graphs[mode] = nullptr;
   }
-  prepare_token_kernel(s);
-  // one eager pass first: sets per-kernel attributes outside the capture
-  if (!ctx_cuda_ok(s->c, launch_step_begin(s->state, token, position, s->c->stream))) return nullptr;
-  Enqueue warm{s, s->c->stream};
-  warm.token_step(mode);
-  if (!warm.ok || !ctx_cuda_ok(s->c, cudaStreamSynchronize(s->c->stream))) return nullptr;
+  if (!s->layered) {
+    prepare_token_kernel(s);
+    // one eager pass first: sets per-kernel attributes outside the capture.  (A layered session's step moves its
+    // recurrent state on, so there is none: its launches set attributes while they are captured, which is allowed)
+    if (!ctx_cuda_ok(s->c, launch_step_begin(s->state, token, position, s->c->stream))) return nullptr;
+    Enqueue warm{s, s->c->stream};
+    warm.token_step(mode);
+    if (!warm.ok || !ctx_cuda_ok(s->c, cudaStreamSynchronize(s->c->stream))) return nullptr;
+  }
   if (!ctx_cuda_ok(s->c, cudaStreamBeginCapture(s->c->stream, cudaStreamCaptureModeThreadLocal))) return nullptr;
   Enqueue e{s, s->c->stream};
   e.token_step(mode);
@@ -941,6 +1007,14 @@ bool step_launch(emelb_llama* s, Mode mode) {
   s->launches_mode[mode] = e.launches;
   if (mode == MODE_ARGMAX) s->launches_per_token = e.launches;
   return e.ok;
+}
+
+// a layered session's sequences continue where they ended, or start again
+bool continues(const emelb_llama* s, int seq, int position) {
+  return !s->layered || position == 0 || position == s->seq_len[(size_t)seq];
+}
+void set_length(emelb_llama* s, int seq, int length) {
+  if (s->layered) s->seq_len[(size_t)seq] = length;
 }
 
 bool valid_step(const emelb_llama* s, int token, int position) {
@@ -1079,6 +1153,36 @@ uint32_t emelb_llama_create(emelb_ctx* c, const emelb_llama_config* cfg, emelb_l
   return EMELB_OK;
 }
 
+uint32_t emelb_llama_check_layers(const emelb_llama_config* cfg, const emelb_layer_config* layers) {
+  return cfg ? layered_check(*cfg, layers) : EMELB_INVALID_REQUEST;
+}
+
+uint32_t emelb_llama_create_layers(emelb_ctx* c, const emelb_llama_config* cfg, const emelb_layer_config* layers, int32_t float32, emelb_llama** out) {
+  if (!c || !cfg || !out || (float32 != 0 && float32 != 1)) return EMELB_INVALID_REQUEST;
+  *out = nullptr;
+  if (layered_check(*cfg, layers) != EMELB_OK) return EMELB_INVALID_REQUEST;
+  cudaSetDevice(c->device);
+  emelb_llama* s = new (std::nothrow) emelb_llama();
+  if (!s) return EMELB_INTERNAL_ERROR;
+  s->c = c;
+  s->cfg = *cfg;
+  s->cfg.shard_count = 1;
+  s->seq_len.assign(1, 0);
+  s->layered = layered_create(c, s->cfg, layers, float32 == 1);
+  bool ok = s->layered != nullptr;
+  ok = ok && dev_alloc(s, (void**)&s->logits, 4 * (size_t)cfg->n_vocab) && dev_alloc(s, (void**)&s->state, 4 * sizeof(int));
+  ok = ok && dev_alloc(s, (void**)&s->tokens_dev, sizeof(int) * (size_t)(cfg->n_ctx + 8));
+  ok = ok && cudaMallocHost((void**)&s->host_pinned, sizeof(int) * (size_t)(cfg->n_ctx + 4 + 2 * kMaxSeqs)) == cudaSuccess;
+  ok = ok && cudaMemsetAsync(s->state, 0, 4 * sizeof(int), c->stream) == cudaSuccess && cudaStreamSynchronize(c->stream) == cudaSuccess;
+  if (!ok) {
+    cudaGetLastError();
+    emelb_llama_destroy(s);
+    return EMELB_INTERNAL_ERROR;
+  }
+  *out = s;
+  return EMELB_OK;
+}
+
 uint32_t emelb_llama_destroy(emelb_llama* s) {
   if (!s) return EMELB_INVALID_REQUEST;
   cudaSetDevice(s->c->device);
@@ -1088,6 +1192,7 @@ uint32_t emelb_llama_destroy(emelb_llama* s) {
   if (s->batch_graph) cudaGraphExecDestroy(s->batch_graph);
   for (int g = 0; g < kMaxPeers; ++g)
     if (s->peer_base[g] && g != s->rank) cudaIpcCloseMemHandle(s->peer_base[g]);
+  layered_destroy(s->layered);
   for (void* p : s->owned) cudaFree(p);
   if (s->host_pinned) cudaFreeHost(s->host_pinned);
   cudaGetLastError();
@@ -1097,6 +1202,13 @@ uint32_t emelb_llama_destroy(emelb_llama* s) {
 
 uint32_t emelb_llama_bind(emelb_llama* s, int32_t layer, int32_t role, const emelb_view* t) {
   if (!s || !t || !t->data) return EMELB_INVALID_REQUEST;
+  if (s->layered) {
+    cudaSetDevice(s->c->device);
+    const uint32_t err = layered_bind(s->layered, layer, role, t);
+    for (int m = 0; m < MODE_COUNT; ++m) s->graph_attention_mode[m] = -1;
+    s->batch_graph_mode = -1;
+    return err;
+  }
   const emelb_llama_config& c = s->cfg;
   const bool model_level = role <= EMELB_T_OUTPUT;
   if (role < 0 || role > EMELB_T_FFN_DOWN || (model_level ? layer != -1 : (layer < 0 || layer >= c.n_layer)))
@@ -1161,6 +1273,7 @@ uint32_t emelb_llama_bind(emelb_llama* s, int32_t layer, int32_t role, const eme
 
 uint32_t emelb_llama_set_window(emelb_llama* s, emelb_window* w) {
   if (!s) return EMELB_INVALID_REQUEST;
+  if (s->layered) return EMELB_UNSUPPORTED_OP;
   // tensors bound through the previous window keep offsets into its slots: they must be bound again first
   if (streamed_tensors(s) > 0) return EMELB_INVALID_REQUEST;
   if (w) {
@@ -1172,9 +1285,10 @@ uint32_t emelb_llama_set_window(emelb_llama* s, emelb_window* w) {
 }
 
 uint32_t emelb_llama_decode(emelb_llama* s, int32_t token, int32_t position, float* logits_out, int32_t* token_out) {
-  if (!s || !valid_step(s, token, position) || !all_bound(s)) return EMELB_INVALID_REQUEST;
+  if (!s || !valid_step(s, token, position) || !all_bound(s) || !continues(s, s->cur_seq, position)) return EMELB_INVALID_REQUEST;
   emelb_ctx* c = s->c;
   cudaSetDevice(c->device);
+  set_length(s, s->cur_seq, -1);
   const Mode mode = logits_out ? MODE_LOGITS : MODE_ARGMAX;
   if (!step_ready(s, mode, token, position)) return EMELB_INTERNAL_ERROR;
   bool ok = ctx_cuda_ok(c, launch_step_begin(s->state, token, position, c->stream));
@@ -1199,6 +1313,7 @@ uint32_t emelb_llama_decode(emelb_llama* s, int32_t token, int32_t position, flo
   }
   ok = ok && ctx_cuda_ok(c, cudaStreamSynchronize(c->stream));
   if (ok && token_out) *token_out = s->host_pinned[0];
+  if (ok) set_length(s, s->cur_seq, position + 1);
   return ok ? EMELB_OK : EMELB_INTERNAL_ERROR;
 }
 
@@ -1209,6 +1324,7 @@ namespace {
 // batch in the context's activation planes and, in a sharded session, the context's communicator for the joins.
 int prefill_batch_size(emelb_llama* s, int n) {
   const emelb_llama_config& c = s->cfg;
+  if (s->layered) return n < 2 || s->prefill_batch <= 0 ? 0 : s->prefill_batch;
   if (s->prefill_batch <= 0 || s->c->attention_mode != 0 || n < 2) return 0;
   if (s->G > 1 && (!s->c->comm || s->c->comm_world != s->G)) return 0;   // batch joins go through the communicator
   PrefillAttnArgs pa{nullptr, nullptr, s->kcache, s->vcache, s->capacity * c.head_dim, c.head_dim, c.n_head / s->G,
@@ -1229,6 +1345,11 @@ bool reserve_batch(emelb_llama* s, int B) {
   const emelb_llama_config& c = s->cfg;
   const size_t q_dim = (size_t)c.n_head * c.head_dim, kv_dim = (size_t)c.n_head_kv * c.head_dim, b = (size_t)B;
   bool ok = dev_alloc(s, (void**)&s->batch_tokens, sizeof(int) * b);
+  if (s->layered) {
+    ok = ok && layered_reserve_rows(s->layered, B);
+    s->batch_cap = ok ? B : -1;
+    return ok;
+  }
   ok = ok && dev_alloc(s, (void**)&s->b_hidden, 4 * b * c.n_embd) && dev_alloc(s, (void**)&s->b_norm, 4 * b * c.n_embd);
   ok = ok && dev_alloc(s, (void**)&s->b_y, 4 * b * c.n_embd);
   ok = ok && dev_alloc(s, (void**)&s->b_q, 4 * b * q_dim) && dev_alloc(s, (void**)&s->b_attn, 4 * b * q_dim);
@@ -1242,14 +1363,29 @@ bool reserve_batch(emelb_llama* s, int B) {
 
 }  // namespace
 
-uint32_t emelb_llama_prefill(emelb_llama* s, const int32_t* tokens, int32_t n, int32_t start_pos) {
-  if (!s || !tokens || n <= 0 || !all_bound(s) || start_pos < 0 || start_pos + n > s->cfg.n_ctx) return EMELB_INVALID_REQUEST;
+namespace {
+
+bool reserve_want(emelb_llama* s) {
+  if (s->want_idx) return true;
+  return dev_alloc(s, (void**)&s->want_logits, 2 * sizeof(float) * (size_t)kWantRows * s->cfg.n_vocab) &&
+         dev_alloc(s, (void**)&s->want_idx, sizeof(int) * kWantRows);
+}
+
+uint32_t run_prefill(emelb_llama* s, const int32_t* tokens, int32_t n, int32_t start_pos, const int32_t* want, int32_t n_want, float* logits_out) {
+  if (!s || !tokens || n <= 0 || !all_bound(s) || start_pos < 0 || start_pos + n > s->cfg.n_ctx || !continues(s, s->cur_seq, start_pos))
+    return EMELB_INVALID_REQUEST;
   for (int i = 0; i < n; ++i)
     if (!valid_step(s, tokens[i], start_pos + i)) return EMELB_INVALID_REQUEST;
+  if (n_want < 0 || (n_want > 0 && (!want || !logits_out || s->G > 1))) return EMELB_INVALID_REQUEST;
+  for (int i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= n || (i > 0 && want[i] <= want[i - 1])) return EMELB_INVALID_REQUEST;
   emelb_ctx* c = s->c;
   cudaSetDevice(c->device);
+  set_length(s, s->cur_seq, -1);
+  if (n_want > 0 && !reserve_want(s)) return EMELB_INTERNAL_ERROR;
+  const size_t row = sizeof(float) * (size_t)s->cfg.n_vocab;
   bool ok = true;
-  int done = 0;
+  int done = 0, given = 0;
   const int batch = prefill_batch_size(s, n);
   if (batch > 0 && reserve_batch(s, batch < s->cfg.n_ctx ? batch : s->cfg.n_ctx)) {
     // whole batches, then whatever is left as one shorter batch
@@ -1261,6 +1397,22 @@ uint32_t emelb_llama_prefill(emelb_llama* s, const int32_t* tokens, int32_t n, i
       c->diag.h2d_bytes += sizeof(int) * (uint64_t)B;
       Enqueue e{s, c->stream};
       e.prefill_chunk(B, start_pos + done);
+      while (ok && e.ok && given < n_want && want[given] < done + B) {
+        int k = 0;
+        const int room = kWantRows < s->batch_cap ? kWantRows : s->batch_cap;
+        int* idx = s->host_pinned + s->cfg.n_ctx;
+        while (k < room && given + k < n_want && want[given + k] < done + B) {
+          idx[k] = want[given + k] - done;
+          ++k;
+        }
+        ok = ctx_cuda_ok(c, cudaMemcpyAsync(s->want_idx, idx, sizeof(int) * (size_t)k, cudaMemcpyHostToDevice, c->stream));
+        e.prefill_logits(k, B);
+        ok = ok && e.ok && ctx_cuda_ok(c, cudaMemcpyAsync(logits_out + (size_t)given * s->cfg.n_vocab, s->want_logits, row * (size_t)k, cudaMemcpyDeviceToHost, c->stream));
+        ok = ok && ctx_cuda_ok(c, cudaStreamSynchronize(c->stream));
+        c->diag.h2d_bytes += sizeof(int) * (uint64_t)k;
+        c->diag.d2h_bytes += row * (uint64_t)k;
+        given += k;
+      }
       ok = ok && e.ok && ctx_cuda_ok(c, cudaStreamSynchronize(c->stream));  // host_pinned is reused by the next batch
       c->diag.kernel_launches += e.launches;
       done += B;
@@ -1268,15 +1420,41 @@ uint32_t emelb_llama_prefill(emelb_llama* s, const int32_t* tokens, int32_t n, i
     if (!ok) return EMELB_INTERNAL_ERROR;
   }
   if (done < n) {
-    if (!step_ready(s, MODE_PREFILL, tokens[done], start_pos + done)) return EMELB_INTERNAL_ERROR;
     for (int i = done; ok && i < n; ++i) {
-      ok = ctx_cuda_ok(c, launch_step_begin(s->state, tokens[i], start_pos + i, c->stream));
-      ok = ok && step_launch(s, MODE_PREFILL);
+      const bool wanted = given < n_want && want[given] == i;
+      const Mode mode = wanted ? MODE_LOGITS : MODE_PREFILL;
+      ok = step_ready(s, mode, tokens[i], start_pos + i);
+      ok = ok && ctx_cuda_ok(c, launch_step_begin(s->state, tokens[i], start_pos + i, c->stream));
+      ok = ok && step_launch(s, mode);
+      if (wanted) {
+        ok = ok && ctx_cuda_ok(c, cudaMemcpyAsync(logits_out + (size_t)given * s->cfg.n_vocab, s->logits, row, cudaMemcpyDeviceToHost, c->stream));
+        c->diag.d2h_bytes += row;
+        ++given;
+      }
     }
     c->diag.kernel_launches += (uint64_t)(n - done);
   }
   ok = ok && ctx_cuda_ok(c, cudaStreamSynchronize(c->stream));
+  if (ok) set_length(s, s->cur_seq, start_pos + n);
   return ok ? EMELB_OK : EMELB_INTERNAL_ERROR;
+}
+
+}  // namespace
+
+uint32_t emelb_llama_prefill(emelb_llama* s, const int32_t* tokens, int32_t n, int32_t start_pos) {
+  return run_prefill(s, tokens, n, start_pos, nullptr, 0, nullptr);
+}
+
+uint32_t emelb_llama_prefill_logits(emelb_llama* s, const int32_t* tokens, int32_t n, int32_t start_pos, const int32_t* want, int32_t n_want,
+                                    float* logits_out) {
+  return run_prefill(s, tokens, n, start_pos, want, n_want, logits_out);
+}
+
+uint32_t emelb_llama_trace_layers(emelb_llama* s, float* out, int32_t max_tokens) {
+  if (!s || !s->layered || max_tokens < 0) return EMELB_INVALID_REQUEST;
+  cudaSetDevice(s->c->device);
+  layered_set_trace(s->layered, out, max_tokens);
+  return EMELB_OK;
 }
 
 namespace {
@@ -1299,6 +1477,11 @@ bool reserve_sequences(emelb_llama* s) {
     ok = dev_alloc(s, (void**)&s->bstate, sizeof(int) * (3 * kMaxSeqs + 4)) && dev_alloc(s, (void**)&s->b_idx, sizeof(int) * kMaxSeqs);
     ok = ok && dev_alloc(s, (void**)&s->b_amax_val, 4 * (size_t)kArgmaxColumnParts * kMaxSeqs) &&
          dev_alloc(s, (void**)&s->b_amax_idx, 4 * (size_t)kArgmaxColumnParts * kMaxSeqs);
+  }
+  if (s->layered) {
+    ok = ok && reserve_want(s) && dev_alloc(s, (void**)&s->b_logits, 4 * b * c.n_vocab) && dev_alloc(s, (void**)&s->b_out, sizeof(int) * b * (size_t)(c.n_ctx + 8));
+    if (ok) s->seq_cap = s->n_seq;
+    return ok;
   }
   ok = ok && dev_alloc(s, (void**)&s->b_qs, 4 * b * q_dim) && dev_alloc(s, (void**)&s->b_logits, 4 * b * c.n_vocab);
   ok = ok && dev_alloc(s, (void**)&s->b_part_acc, 4 * b * (q_dim / s->G) * s->fa_splits) &&
@@ -1333,6 +1516,7 @@ bool free_owned(emelb_llama* s, void* p) {
 // widest activation in the context's planes, the communicator in a sharded session
 bool batch_step_ok(emelb_llama* s, int B) {
   const emelb_llama_config& c = s->cfg;
+  if (s->layered) return B >= 1 && B <= s->n_seq;
   if (s->c->attention_mode != 0 || B < 1 || B > s->n_seq) return false;
   if (s->G > 1 && (!s->c->comm || s->c->comm_world != s->G)) return false;
   int widest = c.n_ff > c.n_embd ? c.n_ff : c.n_embd;
@@ -1356,9 +1540,11 @@ cudaGraphExec_t batch_step_graph(emelb_llama* s, int B) {
   }
   // one eager pass first (sets per-kernel attributes outside the capture); it is a real step for the state the
   // caller has just written, so the KV rows it writes are the rows the replay writes again
-  Enqueue warm{s, c->stream};
-  warm.batch_step(B);
-  if (!warm.ok || !ctx_cuda_ok(c, cudaStreamSynchronize(c->stream))) return nullptr;
+  if (!s->layered) {
+    Enqueue warm{s, c->stream};
+    warm.batch_step(B);
+    if (!warm.ok || !ctx_cuda_ok(c, cudaStreamSynchronize(c->stream))) return nullptr;
+  }
   if (!ctx_cuda_ok(c, cudaStreamBeginCapture(c->stream, cudaStreamCaptureModeThreadLocal))) return nullptr;
   Enqueue e{s, c->stream};
   e.batch_step(B);
@@ -1393,12 +1579,22 @@ bool write_batch_state(emelb_llama* s, const int32_t* tokens, const int32_t* pos
 bool valid_batch(const emelb_llama* s, const int32_t* tokens, const int32_t* positions, int B, int steps) {
   if (!tokens || !positions || B < 1 || B > s->n_seq || B > kMaxSeqs) return false;
   for (int j = 0; j < B; ++j)
-    if (!valid_step(s, tokens[j], positions[j]) || positions[j] + steps > s->cfg.n_ctx) return false;
+    if (!valid_step(s, tokens[j], positions[j]) || positions[j] + steps > s->cfg.n_ctx || !continues(s, j, positions[j])) return false;
   return true;
 }
 
 // the token-batch buffers were sized by an earlier, smaller batch: release them so that reserve_batch sizes them again
 void release_small_batch(emelb_llama* s, int need) {
+  if (s->layered) {
+    // more rows than the model object holds: reserve_batch grows its buffers, and captured steps point into the old ones
+    if (s->batch_cap > 0 && s->batch_cap < need) {
+      free_owned(s, s->batch_tokens);
+      s->batch_tokens = nullptr;
+      s->batch_cap = 0;
+      s->batch_graph_mode = -1;
+    }
+    return;
+  }
   if (s->batch_cap <= 0 || s->batch_cap >= need) return;
   cudaStreamSynchronize(s->c->stream);
   for (void* p : {(void*)s->batch_tokens, (void*)s->b_hidden, (void*)s->b_norm, (void*)s->b_y, (void*)s->b_q, (void*)s->b_attn,
@@ -1422,6 +1618,14 @@ uint32_t emelb_llama_set_sequences(emelb_llama* s, int32_t n_seq) {
   cudaSetDevice(c->device);
   if (!ctx_cuda_ok(c, cudaStreamSynchronize(c->stream))) return EMELB_INTERNAL_ERROR;
   if (n_seq == s->n_seq) return EMELB_OK;
+  if (s->layered) {
+    s->cur_seq = 0;
+    drop_graphs(s);
+    s->seq_len.assign((size_t)n_seq, 0);
+    if (!layered_set_sequences(s->layered, n_seq)) return EMELB_INTERNAL_ERROR;
+    s->n_seq = n_seq;
+    return EMELB_OK;
+  }
   const emelb_llama_config& g = s->cfg;
   const size_t halves = (size_t)g.n_layer * (size_t)n_seq * (g.n_head_kv / s->G) * s->capacity * g.head_dim;
   __half *k = nullptr, *v = nullptr;
@@ -1460,6 +1664,7 @@ uint32_t emelb_llama_decode_batch(emelb_llama* s, const int32_t* tokens, const i
   if (!batch_step_ok(s, n_seq)) return EMELB_UNSUPPORTED_OP;
   release_small_batch(s, n_seq);
   if (!reserve_sequences(s) || !reserve_batch(s, batch_buffer_columns(s)) || s->batch_cap < n_seq) return EMELB_INTERNAL_ERROR;
+  for (int j = 0; j < n_seq; ++j) set_length(s, j, -1);
   bool ok = write_batch_state(s, tokens, positions, n_seq);
   Enqueue e{s, c->stream};
   if (ok) e.batch_step(n_seq);
@@ -1476,6 +1681,7 @@ uint32_t emelb_llama_decode_batch(emelb_llama* s, const int32_t* tokens, const i
   }
   ok = ok && ctx_cuda_ok(c, cudaStreamSynchronize(c->stream));
   if (ok && tokens_out) std::memcpy(tokens_out, s->host_pinned, sizeof(int) * (size_t)n_seq);
+  for (int j = 0; ok && j < n_seq; ++j) set_length(s, j, positions[j] + 1);
   return ok ? EMELB_OK : EMELB_INTERNAL_ERROR;
 }
 
@@ -1488,6 +1694,7 @@ uint32_t emelb_llama_generate_batch(emelb_llama* s, const int32_t* first_tokens,
   if (!batch_step_ok(s, n_seq)) return EMELB_UNSUPPORTED_OP;
   release_small_batch(s, n_seq);
   if (!reserve_sequences(s) || !reserve_batch(s, batch_buffer_columns(s)) || s->batch_cap < n_seq) return EMELB_INTERNAL_ERROR;
+  for (int j = 0; j < n_seq; ++j) set_length(s, j, -1);
   bool ok = write_batch_state(s, first_tokens, start_positions, n_seq);
   cudaGraphExec_t g = ok && !s->streamed ? batch_step_graph(s, n_seq) : nullptr;
   if (!g && !(ok && s->streamed)) return EMELB_INTERNAL_ERROR;
@@ -1508,6 +1715,7 @@ uint32_t emelb_llama_generate_batch(emelb_llama* s, const int32_t* first_tokens,
   ok = ok && ctx_cuda_ok(c, cudaMemcpyAsync(tokens_out, s->b_out, bytes, cudaMemcpyDeviceToHost, c->stream));
   ok = ok && ctx_cuda_ok(c, cudaStreamSynchronize(c->stream));
   c->diag.d2h_bytes += bytes;
+  for (int j = 0; ok && j < n_seq; ++j) set_length(s, j, start_positions[j] + n_steps);
   return ok ? EMELB_OK : EMELB_INTERNAL_ERROR;
 }
 
@@ -1518,10 +1726,12 @@ uint32_t emelb_llama_batch_launches_per_step(const emelb_llama* s, int32_t* out)
 }
 
 uint32_t emelb_llama_generate(emelb_llama* s, int32_t first_token, int32_t start_pos, int32_t n, int32_t* tokens_out) {
-  if (!s || !tokens_out || n <= 0 || !all_bound(s) || !valid_step(s, first_token, start_pos) || start_pos + n > s->cfg.n_ctx)
+  if (!s || !tokens_out || n <= 0 || !all_bound(s) || !valid_step(s, first_token, start_pos) || start_pos + n > s->cfg.n_ctx ||
+      !continues(s, s->cur_seq, start_pos))
     return EMELB_INVALID_REQUEST;
   emelb_ctx* c = s->c;
   cudaSetDevice(c->device);
+  set_length(s, s->cur_seq, -1);
   if (!step_ready(s, MODE_ARGMAX, first_token, start_pos)) return EMELB_INTERNAL_ERROR;
   bool ok = ctx_cuda_ok(c, launch_step_begin(s->state, first_token, start_pos, c->stream));
   for (int i = 0; ok && i < n; ++i) ok = step_launch(s, MODE_ARGMAX);
@@ -1531,6 +1741,7 @@ uint32_t emelb_llama_generate(emelb_llama* s, int32_t first_token, int32_t start
   if (!ok) return EMELB_INTERNAL_ERROR;
   c->diag.d2h_bytes += sizeof(int) * (uint64_t)n;
   std::memcpy(tokens_out, s->host_pinned, sizeof(int) * (size_t)n);
+  set_length(s, s->cur_seq, start_pos + n);
   return EMELB_OK;
 }
 
@@ -1616,6 +1827,7 @@ uint32_t emelb_llama_exchange_detach(emelb_llama* s) {
 
 uint32_t emelb_llama_decode_profile(emelb_llama* s, int32_t token, int32_t position, uint64_t* stamps_ns, uint64_t stamps_count) {
   if (!s || !stamps_ns || !valid_step(s, token, position) || !all_bound(s)) return EMELB_INVALID_REQUEST;
+  if (s->layered) return EMELB_UNSUPPORTED_OP;
   const uint64_t need = (uint64_t)s->cfg.n_layer * kTokenTracePoints;
   if (stamps_count < need) return EMELB_INVALID_REQUEST;
   emelb_ctx* c = s->c;

@@ -1,0 +1,304 @@
+// Softmax attention over a sliding window that keeps the sequence's first tokens, with the heads' weights mixed after
+// the softmax: weight_h <- sum_g talk[h][g] weight_g, head h then weighs its own key/value head's rows.
+//
+// A head's output needs every head's normalised weights, so scores and weighted sum are separate launches:
+//   scores   raw scaled scores of each (row, head) over the visible keys, and {max, sum of exponentials} per key range
+//   values   per key range and key/value head: all heads' weights from the scores, the mixed weights of that group's
+//            heads, and their partial sums over the value rows
+//   reduce   partial sums of the ranges added in order
+// Visible keys of position i, in order: the kept tokens below the window (0 .. kk-1), then the window (lo .. i).
+#include <math.h>
+
+#include "common.cuh"
+#include "layered.h"
+
+namespace emelb {
+namespace {
+
+constexpr int kThreads = 128;
+constexpr int kTileKeys = 64;
+constexpr int kMaxNRep = 8;
+
+struct Span {
+  int lo, kk, n;
+  __device__ __forceinline__ int key(int idx) const { return idx < kk ? idx : lo + idx - kk; }
+};
+__device__ __forceinline__ Span span_of(int pos, int window, int keep) {
+  Span s;
+  s.lo = window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
+  s.kk = keep < s.lo ? keep : s.lo;
+  s.n = s.kk + pos - s.lo + 1;
+  return s;
+}
+
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 v = *reinterpret_cast<const uint4*>(p);
+  const uint32_t q[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    f[2 * i] = __uint_as_float(q[i] << 16);
+    f[2 * i + 1] = __uint_as_float(q[i] & 0xffff0000u);
+  }
+}
+
+template <class T> __device__ __forceinline__ T to(float x);
+template <> __device__ __forceinline__ float to<float>(float x) { return x; }
+template <> __device__ __forceinline__ __nv_bfloat16 to<__nv_bfloat16>(float x) { return __float2bfloat16_rn(x); }
+
+__device__ __forceinline__ int row_pos(const Rows& r, int i) { return r.prompt ? r.pos[0] + i : r.pos[i]; }
+__device__ __forceinline__ int row_seq(const Rows& r, int i) { return r.prompt ? r.seq0 : r.seq0 + i; }
+
+// grid (ranges, kv heads, rows).  Eight lanes per key, KU keys per lane group at a time, NR query heads at a time.
+template <class T, int NR>
+__global__ void __launch_bounds__(kThreads) mix_scores_kernel(const MixAttnArgs a, const Rows rows, int row0, int splits, int stride) {
+  extern __shared__ __align__(16) float qs[];   // [n_rep][dim_pad]
+  __shared__ float red[2][kMaxNRep][4];
+  constexpr int KU = 4;
+  const int tid = threadIdx.x, l8 = tid & 7, slot = tid >> 3;
+  const int split = blockIdx.x, g = blockIdx.y, row = row0 + blockIdx.z;
+  const int n_rep = a.heads / a.kv_heads, D = a.dim_pad;
+  const Span sp = span_of(row_pos(rows, row), a.window, a.keep_first);
+  const int L = (sp.n + splits - 1) / splits, i0 = min(sp.n, split * L), i1 = min(sp.n, i0 + L);
+  const T* q = static_cast<const T*>(a.q) + ((int64_t)row * a.heads + g * n_rep) * D;
+  for (int i = tid * 8; i < n_rep * D; i += kThreads * 8) {
+    float f[8];
+    load8(q + i, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) qs[i + e] = f[e];
+  }
+  __syncthreads();
+  const T* kbase = static_cast<const T*>(a.k) + ((int64_t)row_seq(rows, row) * a.kv_heads + g) * a.capacity * D;
+  float* sc = a.scores + ((int64_t)blockIdx.z * a.heads + g * n_rep) * stride;
+  float2* stats = reinterpret_cast<float2*>(a.stats) + ((int64_t)blockIdx.z * splits + split) * a.heads + g * n_rep;
+
+  for (int h0 = 0; h0 < n_rep; h0 += NR) {
+    float mx[NR];
+#pragma unroll
+    for (int r = 0; r < NR; ++r) mx[r] = -INFINITY;
+    for (int ib = i0; ib < i1; ib += 16 * KU) {
+      const T* kp[KU];
+#pragma unroll
+      for (int u = 0; u < KU; ++u) kp[u] = kbase + (int64_t)sp.key(min(ib + slot + 16 * u, i1 - 1)) * D;
+      float acc[NR][KU] = {};
+      for (int c = l8 * 8; c < D; c += 64) {
+        float kf[KU][8];
+#pragma unroll
+        for (int u = 0; u < KU; ++u) load8(kp[u] + c, kf[u]);
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+          float qf[8];
+          load8(qs + (h0 + r) * D + c, qf);
+#pragma unroll
+          for (int u = 0; u < KU; ++u)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc[r][u] = fmaf(qf[e], kf[u][e], acc[r][u]);
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < NR; ++r)
+#pragma unroll
+        for (int u = 0; u < KU; ++u) {
+          float s = acc[r][u];
+          s += __shfl_xor_sync(0xffffffffu, s, 1);
+          s += __shfl_xor_sync(0xffffffffu, s, 2);
+          s += __shfl_xor_sync(0xffffffffu, s, 4);
+          s *= a.scale;
+          const int idx = ib + slot + 16 * u;
+          if (idx < i1) {
+            mx[r] = fmaxf(mx[r], s);
+            if (l8 == 0) sc[(int64_t)(h0 + r) * stride + idx] = s;
+          }
+        }
+    }
+    // range maximum and sum of exponentials per head
+#pragma unroll
+    for (int r = 0; r < NR; ++r) {
+#pragma unroll
+      for (int o = 16; o >= 8; o >>= 1) mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], o));
+      if ((tid & 31) == 0) red[0][r][tid >> 5] = mx[r];
+    }
+    __syncthreads();   // scores of this range visible to the block
+    float sum[NR];
+#pragma unroll
+    for (int r = 0; r < NR; ++r) {
+      mx[r] = fmaxf(fmaxf(red[0][r][0], red[0][r][1]), fmaxf(red[0][r][2], red[0][r][3]));
+      sum[r] = 0.0f;
+      for (int idx = i0 + tid; idx < i1; idx += kThreads) sum[r] += expf(sc[(int64_t)(h0 + r) * stride + idx] - mx[r]);
+      sum[r] = warp_sum(sum[r]);
+      if ((tid & 31) == 0) red[1][r][tid >> 5] = sum[r];
+    }
+    __syncthreads();
+    if (tid < NR) stats[h0 + tid] = make_float2(fmaxf(fmaxf(red[0][tid][0], red[0][tid][1]), fmaxf(red[0][tid][2], red[0][tid][3])),
+                                                red[1][tid][0] + red[1][tid][1] + red[1][tid][2] + red[1][tid][3]);
+    __syncthreads();
+  }
+}
+
+// grid (ranges, kv heads, rows): partial sums of this group's heads over one key range
+template <class T, int NR>
+__global__ void __launch_bounds__(kThreads) mix_values_kernel(const MixAttnArgs a, const Rows rows, int row0, int splits, int stride) {
+  extern __shared__ __align__(16) float sm[];
+  const int tid = threadIdx.x, H = a.heads;
+  const int split = blockIdx.x, g = blockIdx.y, row = row0 + blockIdx.z;
+  const int n_rep = H / a.kv_heads, DV = a.vdim_pad;
+  float* mxs = sm;                          // [H] maximum
+  float* inv = mxs + H;                     // [H] 1 / sum
+  float* talk = inv + H;                    // [n_rep][H]
+  float* p = talk + n_rep * H;              // [H][kTileKeys]
+  float* w = p + H * kTileKeys;             // [n_rep][kTileKeys]
+  float* red = w + n_rep * kTileKeys;       // [slots][8 * vchunks]
+  const Span sp = span_of(row_pos(rows, row), a.window, a.keep_first);
+  const int L = (sp.n + splits - 1) / splits, i0 = min(sp.n, split * L), i1 = min(sp.n, i0 + L);
+  const float2* stats = reinterpret_cast<const float2*>(a.stats) + (int64_t)blockIdx.z * splits * H;
+  for (int h = tid; h < H; h += kThreads) {
+    float M = -INFINITY, S = 0.0f;
+    for (int s = 0; s < splits; ++s) M = fmaxf(M, stats[s * H + h].x);
+    for (int s = 0; s < splits; ++s) {
+      const float2 t = stats[s * H + h];
+      if (t.x > -INFINITY) S += t.y * expf(t.x - M);
+    }
+    mxs[h] = M;
+    inv[h] = 1.0f / S;
+  }
+  for (int i = tid; i < n_rep * H; i += kThreads)
+    talk[i] = a.talk ? a.talk[(g * n_rep) * H + i] : (i / H + g * n_rep == i % H ? 1.0f : 0.0f);
+  __syncthreads();
+
+  const float* sc = a.scores + (int64_t)blockIdx.z * H * stride;
+  const T* vbase = static_cast<const T*>(a.v) + ((int64_t)row_seq(rows, row) * a.kv_heads + g) * a.capacity * DV;
+  const int vchunks = DV / 8, slots = vchunks < kThreads ? kThreads / vchunks : 1;
+  const int slot = tid / vchunks;
+  float* out = a.part + (((int64_t)blockIdx.z * splits + split) * H + g * n_rep) * a.vdim;
+
+  for (int c0 = 0; c0 < vchunks; c0 += kThreads) {   // value sizes above 8 * kThreads take several passes
+    const int chunk = c0 + (vchunks < kThreads ? tid % vchunks : tid);
+    for (int h0 = 0; h0 < n_rep; h0 += NR) {
+      float acc[NR][8] = {};
+      for (int t0 = i0; t0 < i1; t0 += kTileKeys) {
+        const int nt = min(kTileKeys, i1 - t0);
+        for (int i = tid; i < H * kTileKeys; i += kThreads) {
+          const int h = i / kTileKeys, k = i % kTileKeys;
+          p[i] = k < nt ? expf(sc[(int64_t)h * stride + t0 + k] - mxs[h]) * inv[h] : 0.0f;
+        }
+        __syncthreads();
+        for (int i = tid; i < NR * kTileKeys; i += kThreads) {
+          const int r = i / kTileKeys, k = i % kTileKeys;
+          float s = 0.0f;
+          for (int h = 0; h < H; ++h) s = fmaf(talk[(h0 + r) * H + h], p[h * kTileKeys + k], s);
+          w[i] = s;
+        }
+        __syncthreads();
+        if (slot < slots && chunk < vchunks)
+          for (int k = slot; k < nt; k += slots) {
+            float vf[8];
+            load8(vbase + (int64_t)sp.key(t0 + k) * DV + 8 * chunk, vf);
+#pragma unroll
+            for (int r = 0; r < NR; ++r)
+#pragma unroll
+              for (int e = 0; e < 8; ++e) acc[r][e] = fmaf(w[r * kTileKeys + k], vf[e], acc[r][e]);
+          }
+        __syncthreads();
+      }
+      // add the slots
+#pragma unroll
+      for (int r = 0; r < NR; ++r) {
+        if (slot < slots && chunk < vchunks)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) red[slot * 8 * min(vchunks, kThreads) + (chunk - c0) * 8 + e] = acc[r][e];
+        __syncthreads();
+        for (int d = tid; d < 8 * min(vchunks - c0, kThreads); d += kThreads) {
+          float s = 0.0f;
+          for (int k = 0; k < slots; ++k) s += red[k * 8 * min(vchunks, kThreads) + d];
+          if (8 * c0 + d < a.vdim) out[(int64_t)(h0 + r) * a.vdim + 8 * c0 + d] = s;
+        }
+        __syncthreads();
+      }
+    }
+  }
+}
+
+template <class TO>
+__global__ void mix_reduce_kernel(const float* __restrict__ part, int splits, int n, TO* __restrict__ out, int64_t ldo, int row0) {
+  const int i = blockIdx.x * kThreads + threadIdx.x;
+  if (i >= n) return;
+  const float* p = part + (int64_t)blockIdx.y * splits * n + i;
+  float s = 0.0f;
+  for (int k = 0; k < splits; ++k) s += p[(int64_t)k * n];
+  out[(int64_t)(row0 + blockIdx.y) * ldo + i] = to<TO>(s);
+}
+
+int scores_stride(const MixAttnArgs& a) { return (a.max_visible + 3) & ~3; }
+
+size_t values_smem(const MixAttnArgs& a) {
+  const int n_rep = a.heads / a.kv_heads, vchunks = a.vdim_pad / 8;
+  const size_t red = 8 * (size_t)(vchunks < kThreads ? (kThreads / vchunks) * vchunks : kThreads);
+  return 4 * (2 * (size_t)a.heads + (size_t)n_rep * a.heads + (size_t)a.heads * kTileKeys + (size_t)n_rep * kTileKeys + red);
+}
+
+template <class T, int NR>
+cudaError_t launch_rows_nr(const MixAttnArgs& a, const Rows& rows, int row0, int n, int splits, cudaStream_t st) {
+  const int stride = scores_stride(a);
+  const size_t s1 = 4 * (size_t)(a.heads / a.kv_heads) * a.dim_pad, s2 = values_smem(a);
+  if (s1 > 200 * 1024 || s2 > 200 * 1024) return cudaErrorInvalidValue;
+  cudaError_t e = cudaSuccess;
+  if (s1 > 48 * 1024) e = cudaFuncSetAttribute(mix_scores_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
+  if (e == cudaSuccess && s2 > 48 * 1024) e = cudaFuncSetAttribute(mix_values_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
+  if (e != cudaSuccess) return e;
+  const dim3 grid(splits, a.kv_heads, n);
+  mix_scores_kernel<T, NR><<<grid, kThreads, s1, st>>>(a, rows, row0, splits, stride);
+  mix_values_kernel<T, NR><<<grid, kThreads, s2, st>>>(a, rows, row0, splits, stride);
+  return cudaGetLastError();
+}
+
+}  // namespace
+
+int mix_attn_splits(const MixAttnArgs& a, int sm_count) {
+  // about 32 keys per range at least, two blocks per SM at most
+  int s = (a.max_visible + 31) / 32;
+  const int fill = (2 * sm_count + a.kv_heads - 1) / a.kv_heads;
+  if (s > fill) s = fill;
+  if (s > kMixAttnMaxSplits) s = kMixAttnMaxSplits;
+  return s < 1 ? 1 : s;
+}
+
+template <class T, class TO>
+cudaError_t launch_mix_attention_rows(const MixAttnArgs& a, const Rows& rows, TO* out, int64_t ldo, int sm_count, cudaStream_t st, int* launches) {
+  const int splits = rows.n > 64 ? 1 : mix_attn_splits(a, sm_count);
+  const int n_rep = a.heads / a.kv_heads, hv = a.heads * a.vdim;
+  // rows per launch: what the scratch holds
+  const uint64_t per_scores = (uint64_t)a.heads * scores_stride(a), per_stats = 2ull * splits * a.heads, per_part = (uint64_t)splits * hv;
+  uint64_t fit = a.scores_floats / per_scores;
+  if (a.stats_floats / per_stats < fit) fit = a.stats_floats / per_stats;
+  if (a.part_floats / per_part < fit) fit = a.part_floats / per_part;
+  if (fit > 32768) fit = 32768;
+  if (fit < 1) return cudaErrorInvalidValue;
+  for (int r0 = 0; r0 < rows.n; r0 += (int)fit) {
+    const int n = rows.n - r0 < (int)fit ? rows.n - r0 : (int)fit;
+    cudaError_t e;
+    if (n_rep % 8 == 0) e = launch_rows_nr<T, 8>(a, rows, r0, n, splits, st);
+    else if (n_rep % 4 == 0) e = launch_rows_nr<T, 4>(a, rows, r0, n, splits, st);
+    else if (n_rep % 3 == 0) e = launch_rows_nr<T, 3>(a, rows, r0, n, splits, st);
+    else if (n_rep % 2 == 0) e = launch_rows_nr<T, 2>(a, rows, r0, n, splits, st);
+    else e = launch_rows_nr<T, 1>(a, rows, r0, n, splits, st);
+    if (e != cudaSuccess) return e;
+    mix_reduce_kernel<TO><<<dim3((hv + kThreads - 1) / kThreads, n), kThreads, 0, st>>>(a.part, splits, hv, out, ldo, r0);
+    e = cudaGetLastError();
+    if (e != cudaSuccess) return e;
+    *launches += 3;
+  }
+  return cudaSuccess;
+}
+template cudaError_t launch_mix_attention_rows<float, float>(const MixAttnArgs&, const Rows&, float*, int64_t, int, cudaStream_t, int*);
+template cudaError_t launch_mix_attention_rows<__nv_bfloat16, float>(const MixAttnArgs&, const Rows&, float*, int64_t, int, cudaStream_t, int*);
+template cudaError_t launch_mix_attention_rows<__nv_bfloat16, __nv_bfloat16>(const MixAttnArgs&, const Rows&, __nv_bfloat16*, int64_t, int,
+                                                                             cudaStream_t, int*);
+
+bool mix_attention_prompt_supported(const MixAttnArgs&) { return false; }
+cudaError_t launch_mix_attention_prompt(const MixAttnArgs&, const Rows&, int, __nv_bfloat16*, int64_t, cudaStream_t, int*) { return cudaErrorInvalidValue; }
+
+}  // namespace emelb

@@ -1,0 +1,278 @@
+// Row kernels of layered decoders between the products: embedding, residual + layer norm, gated RMS norm, GLU, and the
+// step from an attention layer's projections to its queries and cache rows (short convolution, query / key norm over
+// the whole projection, partial rotation, value norm, store).  f32 arithmetic throughout.
+#include <math.h>
+
+#include "common.cuh"
+#include "layered.h"
+
+namespace emelb {
+namespace {
+
+constexpr int kThreads = 256;
+constexpr int kWarps = kThreads / 32;
+
+template <class T>
+__device__ __forceinline__ T to(float x);
+template <>
+__device__ __forceinline__ float to<float>(float x) { return x; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 to<__nv_bfloat16>(float x) { return __float2bfloat16_rn(x); }
+__device__ __forceinline__ float from(float x) { return x; }
+__device__ __forceinline__ float from(__nv_bfloat16 x) { return __bfloat162float(x); }
+
+__device__ __forceinline__ float block_sum(float v, float* scratch) {
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.0f;
+#pragma unroll
+  for (int w = 0; w < kWarps; ++w) t += scratch[w];
+  return t;
+}
+
+template <class T>
+__global__ void embed_rows_bf16_kernel(const __nv_bfloat16* __restrict__ table, int64_t ld, const int* __restrict__ tokens, int width,
+                                       float* x, T* xb, int64_t ldb) {
+  const int r = blockIdx.x;
+  const __nv_bfloat16* row = table + (int64_t)tokens[r] * ld;
+  for (int i = threadIdx.x; i < width; i += kThreads) {
+    const float v = __bfloat162float(row[i]);
+    x[(int64_t)r * width + i] = v;
+    xb[(int64_t)r * ldb + i] = to<T>(v);
+  }
+}
+
+// layer norm of the vector in shared memory: mean and 1 / sqrt(variance + eps), squared deviations in a second pass
+__device__ __forceinline__ void norm_stats(const float* s, int n, float eps, float* scratch, float& mean, float& inv) {
+  float t = 0.0f;
+  for (int i = threadIdx.x; i < n; i += kThreads) t += s[i];
+  mean = block_sum(t, scratch) / n;
+  t = 0.0f;
+  for (int i = threadIdx.x; i < n; i += kThreads) {
+    const float d = s[i] - mean;
+    t = fmaf(d, d, t);
+  }
+  inv = 1.0f / sqrtf(block_sum(t, scratch) / n + eps);
+}
+
+template <class T>
+__global__ void residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps, int width,
+                                     T* __restrict__ xb, int64_t ldb, float* keep) {
+  extern __shared__ float s[];
+  __shared__ float scratch[kWarps];
+  const int64_t r = blockIdx.x;
+  for (int i = threadIdx.x; i < width; i += kThreads) s[i] = y[r * width + i];
+  float mean, inv;
+  norm_stats(s, width, eps, scratch, mean, inv);
+  for (int i = threadIdx.x; i < width; i += kThreads) {
+    const float v = x[r * width + i] + (s[i] - mean) * inv * w[i];
+    x[r * width + i] = v;
+    xb[r * ldb + i] = to<T>(v);
+    if (keep) keep[r * width + i] = v;
+  }
+}
+
+template <class T>
+__global__ void norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ index, const float* __restrict__ w, float eps, int width,
+                                 T* __restrict__ out, int64_t ldo) {
+  extern __shared__ float s[];
+  __shared__ float scratch[kWarps];
+  const int64_t r = blockIdx.x, src = index ? index[r] : r;
+  for (int i = threadIdx.x; i < width; i += kThreads) s[i] = x[src * width + i];
+  float mean, inv;
+  norm_stats(s, width, eps, scratch, mean, inv);
+  for (int i = threadIdx.x; i < width; i += kThreads) out[r * ldo + i] = to<T>((s[i] - mean) * inv * w[i]);
+}
+
+template <class T>
+__global__ void rms_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, int64_t ldg, float eps,
+                                int width, T* __restrict__ out, int64_t ldo) {
+  __shared__ float scratch[kWarps];
+  const int64_t r = blockIdx.x;
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < width; i += kThreads) {
+    const float v = o[r * width + i];
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / width + eps);
+  for (int i = threadIdx.x; i < width; i += kThreads) out[r * ldo + i] = to<T>(o[r * width + i] * inv * w[i] * from(gate[r * ldg + i]));
+}
+
+__global__ void glu_rows_kernel(const float* __restrict__ gu, int ff, float* __restrict__ out, int64_t ldo) {
+  const int64_t r = blockIdx.y;
+  const int i = blockIdx.x * kThreads + threadIdx.x;
+  if (i >= ff) return;
+  const float g = gu[r * 2 * ff + i], u = gu[r * 2 * ff + ff + i];
+  out[r * ldo + i] = g / (1.0f + expf(-g)) * u;
+}
+
+// One block = one row of the queries (part 0), keys (1) or values (2).
+template <class T>
+__global__ void __launch_bounds__(kThreads) attn_in_kernel(const AttnInArgs a, const Rows rows) {
+  extern __shared__ float s[];
+  __shared__ float scratch[kWarps];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
+  const int pos = rows.prompt ? rows.pos[0] + r : rows.pos[r];
+  const int seq = rows.prompt ? rows.seq0 : rows.seq0 + r;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+  const int n = part == 0 ? nq : part == 1 ? nk : nv, off = part == 0 ? 0 : part == 1 ? nq : nq + nk;
+  const int hist = a.taps - 1;
+
+  float ss = 0.0f;
+  for (int i = tid; i < n; i += kThreads) {
+    const int c = off + i;
+    const float u = a.proj[(int64_t)r * a.channels + c];
+    float y = u;
+    if (a.conv) {
+      const float* w = a.conv + (int64_t)c * a.taps;
+      float* st = a.conv_state + ((int64_t)seq * a.channels + c) * hist;
+      y = w[hist] * u;
+      for (int b = 1; b <= hist; ++b) {   // b tokens back
+        float past = 0.0f;
+        if (pos - b >= 0) past = rows.prompt && r - b >= 0 ? a.proj[(int64_t)(r - b) * a.channels + c] : st[hist - (rows.prompt ? b - r : b)];
+        y = fmaf(w[hist - b], past, y);
+      }
+      if (!rows.prompt) {
+        for (int j = 0; j + 1 < hist; ++j) st[j] = pos - hist + 1 + j >= 0 ? st[j + 1] : 0.0f;
+        if (hist > 0) st[hist - 1] = u;
+      }
+    }
+    s[i] = y;
+    ss = fmaf(y, y, ss);
+  }
+
+  if (part == 2) {
+    __syncthreads();
+    // a warp per value head
+    T* cache = static_cast<T*>(a.v);
+    for (int h = tid >> 5; h < a.kv_heads; h += kWarps) {
+      const float* v = s + h * a.vdim;
+      float inv = 1.0f;
+      if (a.norm_v) {
+        float t = 0.0f;
+        for (int d = tid & 31; d < a.vdim; d += 32) t = fmaf(v[d], v[d], t);
+        inv = 1.0f / sqrtf(warp_sum(t) / a.vdim + a.eps);
+      }
+      T* row = cache + (((int64_t)seq * a.kv_heads + h) * a.capacity + pos) * a.vdim_pad;
+      for (int d = tid & 31; d < a.vdim_pad; d += 32) row[d] = to<T>(d < a.vdim ? v[d] * inv : 0.0f);
+    }
+    return;
+  }
+  const float* nw = part == 0 ? a.norm_q : a.norm_k;
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / n + a.eps);   // also orders the writes of s
+  const int heads = part == 0 ? a.heads : a.kv_heads;
+  auto normed = [&](int i) { return nw ? s[i] * inv * nw[i] : s[i]; };
+  const int half_pad = a.dim_pad / 2;
+  for (int idx = tid; idx < heads * half_pad; idx += kThreads) {
+    const int h = idx / half_pad, p = idx % half_pad, d = 2 * p;
+    float x0 = d < a.dim ? normed(h * a.dim + d) : 0.0f, x1 = d + 1 < a.dim ? normed(h * a.dim + d + 1) : 0.0f;
+    if (d < a.rope_dim) {
+      const int64_t t = (int64_t)pos * (a.rope_dim / 2) + p;
+      const float c = a.rope_cos[t], sn = a.rope_sin[t];
+      const float u = x0 * c - x1 * sn, v = x1 * c + x0 * sn;
+      x0 = u;
+      x1 = v;
+    }
+    T* row = part == 0 ? static_cast<T*>(a.q) + ((int64_t)r * a.heads + h) * a.dim_pad
+                       : static_cast<T*>(a.k) + (((int64_t)seq * a.kv_heads + h) * a.capacity + pos) * a.dim_pad;
+    row[d] = to<T>(x0);
+    row[d + 1] = to<T>(x1);
+  }
+}
+
+__global__ void conv_state_kernel(const AttnInArgs a, const Rows rows) {
+  const int c = blockIdx.x * kThreads + threadIdx.x, hist = a.taps - 1;
+  if (c >= a.channels) return;
+  float* st = a.conv_state + ((int64_t)rows.seq0 * a.channels + c) * hist;
+  // entry j holds the row hist - j before the next one; an old entry moves down by rows.n >= 1 places
+  for (int j = 0; j < hist; ++j) {
+    const int r = rows.n - hist + j;
+    float v = 0.0f;
+    if (r >= 0) v = a.proj[(int64_t)r * a.channels + c];
+    else if (rows.pos[0] + r >= 0) v = st[hist + r];
+    st[j] = v;
+  }
+}
+
+}  // namespace
+
+template <class T>
+cudaError_t launch_embed_rows_bf16(const __nv_bfloat16* table, int64_t ld, const int* tokens, int rows, int width, float* x, T* xb,
+                                   int64_t ldb, cudaStream_t st) {
+  embed_rows_bf16_kernel<T><<<rows, kThreads, 0, st>>>(table, ld, tokens, width, x, xb, ldb);
+  return cudaGetLastError();
+}
+template cudaError_t launch_embed_rows_bf16<float>(const __nv_bfloat16*, int64_t, const int*, int, int, float*, float*, int64_t, cudaStream_t);
+template cudaError_t launch_embed_rows_bf16<__nv_bfloat16>(const __nv_bfloat16*, int64_t, const int*, int, int, float*, __nv_bfloat16*, int64_t,
+                                                           cudaStream_t);
+
+namespace {
+template <class K>
+cudaError_t allow_smem(K kern, size_t bytes) {
+  return bytes > 48 * 1024 ? cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) : cudaSuccess;
+}
+}  // namespace
+
+template <class T>
+cudaError_t launch_residual_norm(float* x, const float* y, const float* w, float eps, int rows, int width, T* xb, int64_t ldb, float* keep,
+                                 cudaStream_t st) {
+  const size_t smem = 4 * (size_t)width;
+  const cudaError_t e = allow_smem(residual_norm_kernel<T>, smem);
+  if (e != cudaSuccess) return e;
+  residual_norm_kernel<T><<<rows, kThreads, smem, st>>>(x, y, w, eps, width, xb, ldb, keep);
+  return cudaGetLastError();
+}
+template cudaError_t launch_residual_norm<float>(float*, const float*, const float*, float, int, int, float*, int64_t, float*, cudaStream_t);
+template cudaError_t launch_residual_norm<__nv_bfloat16>(float*, const float*, const float*, float, int, int, __nv_bfloat16*, int64_t, float*,
+                                                         cudaStream_t);
+
+template <class T>
+cudaError_t launch_norm_rows(const float* x, const int* index, const float* w, float eps, int rows, int width, T* out, int64_t ldo,
+                             cudaStream_t st) {
+  const size_t smem = 4 * (size_t)width;
+  const cudaError_t e = allow_smem(norm_rows_kernel<T>, smem);
+  if (e != cudaSuccess) return e;
+  norm_rows_kernel<T><<<rows, kThreads, smem, st>>>(x, index, w, eps, width, out, ldo);
+  return cudaGetLastError();
+}
+template cudaError_t launch_norm_rows<float>(const float*, const int*, const float*, float, int, int, float*, int64_t, cudaStream_t);
+template cudaError_t launch_norm_rows<__nv_bfloat16>(const float*, const int*, const float*, float, int, int, __nv_bfloat16*, int64_t, cudaStream_t);
+
+template <class T>
+cudaError_t launch_rms_gate(const float* o, const float* w, const T* gate, int64_t ldg, float eps, int rows, int width, T* out, int64_t ldo,
+                            cudaStream_t st) {
+  rms_gate_kernel<T><<<rows, kThreads, 0, st>>>(o, w, gate, ldg, eps, width, out, ldo);
+  return cudaGetLastError();
+}
+template cudaError_t launch_rms_gate<float>(const float*, const float*, const float*, int64_t, float, int, int, float*, int64_t, cudaStream_t);
+template cudaError_t launch_rms_gate<__nv_bfloat16>(const float*, const float*, const __nv_bfloat16*, int64_t, float, int, int, __nv_bfloat16*,
+                                                    int64_t, cudaStream_t);
+
+cudaError_t launch_glu_rows(const float* gu, int rows, int ff, float* out, int64_t ldo, cudaStream_t st) {
+  glu_rows_kernel<<<dim3((ff + kThreads - 1) / kThreads, rows), kThreads, 0, st>>>(gu, ff, out, ldo);
+  return cudaGetLastError();
+}
+
+template <class T>
+cudaError_t launch_attn_in(const AttnInArgs& a, const Rows& rows, cudaStream_t st) {
+  int n = a.heads * a.dim;
+  if (a.own_kv && a.kv_heads * a.vdim > n) n = a.kv_heads * a.vdim;
+  const size_t smem = 4 * (size_t)n;
+  const cudaError_t e = allow_smem(attn_in_kernel<T>, smem);
+  if (e != cudaSuccess) return e;
+  attn_in_kernel<T><<<dim3(rows.n, a.own_kv ? 3 : 1), kThreads, smem, st>>>(a, rows);
+  return cudaGetLastError();
+}
+template cudaError_t launch_attn_in<float>(const AttnInArgs&, const Rows&, cudaStream_t);
+template cudaError_t launch_attn_in<__nv_bfloat16>(const AttnInArgs&, const Rows&, cudaStream_t);
+
+cudaError_t launch_conv_state(const AttnInArgs& a, const Rows& rows, cudaStream_t st) {
+  conv_state_kernel<<<(a.channels + kThreads - 1) / kThreads, kThreads, 0, st>>>(a, rows);
+  return cudaGetLastError();
+}
+
+}  // namespace emelb

@@ -30,6 +30,10 @@ SIGNATURES = {
     "emelb_llama_bind": [_P, C.c_int32, C.c_int32, C.POINTER(eb.View)],
     "emelb_llama_decode": [_P, C.c_int32, C.c_int32, _P, C.POINTER(C.c_int32)],
     "emelb_llama_prefill": [_P, C.POINTER(C.c_int32), C.c_int32, C.c_int32],
+    "emelb_llama_check_layers": [C.POINTER(Config), _P],
+    "emelb_llama_create_layers": [_P, C.POINTER(Config), _P, C.c_int32, C.POINTER(_P)],
+    "emelb_llama_prefill_logits": [_P, C.POINTER(C.c_int32), C.c_int32, C.c_int32, C.POINTER(C.c_int32), C.c_int32, _P],
+    "emelb_llama_trace_layers": [_P, _P, C.c_int32],
     "emelb_llama_generate": [_P, C.c_int32, C.c_int32, C.c_int32, C.POINTER(C.c_int32)],
     "emelb_llama_launches_per_token": [_P, C.POINTER(C.c_int32)],
     "emelb_llama_set_step_mode": [_P, C.c_int32],
@@ -142,6 +146,16 @@ class Session:
     def prefill(self, tokens, start_pos: int = 0) -> bool:
         arr = np.ascontiguousarray(tokens, np.int32)
         return self._ret(eb.lib().emelb_llama_prefill(self._h, arr.ctypes.data_as(C.POINTER(C.c_int32)), arr.size, start_pos))
+
+    def prefill_logits(self, tokens, start_pos: int, want):
+        """prefill() that returns the logits at the places `want` (ascending) among the tokens, [len(want), n_vocab]."""
+        arr, w = np.ascontiguousarray(tokens, np.int32), np.ascontiguousarray(want, np.int32)
+        out = np.zeros((w.size, self.cfg.n_vocab), np.float32)
+        ip = C.POINTER(C.c_int32)
+        if not self._ret(eb.lib().emelb_llama_prefill_logits(self._h, arr.ctypes.data_as(ip), arr.size, start_pos, w.ctypes.data_as(ip), w.size,
+                                                             out.ctypes.data)):
+            raise eb.BackendError(f"prefill_logits failed with error mask {self.last_error}")
+        return out
 
     def generate(self, first_token: int, start_pos: int, n: int):
         out = np.zeros(n, np.int32)

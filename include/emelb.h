@@ -59,6 +59,7 @@ enum {
   EMELB_Q6_K = 14,
   EMELB_Q8_K = 15,
   EMELB_I32 = 26,
+  EMELB_BF16 = 30, /* weights of layered decoder sessions only (emelb_llama.h) */
   EMELB_UNKNOWN = 255
 };
 

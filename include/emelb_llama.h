@@ -70,7 +70,56 @@ enum {
   EMELB_T_FFN_DOWN = 11
 };
 
+/* roles of layered sessions (emelb_llama_create_layers), beside EMELB_T_TOKEN_EMBD, EMELB_T_OUTPUT_NORM,
+ * EMELB_T_OUTPUT, EMELB_T_ATTN_NORM (norm of the mixer's output), EMELB_T_ATTN_OUT, EMELB_T_FFN_NORM (norm of the
+ * feed-forward's output) and EMELB_T_FFN_DOWN */
+enum {
+  EMELB_T_MIX_IN = 12,       /* the mixer's input projections stacked by rows: q|k|v (attention), q (a layer that
+                                borrows keys and values), q|k|v|gate (linear) */
+  EMELB_T_MIX_CONV = 13,     /* f32 [rows of MIX_IN][taps] */
+  EMELB_T_MIX_NORM_Q = 14,   /* f32, over the whole query projection */
+  EMELB_T_MIX_NORM_K = 15,   /* f32, over the whole key projection */
+  EMELB_T_MIX_HEADS = 16,    /* f32 [n_head][n_head]: mixes the heads' attention weights */
+  EMELB_T_MIX_NORM_OUT = 17, /* f32, over the concatenated heads of a linear mixer */
+  EMELB_T_FFN_IN = 18,       /* gate|up stacked by rows */
+  EMELB_T_FFN_IN_BIAS = 19,  /* f32, gate|up */
+  EMELB_T_FFN_DOWN_BIAS = 20 /* f32 */
+};
+
 typedef struct emelb_llama emelb_llama;
+
+/* ---- layered sessions: decoders described layer by layer.  Each layer is a sequence mixer and, optionally, a
+ * gated feed-forward; both read the residual stream itself and the norm (layer norm, weight only) is applied to what
+ * they return: x += norm1(mixer(x)), x += norm2(ff(x)).  Weights are bf16, vectors f32; the residual stream, norms,
+ * attention scores and weights, and recurrent state are f32.  A session of this kind works through the same entry
+ * points as the block-quantized ones (prefill, decode, generate, the batch calls, sequences), with one difference:
+ * its mixers carry state, so a call must continue a sequence at the position where the last one ended, or start it
+ * again at position 0 (which forgets the sequence's state); any other position is EMELB_INVALID_REQUEST. */
+enum {
+  EMELB_MIXER_ATTENTION = 0, /* softmax attention: short causal convolution after the projections, query / key norm over
+                                the whole projection, adjacent-pair RoPE on the first rope_dim dimensions, value norm
+                                per head, sliding window that keeps the sequence's first tokens, mixing of the
+                                heads' weights after the softmax; keys and values may be another layer's */
+  EMELB_MIXER_LINEAR = 1     /* linear attention with a fixed decay per head: S = decay S + k v^T, o = S^T q, with silu
+                                on q, k and v; heads RMS-normed together and gated by sigmoid(gate) */
+};
+typedef struct emelb_layer_config {
+  int32_t mixer;
+  int32_t n_head, n_head_kv; /* n_head_kv: attention only */
+  int32_t key_dim, value_dim;
+  int32_t conv_taps;         /* attention: taps of the short convolution on q, k and v; 0: none */
+  int32_t norm_qk;           /* attention: 1 = query and key norm */
+  int32_t norm_v;            /* attention: 1 = values divided by their root mean square per head */
+  int32_t mix_heads;         /* attention: 1 = heads' weights mixed after the softmax */
+  int32_t rope_dim;          /* rotated dimensions per head (even, 0: none) */
+  float rope_freq_base;
+  float attn_scale;
+  int32_t window;            /* position i sees j with i - j < window (0: all) ... */
+  int32_t keep_first;        /* ... and every j < keep_first */
+  int32_t kv_from;           /* layer whose keys and values are used (-1: this layer's own) */
+  int32_t n_ff;              /* 0: no feed-forward */
+  const float* decay;        /* linear: n_head factors (read by the create call) */
+} emelb_layer_config;
 
 /* pure check of a configuration (no device needed): EMELB_OK or
  * EMELB_INVALID_REQUEST.  Beyond the plain range checks, a sharded layout
@@ -86,6 +135,15 @@ EMELB_API uint32_t emelb_llama_check_config(const emelb_llama_config* cfg);
 EMELB_API uint32_t emelb_llama_create(emelb_ctx* ctx, const emelb_llama_config* cfg,
                                       emelb_llama** out);
 EMELB_API uint32_t emelb_llama_destroy(emelb_llama* s);
+
+/* a layered session.  Of cfg, n_layer, n_embd, n_vocab, n_ctx, rms_eps (every norm's eps) and kv_block are used and
+ * shard_count must be 1.  float32 = 1: activations, products and caches in f32 throughout (no reduced-precision
+ * matrix mode); 0: matrix operands and the key / value cache in bf16 with f32 accumulation.
+ * Matrices are bound as {K, M} views of type EMELB_BF16 whose row stride is a multiple of 16 bytes, with zeros
+ * between K and the stride; vectors as EMELB_F32. */
+EMELB_API uint32_t emelb_llama_check_layers(const emelb_llama_config* cfg, const emelb_layer_config* layers);
+EMELB_API uint32_t emelb_llama_create_layers(emelb_ctx* ctx, const emelb_llama_config* cfg,
+                                             const emelb_layer_config* layers, int32_t float32, emelb_llama** out);
 
 /* binds one tensor (replaces bind_tensor_rows / make_src_view,
  * src/emel/text/generator/detail.hpp:788-817, 1886-1919): a {K, M} view of
@@ -112,6 +170,16 @@ EMELB_API uint32_t emelb_llama_decode(emelb_llama* s, int32_t token, int32_t pos
  * attention modes walk token by token. */
 EMELB_API uint32_t emelb_llama_prefill(emelb_llama* s, const int32_t* tokens, int32_t n,
                                        int32_t start_pos);
+
+/* emelb_llama_prefill that also returns logits: want[0..n_want) are places among the n tokens (ascending), and
+ * logits_out (host) gets n_want rows of n_vocab f32.  Unsharded sessions. */
+EMELB_API uint32_t emelb_llama_prefill_logits(emelb_llama* s, const int32_t* tokens, int32_t n, int32_t start_pos,
+                                              const int32_t* want, int32_t n_want, float* logits_out);
+
+/* layered sessions: the residual stream after every layer for the tokens of the last prefill batch is copied to
+ * `out` (device or host, {n_layer, tokens, n_embd} f32, tokens <= max_tokens) by the following prefill calls; null
+ * turns it off (diagnostics). */
+EMELB_API uint32_t emelb_llama_trace_layers(emelb_llama* s, float* out, int32_t max_tokens);
 
 /* prompt tokens per batch of emelb_llama_prefill: default 2048; 0 or 1 walks the
  * prompt token by token (what the reference does); the first batched prompt sizes
