@@ -3,6 +3,7 @@
 // from zero whatever the memory holds.
 #include "common.cuh"
 #include "layered.h"
+#include "mma_bf16.cuh"
 
 namespace emelb {
 namespace {
@@ -58,7 +59,243 @@ __global__ void __launch_bounds__(kCols * kGroups) linear_attention_rows_kernel(
     for (int i = ty; i < a.dim; i += kGroups) state[(int64_t)i * a.vdim + col] = S[i * kCols + tx];
 }
 
+// ---- prompts on the tensor cores (mma.sync bf16, f32 accumulators), chunk by chunk.  With the state S before a chunk of
+// n tokens:
+//   o_i  = decay^(i+1) S^T q_i + sum_(j<=i) decay^(i-j) (q_i . k_j) v_j
+//   S'   = decay^n S + sum_j decay^(n-1-j) k_j v_j^T
+// q, k and v are bf16; every f32 factor that meets them (the state, the decayed scores, the decayed values) is fed as
+// two bf16 operands, high part and remainder, so the recurrence keeps f32 accuracy.
+// One block = one head x kVS value columns, four warps: 16 query rows each for the outputs, every fourth 16-row tile of
+// the state, which lives in accumulator fragments between the chunks.
+constexpr int kChunk = 64, kVS = 32, kMmaThreads = 128;
+
+template <int D>
+struct ChunkSmem {
+  static constexpr int kRow = D + 8, kVRow = kVS + 8;
+  __nv_bfloat16 q[2][kChunk][kRow], k[2][kChunk][kRow], v[2][kChunk][kVRow];
+  __nv_bfloat16 s_hi[D][kVRow], s_lo[D][kVRow];
+  float pw[kChunk + 1];
+};
+
+template <int D>
+__global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(const LinAttnArgs a, const __nv_bfloat16* __restrict__ x, const Rows rows) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  using Smem = ChunkSmem<D>;
+  Smem& sm = *reinterpret_cast<Smem*>(raw);
+  constexpr int KS = D / 16, MT = (KS + 3) / 4, NT = kVS / 8;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int h = blockIdx.x, v0 = blockIdx.y * kVS;
+  const float decay = a.decay[h];
+  float* state = a.state + ((int64_t)rows.seq0 * a.heads + h) * D * a.vdim;
+  const __nv_bfloat16 *xq = x + h * D, *xk = x + (a.heads + h) * D, *xv = x + 2 * a.heads * D + h * a.vdim + v0;
+
+  auto issue = [&](int c0, int buf) {
+    for (int i = tid; i < kChunk * (D / 8); i += kMmaThreads) {
+      const int r = i / (D / 8), c = i % (D / 8) * 8;
+      const bool live = c0 + r < rows.n;
+      const int64_t at = (int64_t)(live ? c0 + r : 0) * a.ldx + c;
+      cp16_zfill(&sm.q[buf][r][c], xq + at, live);
+      cp16_zfill(&sm.k[buf][r][c], xk + at, live);
+    }
+    for (int i = tid; i < kChunk * (kVS / 8); i += kMmaThreads) {
+      const int r = i / (kVS / 8), c = i % (kVS / 8) * 8;
+      const bool live = c0 + r < rows.n && v0 + c < a.vdim;
+      cp16_zfill(&sm.v[buf][r][c], live ? xv + (int64_t)(c0 + r) * a.ldx + c : xq, live);
+    }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  issue(0, 0);
+  for (int i = tid; i <= kChunk; i += kMmaThreads) sm.pw[i] = powf(decay, (float)i);
+
+  // state rows 16 (warp + 4 mt) + g (+8), columns 8 nt + 2t (+1)
+  float S[MT][NT][4];
+  const bool carried = rows.pos[0] > 0;
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = 16 * (warp + 4 * mt) + g + 8 * (e >> 1), c = 8 * nt + 2 * t + (e & 1);
+        S[mt][nt][e] = carried && r < D && v0 + c < a.vdim ? state[(int64_t)r * a.vdim + v0 + c] : 0.0f;
+      }
+  auto publish = [&]() {
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      if (warp + 4 * mt >= KS) continue;
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          uint32_t hi, lo;
+          split2(S[mt][nt][2 * half], S[mt][nt][2 * half + 1], hi, lo);
+          const int r = 16 * (warp + 4 * mt) + g + 8 * half, c = 8 * nt + 2 * t;
+          *reinterpret_cast<uint32_t*>(&sm.s_hi[r][c]) = hi;
+          *reinterpret_cast<uint32_t*>(&sm.s_lo[r][c]) = lo;
+        }
+    }
+  };
+  publish();
+
+  int buf = 0;
+  for (int c0 = 0; c0 < rows.n; c0 += kChunk, buf ^= 1) {
+    const int n = min(kChunk, rows.n - c0);
+    if (c0 + kChunk < rows.n) {
+      issue(c0 + kChunk, buf ^ 1);
+      asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    }
+    __syncthreads();
+    const int r0 = 16 * warp;   // this warp's query rows
+    if (r0 < n) {
+      float s[kChunk / 8][4] = {}, o[NT][4] = {};
+      const int ktiles = warp + 1;   // keys up to this warp's last row, 16 at a time
+#pragma unroll
+      for (int kk = 0; kk < KS; ++kk) {
+        uint32_t q[4];
+        ldsm(q, &sm.q[buf][r0 + (lane & 15)][16 * kk + (lane >> 4) * 8]);
+#pragma unroll
+        for (int kt = 0; kt < kChunk / 16; ++kt) {
+          if (kt >= ktiles) break;
+          uint32_t b[4];
+          ldsm(b, &sm.k[buf][16 * kt + (lane & 7) + (lane >> 4) * 8][16 * kk + ((lane >> 3) & 1) * 8]);
+          mma_bf16_16816(s[2 * kt], q, b[0], b[1]);
+          mma_bf16_16816(s[2 * kt + 1], q, b[2], b[3]);
+        }
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np) {
+          uint32_t b[4];
+          ldsm_trans(b, &sm.s_hi[16 * kk + (lane & 15)][16 * np + (lane >> 4) * 8]);
+          mma_bf16_16816(o[2 * np], q, b[0], b[1]);
+          mma_bf16_16816(o[2 * np + 1], q, b[2], b[3]);
+          ldsm_trans(b, &sm.s_lo[16 * kk + (lane & 15)][16 * np + (lane >> 4) * 8]);
+          mma_bf16_16816(o[2 * np], q, b[0], b[1]);
+          mma_bf16_16816(o[2 * np + 1], q, b[2], b[3]);
+        }
+      }
+      const float d0 = sm.pw[r0 + g + 1], d1 = sm.pw[r0 + g + 9];
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        o[nt][0] *= d0;
+        o[nt][1] *= d0;
+        o[nt][2] *= d1;
+        o[nt][3] *= d1;
+      }
+#pragma unroll
+      for (int kt = 0; kt < kChunk / 16; ++kt) {
+        if (kt >= ktiles) break;
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int i = r0 + g + 8 * half, j = 16 * kt + 8 * part + 2 * t;
+            const float* p = s[2 * kt + part];
+            const float p0 = j <= i ? p[2 * half] * sm.pw[i - j] : 0.0f, p1 = j + 1 <= i ? p[2 * half + 1] * sm.pw[i - j - 1] : 0.0f;
+            split2(p0, p1, hi[2 * part + half], lo[2 * part + half]);
+          }
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np) {
+          uint32_t b[4];
+          ldsm_trans(b, &sm.v[buf][16 * kt + (lane & 15)][16 * np + (lane >> 4) * 8]);
+          mma_bf16_16816(o[2 * np], hi, b[0], b[1]);
+          mma_bf16_16816(o[2 * np], lo, b[0], b[1]);
+          mma_bf16_16816(o[2 * np + 1], hi, b[2], b[3]);
+          mma_bf16_16816(o[2 * np + 1], lo, b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = c0 + r0 + g + 8 * half;
+        if (i >= rows.n) continue;
+        float* out = a.out + ((int64_t)i * a.heads + h) * a.vdim + v0;
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          const int c = 8 * nt + 2 * t;
+          if (v0 + c < a.vdim) *reinterpret_cast<float2*>(out + c) = make_float2(o[nt][2 * half], o[nt][2 * half + 1]);
+        }
+      }
+    }
+    // the state after this chunk
+    const float dn = sm.pw[n];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[mt][nt][e] *= dn;
+#pragma unroll
+    for (int kt = 0; kt < kChunk / 16; ++kt) {
+      if (16 * kt >= n) break;
+      // decayed values of these 16 tokens; the rows past the end are zero
+      uint32_t hi[NT][2], lo[NT][2];
+#pragma unroll
+      for (int np = 0; np < NT / 2; ++np) {
+        uint32_t b[4];
+        ldsm_trans(b, &sm.v[buf][16 * kt + (lane & 15)][16 * np + (lane >> 4) * 8]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int j = 16 * kt + 8 * (i & 1) + 2 * t;
+          const float2 v = unpack2(b[i]);
+          const float w0 = j < n ? sm.pw[n - 1 - j] : 0.0f, w1 = j + 1 < n ? sm.pw[n - 2 - j] : 0.0f;
+          split2(v.x * w0, v.y * w1, hi[2 * np + (i >> 1)][i & 1], lo[2 * np + (i >> 1)][i & 1]);
+        }
+      }
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+        if (warp + 4 * mt >= KS) continue;
+        uint32_t k[4];
+        ldsm_trans(k, &sm.k[buf][16 * kt + (lane & 7) + (lane >> 4) * 8][16 * (warp + 4 * mt) + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          mma_bf16_16816(S[mt][nt], k, hi[nt][0], hi[nt][1]);
+          mma_bf16_16816(S[mt][nt], k, lo[nt][0], lo[nt][1]);
+        }
+      }
+    }
+    __syncthreads();   // every warp is done with this chunk and with the old state
+    publish();
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = 16 * (warp + 4 * mt) + g + 8 * (e >> 1), c = 8 * nt + 2 * t + (e & 1);
+        if (r < D && v0 + c < a.vdim) state[(int64_t)r * a.vdim + v0 + c] = S[mt][nt][e];
+      }
+}
+
+template <int D>
+cudaError_t launch_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, cudaStream_t st) {
+  const int smem = (int)sizeof(ChunkSmem<D>);
+  const cudaError_t e = cudaFuncSetAttribute(linear_attention_prompt_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return e;
+  linear_attention_prompt_kernel<D><<<dim3(a.heads, (a.vdim + kVS - 1) / kVS), kMmaThreads, smem, st>>>(a, x, rows);
+  return cudaGetLastError();
+}
+
 }  // namespace
+
+bool linear_attention_prompt_supported(const LinAttnArgs& a) {
+  return a.dim % 16 == 0 && a.dim <= 128 && a.vdim % 8 == 0 && a.ldx % 8 == 0;
+}
+
+cudaError_t launch_linear_attention_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, cudaStream_t st) {
+  switch (a.dim / 16) {
+    case 1: return launch_prompt<16>(a, x, rows, st);
+    case 2: return launch_prompt<32>(a, x, rows, st);
+    case 3: return launch_prompt<48>(a, x, rows, st);
+    case 4: return launch_prompt<64>(a, x, rows, st);
+    case 5: return launch_prompt<80>(a, x, rows, st);
+    case 6: return launch_prompt<96>(a, x, rows, st);
+    case 7: return launch_prompt<112>(a, x, rows, st);
+    case 8: return launch_prompt<128>(a, x, rows, st);
+    default: return cudaErrorInvalidValue;
+  }
+}
 
 template <class T>
 cudaError_t launch_linear_attention_rows(const LinAttnArgs& a, const T* x, const Rows& rows, cudaStream_t st) {
@@ -73,8 +310,5 @@ cudaError_t launch_linear_attention_rows(const LinAttnArgs& a, const T* x, const
 }
 template cudaError_t launch_linear_attention_rows<float>(const LinAttnArgs&, const float*, const Rows&, cudaStream_t);
 template cudaError_t launch_linear_attention_rows<__nv_bfloat16>(const LinAttnArgs&, const __nv_bfloat16*, const Rows&, cudaStream_t);
-
-bool linear_attention_prompt_supported(const LinAttnArgs&) { return false; }
-cudaError_t launch_linear_attention_prompt(const LinAttnArgs&, const __nv_bfloat16*, const Rows&, cudaStream_t) { return cudaErrorInvalidValue; }
 
 }  // namespace emelb

@@ -11,6 +11,7 @@
 
 #include "common.cuh"
 #include "layered.h"
+#include "mma_bf16.cuh"
 
 namespace emelb {
 namespace {
@@ -298,7 +299,290 @@ template cudaError_t launch_mix_attention_rows<__nv_bfloat16, float>(const MixAt
 template cudaError_t launch_mix_attention_rows<__nv_bfloat16, __nv_bfloat16>(const MixAttnArgs&, const Rows&, __nv_bfloat16*, int64_t, int,
                                                                              cudaStream_t, int*);
 
-bool mix_attention_prompt_supported(const MixAttnArgs&) { return false; }
-cudaError_t launch_mix_attention_prompt(const MixAttnArgs&, const Rows&, int, __nv_bfloat16*, int64_t, cudaStream_t, int*) { return cudaErrorInvalidValue; }
+// ---- prompts on the tensor cores (mma.sync bf16).  A strip of consecutive query rows at a time, so that the scores of
+// every head stay in the L2 cache between three launches:
+//   scores   q . k * scale of 64 rows x 64 key columns, all heads of a key/value head per block
+//   mix      per row: softmax of every head over its visible columns, heads mixed in f32; each weight is left as two
+//            bf16 parts (high, remainder) in the place of its score, invisible columns as zero
+//   values   weights x value rows, both parts
+// Column c of a strip is key c for c < kk (kept tokens below the strip's first window), else key lo + c - kk.
+namespace {
+
+constexpr int kQT = 64, kCT = 64, kMmaThreads = 128;
+
+struct Strip {
+  int row0, rows;      // rows of the batch
+  int pos0;            // position of row0
+  int lo, kk, cols;    // key columns; cols_pad: columns rounded up to whole tiles
+  int cols_pad;
+};
+
+__device__ __forceinline__ int strip_key(const Strip& s, int c) { return c < s.kk ? c : s.lo + c - s.kk; }
+
+// whether any of the strip's rows [i0, i0 + 64) sees a column of [c0, c0 + 64)
+__device__ __forceinline__ bool tile_visible(const Strip& s, int i0, int c0, int window, int keep) {
+  const int p0 = s.pos0 + i0, p1 = s.pos0 + min(i0 + kQT, s.rows) - 1;
+  const int c1 = min(c0 + kCT, s.cols) - 1;
+  if (c1 < c0) return false;
+  const int k0 = strip_key(s, c0), k1 = strip_key(s, c1);
+  if (k0 > p1) return false;
+  return k0 < keep || window <= 0 || p0 - k1 < window;
+}
+
+__global__ void __launch_bounds__(kMmaThreads) mix_prompt_scores_kernel(const MixAttnArgs a, const int seq, const Strip s) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int D = a.dim_pad, row_halves = D + 8;
+  __nv_bfloat16* qt = reinterpret_cast<__nv_bfloat16*>(raw);      // [64][D + 8]
+  __nv_bfloat16* kt = qt + kQT * row_halves;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int c0 = blockIdx.x * kCT, i0 = blockIdx.y * kQT, kh = blockIdx.z, n_rep = a.heads / a.kv_heads;
+  if (!tile_visible(s, i0, c0, a.window, a.keep_first)) return;
+  const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
+  const __nv_bfloat16* k = static_cast<const __nv_bfloat16*>(a.k) + ((int64_t)seq * a.kv_heads + kh) * a.capacity * D;
+  const int chunks = D / 8;
+  for (int i = tid; i < kCT * chunks; i += kMmaThreads) {
+    const int r = i / chunks, c = i % chunks * 8;
+    const bool live = c0 + r < s.cols;
+    cp16_zfill(kt + r * row_halves + c, k + (live ? (int64_t)strip_key(s, c0 + r) * D + c : 0), live);
+  }
+  for (int rep = 0; rep < n_rep; ++rep) {
+    const int h = kh * n_rep + rep;
+    for (int i = tid; i < kQT * chunks; i += kMmaThreads) {
+      const int r = i / chunks, c = i % chunks * 8;
+      const bool live = i0 + r < s.rows;
+      cp16_zfill(qt + r * row_halves + c, q + (live ? ((int64_t)(s.row0 + i0 + r) * a.heads + h) * D + c : 0), live);
+    }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    __syncthreads();
+    float acc[kCT / 8][4] = {};
+    for (int kk = 0; kk < D / 16; ++kk) {
+      uint32_t qa[4];
+      ldsm(qa, qt + (16 * warp + (lane & 15)) * row_halves + 16 * kk + (lane >> 4) * 8);
+#pragma unroll
+      for (int nt = 0; nt < kCT / 16; ++nt) {
+        uint32_t b[4];
+        ldsm(b, kt + (16 * nt + (lane & 7) + (lane >> 4) * 8) * row_halves + 16 * kk + ((lane >> 3) & 1) * 8);
+        mma_bf16_16816(acc[2 * nt], qa, b[0], b[1]);
+        mma_bf16_16816(acc[2 * nt + 1], qa, b[2], b[3]);
+      }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = i0 + 16 * warp + g + 8 * half;
+      if (i >= s.rows) continue;
+      float* out = a.scores + ((int64_t)i * a.heads + h) * s.cols_pad + c0;
+#pragma unroll
+      for (int nt = 0; nt < kCT / 8; ++nt)
+        *reinterpret_cast<float2*>(out + 8 * nt + 2 * t) = make_float2(acc[nt][2 * half] * a.scale, acc[nt][2 * half + 1] * a.scale);
+    }
+    __syncthreads();   // the query tile is replaced
+  }
+}
+
+constexpr int kMixThreads = 256;
+
+// one block per row; HM >= heads
+template <int HM>
+__global__ void __launch_bounds__(kMixThreads) mix_prompt_weights_kernel(const MixAttnArgs a, const Strip s) {
+  __shared__ __align__(16) float talk[HM * HM];
+  __shared__ float mx[HM], inv[HM];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, H = a.heads;
+  const int i = blockIdx.x, pos = s.pos0 + i;
+  const int lo = a.window > 0 && pos - a.window + 1 > 0 ? pos - a.window + 1 : 0;
+  const int kept = min(a.keep_first, lo);                 // columns [0, kept) and [w0, w1]
+  const int w0 = s.kk + lo - s.lo, w1 = s.kk + pos - s.lo, n = kept + w1 - w0 + 1;
+  float* sc = a.scores + (int64_t)i * H * s.cols_pad;
+  for (int x = tid; x < HM * HM; x += kMixThreads) {
+    const int h = x / HM, g = x % HM;
+    talk[x] = h < H && g < H ? (a.talk ? a.talk[h * H + g] : (h == g ? 1.0f : 0.0f)) : 0.0f;
+  }
+  for (int h = warp; h < H; h += kMixThreads / 32) {
+    const float* row = sc + (int64_t)h * s.cols_pad;
+    float m = -INFINITY;
+    for (int c = lane; c < n; c += 32) m = fmaxf(m, row[c < kept ? c : w0 + c - kept]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    float sum = 0.0f;
+    for (int c = lane; c < n; c += 32) sum += expf(row[c < kept ? c : w0 + c - kept] - m);
+    sum = warp_sum(sum);
+    if (lane == 0) {
+      mx[h] = m;
+      inv[h] = 1.0f / sum;
+    }
+  }
+  __syncthreads();
+  const int q_tile = i / kQT * kQT;
+  for (int c = tid; c < s.cols_pad; c += kMixThreads) {
+    float* col = sc + c;
+    if (!(c < kept || (c >= w0 && c <= w1))) {
+      if (tile_visible(s, q_tile, c / kCT * kCT, a.window, a.keep_first))
+        for (int h = 0; h < H; ++h) reinterpret_cast<uint32_t*>(col)[(int64_t)h * s.cols_pad] = 0u;
+      continue;
+    }
+    float p[HM];
+#pragma unroll
+    for (int h = 0; h < HM; ++h) p[h] = h < H ? expf(col[(int64_t)h * s.cols_pad] - mx[h]) * inv[h] : 0.0f;
+#pragma unroll 4
+    for (int h = 0; h < H; ++h) {
+      float w = 0.0f;
+#pragma unroll
+      for (int g = 0; g < HM; g += 4) {
+        const float4 tk = *reinterpret_cast<const float4*>(talk + h * HM + g);
+        w = fmaf(tk.x, p[g], w);
+        w = fmaf(tk.y, p[g + 1], w);
+        w = fmaf(tk.z, p[g + 2], w);
+        w = fmaf(tk.w, p[g + 3], w);
+      }
+      const __nv_bfloat16 hi = __float2bfloat16_rn(w), rest = __float2bfloat16_rn(w - __bfloat162float(hi));
+      reinterpret_cast<uint32_t*>(col)[(int64_t)h * s.cols_pad] = (uint32_t)__bfloat16_as_ushort(hi) | (uint32_t)__bfloat16_as_ushort(rest) << 16;
+    }
+  }
+}
+
+// grid (query tiles, heads, blocks of 8 NT value columns)
+template <int NT>
+struct ValuesSmem {
+  static constexpr int kWRow = kCT + 4, kVRow = 8 * NT + 8;
+  uint32_t w[2][kQT][kWRow];
+  __nv_bfloat16 v[2][kCT][kVRow];
+};
+template <int NT>
+__global__ void __launch_bounds__(kMmaThreads) mix_prompt_values_kernel(const MixAttnArgs a, const int seq, const Strip s, __nv_bfloat16* __restrict__ out,
+                                                                        int64_t ldo) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  ValuesSmem<NT>& sm = *reinterpret_cast<ValuesSmem<NT>*>(raw);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int i0 = blockIdx.x * kQT, h = blockIdx.y, v0 = blockIdx.z * 8 * NT, n_rep = a.heads / a.kv_heads;
+  const uint32_t* w = reinterpret_cast<const uint32_t*>(a.scores);
+  const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(a.v) + ((int64_t)seq * a.kv_heads + h / n_rep) * a.capacity * a.vdim_pad;
+  auto issue = [&](int c0, int buf) {
+    for (int i = tid; i < kQT * (kCT / 4); i += kMmaThreads) {
+      const int r = i / (kCT / 4), c = i % (kCT / 4) * 4;
+      const bool live = i0 + r < s.rows;
+      cp16_zfill(&sm.w[buf][r][c], w + (live ? ((int64_t)(i0 + r) * a.heads + h) * s.cols_pad + c0 + c : 0), live);
+    }
+    for (int i = tid; i < kCT * NT; i += kMmaThreads) {
+      const int r = i / NT, c = i % NT * 8;
+      const bool live = c0 + r < s.cols && v0 + c < a.vdim_pad;
+      cp16_zfill(&sm.v[buf][r][c], v + (live ? (int64_t)strip_key(s, c0 + r) * a.vdim_pad + v0 + c : 0), live);
+    }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  auto next = [&](int c0) {
+    while (c0 < s.cols_pad && !tile_visible(s, i0, c0, a.window, a.keep_first)) c0 += kCT;
+    return c0;
+  };
+  float acc[NT][4] = {};
+  int c0 = next(0), buf = 0;
+  if (c0 < s.cols_pad) issue(c0, 0);
+  while (c0 < s.cols_pad) {
+    const int c1 = next(c0 + kCT);
+    if (c1 < s.cols_pad) {
+      issue(c1, buf ^ 1);
+      asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < kCT / 16; ++kk) {
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int part = 0; part < 4; ++part) {
+        const uint2 x = *reinterpret_cast<const uint2*>(&sm.w[buf][16 * warp + g + 8 * (part & 1)][16 * kk + 2 * t + 8 * (part >> 1)]);
+        hi[part] = __byte_perm(x.x, x.y, 0x5410);
+        lo[part] = __byte_perm(x.x, x.y, 0x7632);
+      }
+#pragma unroll
+      for (int np = 0; np < NT / 2; ++np) {
+        uint32_t b[4];
+        ldsm_trans(b, &sm.v[buf][16 * kk + (lane & 15)][16 * np + (lane >> 4) * 8]);
+        mma_bf16_16816(acc[2 * np], hi, b[0], b[1]);
+        mma_bf16_16816(acc[2 * np], lo, b[0], b[1]);
+        mma_bf16_16816(acc[2 * np + 1], hi, b[2], b[3]);
+        mma_bf16_16816(acc[2 * np + 1], lo, b[2], b[3]);
+      }
+    }
+    __syncthreads();
+    c0 = c1;
+    buf ^= 1;
+  }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int i = i0 + 16 * warp + g + 8 * half;
+    if (i >= s.rows) continue;
+    __nv_bfloat16* o = out + (int64_t)(s.row0 + i) * ldo + h * a.vdim;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int c = v0 + 8 * nt + 2 * t + e;
+        if (c < a.vdim) o[c] = __float2bfloat16_rn(acc[nt][2 * half + e]);
+      }
+  }
+}
+
+template <int NT>
+cudaError_t launch_prompt_values(const MixAttnArgs& a, int seq, const Strip& s, __nv_bfloat16* out, int64_t ldo, cudaStream_t st) {
+  const int smem = (int)sizeof(ValuesSmem<NT>);
+  const cudaError_t e = cudaFuncSetAttribute(mix_prompt_values_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return e;
+  mix_prompt_values_kernel<NT><<<dim3((s.rows + kQT - 1) / kQT, a.heads, (a.vdim_pad + 8 * NT - 1) / (8 * NT)), kMmaThreads, smem, st>>>(a, seq, s, out, ldo);
+  return cudaGetLastError();
+}
+
+// key columns of the strip of `rows` query rows from position pos0
+Strip make_strip(const MixAttnArgs& a, int row0, int rows, int pos0) {
+  Strip s{};
+  s.row0 = row0;
+  s.rows = rows;
+  s.pos0 = pos0;
+  s.lo = a.window > 0 && pos0 - a.window + 1 > 0 ? pos0 - a.window + 1 : 0;
+  s.kk = a.keep_first < s.lo ? a.keep_first : s.lo;
+  s.cols = s.kk + pos0 + rows - s.lo;
+  s.cols_pad = (s.cols + kCT - 1) / kCT * kCT;
+  return s;
+}
+
+}  // namespace
+
+bool mix_attention_prompt_supported(const MixAttnArgs& a) {
+  // one tile of query rows must fit the scratch
+  const uint64_t widest = ((uint64_t)a.max_visible + 2 * kQT + kCT) * a.heads * kQT;
+  return a.heads <= 64 && a.dim_pad % 16 == 0 && a.dim_pad <= 256 && widest <= a.scores_floats;
+}
+
+cudaError_t launch_mix_attention_prompt(const MixAttnArgs& a, const Rows& rows, int pos0, __nv_bfloat16* out, int64_t ldo, cudaStream_t st,
+                                        int* launches) {
+  const int smem = 2 * kQT * (a.dim_pad + 8) * 2;
+  cudaError_t e = cudaSuccess;
+  if (smem > 48 * 1024) e = cudaFuncSetAttribute(mix_prompt_scores_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  for (int r0 = 0; e == cudaSuccess && r0 < rows.n;) {
+    // as many 64-row tiles as the scratch holds, at most 256 rows (a longer strip adds columns few of its rows see)
+    int n = rows.n - r0 < kQT ? rows.n - r0 : kQT;
+    Strip s = make_strip(a, r0, n, pos0 + r0);
+    while (n < rows.n - r0 && n < 256) {
+      const int more = rows.n - r0 < n + kQT ? rows.n - r0 : n + kQT;
+      const Strip t = make_strip(a, r0, more, pos0 + r0);
+      if ((uint64_t)t.rows * a.heads * t.cols_pad > a.scores_floats) break;
+      n = more;
+      s = t;
+    }
+    mix_prompt_scores_kernel<<<dim3(s.cols_pad / kCT, (n + kQT - 1) / kQT, a.kv_heads), kMmaThreads, smem, st>>>(a, rows.seq0, s);
+    if (a.heads <= 8) mix_prompt_weights_kernel<8><<<n, kMixThreads, 0, st>>>(a, s);
+    else if (a.heads <= 16) mix_prompt_weights_kernel<16><<<n, kMixThreads, 0, st>>>(a, s);
+    else if (a.heads <= 32) mix_prompt_weights_kernel<32><<<n, kMixThreads, 0, st>>>(a, s);
+    else mix_prompt_weights_kernel<64><<<n, kMixThreads, 0, st>>>(a, s);
+    e = cudaGetLastError();
+    if (e != cudaSuccess) break;
+    if (a.vdim_pad <= 32) e = launch_prompt_values<4>(a, rows.seq0, s, out, ldo, st);
+    else if (a.vdim_pad <= 64) e = launch_prompt_values<8>(a, rows.seq0, s, out, ldo, st);
+    else e = launch_prompt_values<16>(a, rows.seq0, s, out, ldo, st);
+    *launches += 3;
+    r0 += n;
+  }
+  return e;
+}
 
 }  // namespace emelb

@@ -80,7 +80,10 @@ class Session(el.Session):
             self.be.evict(t)
         self._tensors, self._keep = [], []
 
-    def _upload(self, tensor_id: int, host: np.ndarray, t: int) -> int:
+    def _upload(self, host: np.ndarray, t: int) -> int:
+        # residency ids above the ones files' tensors get, never used twice on a backend
+        tensor_id = getattr(self.be, "next_layered_tensor", 1 << 24)
+        self.be.next_layered_tensor = tensor_id + 1
         dev = self.be.upload(tensor_id, host, tensor_type=t)
         self._tensors.append(tensor_id)
         self._keep.append(host)   # its address is the residency key
@@ -96,18 +99,18 @@ class Session(el.Session):
     def bind_vector_at(self, layer: int, role: int, dev: int, n: int, rows: int = 1) -> bool:
         return self._bind(layer, role, eb.strided_view(dev, eb.F32, [n, rows, 1, 1], [4, 4 * n, 4 * n * rows, 4 * n * rows]))
 
-    def load_matrix(self, tensor_id: int, layer: int, role: int, bits: np.ndarray) -> bool:
+    def load_matrix(self, layer: int, role: int, bits: np.ndarray) -> bool:
         """bits: bf16 bit patterns [rows, k]; rows are padded to 16 bytes."""
         rows, k = bits.shape
         ld = (k + 7) // 8 * 8
         host = np.zeros((rows, ld), np.uint16)
         host[:, :k] = bits
-        return self.bind_matrix_at(layer, role, self._upload(tensor_id, host, eb.BF16), rows, k, ld)
+        return self.bind_matrix_at(layer, role, self._upload(host, eb.BF16), rows, k, ld)
 
-    def load_vector(self, tensor_id: int, layer: int, role: int, values: np.ndarray) -> bool:
+    def load_vector(self, layer: int, role: int, values: np.ndarray) -> bool:
         host = np.array(values, np.float32, order="C", copy=True)
         rows, n = (1, host.shape[0]) if host.ndim == 1 else host.shape
-        return self.bind_vector_at(layer, role, self._upload(tensor_id, host, eb.F32), n, rows)
+        return self.bind_vector_at(layer, role, self._upload(host, eb.F32), n, rows)
 
     def trace_layers(self, max_tokens: int):
         """Array the following prompt batches write their residual streams to ({n_layer, tokens, n_embd} packed at its

@@ -40,24 +40,23 @@ def session_config(cfg: dict, n_ctx: int) -> el.Config:
     return ly.config(len(cfg["layers"]), cfg["width"], cfg["vocab"], n_ctx, cfg["norm"]["eps"])
 
 
-def load(backend: eb.Backend, path: str, n_ctx: int = 4096, float32: bool = False, first_tensor_id: int = 0) -> ly.Session:
+def load(backend: eb.Backend, path: str, n_ctx: int = 4096, float32: bool = False) -> ly.Session:
     with open(os.path.join(path, "config.json")) as f:
         cfg = json.load(f)
-    return load_tensors(backend, cfg, st.File(os.path.join(path, "model.safetensors")), n_ctx, float32, first_tensor_id)
+    return load_tensors(backend, cfg, st.File(os.path.join(path, "model.safetensors")), n_ctx, float32)
 
 
-def load_tensors(backend: eb.Backend, cfg: dict, f: st.File, n_ctx: int, float32: bool = False, first_tensor_id: int = 0) -> ly.Session:
+def load_tensors(backend: eb.Backend, cfg: dict, f: st.File, n_ctx: int, float32: bool = False) -> ly.Session:
     """Uploads and binds every tensor; a layer's input projections and its gate and up projections are stacked."""
     layers = layer_configs(cfg)
     sess = ly.Session(backend, session_config(cfg, n_ctx), layers, float32)
-    ids = iter(range(first_tensor_id, 1 << 30))
 
     def matrix(layer, role, *names):
-        if not sess.load_matrix(next(ids), layer, role, np.concatenate([f.bf16(n) for n in names])):
+        if not sess.load_matrix(layer, role, np.concatenate([f.bf16(n) for n in names])):
             raise ValueError(f"tensor {'|'.join(names)} does not fit the configuration")
 
     def vector(layer, role, *names):
-        if not sess.load_vector(next(ids), layer, role, np.concatenate([f.f32(n) for n in names])):
+        if not sess.load_vector(layer, role, np.concatenate([f.f32(n) for n in names])):
             raise ValueError(f"tensor {'|'.join(names)} does not fit the configuration")
 
     try:

@@ -106,22 +106,28 @@ def lightning_mixer(x, w, p, m, eps):
 
 def attention_mixer(x, w, p, m, eps, lent):
     """lent: layer index -> (keys as cached, values after the convolution) of the layers before; returns the output and
-    this layer's own entry (None for a layer that borrows)."""
+    this layer's own entry (None for a layer that borrows).  A mechanism whose tensors are missing is left out."""
     T, H, G = len(x), m["heads"], m["kv_heads"]
-    rot = m["rot"]
-    q = rms_norm(short_conv(x @ w[p + "q"].T, w[p + "q.conv"]), w[p + "q.norm"], eps).reshape(T, H, m["dim"])
-    q = rotate(q, rot["dims"], rot["base"])
+    rot = m.get("rot") or {"dims": 0, "base": 1.0}
+
+    def projected(name):
+        u = x @ w[p + name].T
+        return short_conv(u, w[p + name + ".conv"]) if p + name + ".conv" in w else u
+
+    def normed(u, name):
+        return rms_norm(u, w[p + name + ".norm"], eps) if p + name + ".norm" in w else u
+
+    q = rotate(normed(projected("q"), "q").reshape(T, H, m["dim"]), rot["dims"], rot["base"])
     own = None
     if m.get("kv_from") is None:
-        k = rms_norm(short_conv(x @ w[p + "k"].T, w[p + "k.conv"]), w[p + "k.norm"], eps).reshape(T, G, m["dim"])
-        k = rotate(k, rot["dims"], rot["base"])
-        raw = short_conv(x @ w[p + "v"].T, w[p + "v.conv"]).reshape(T, G, m["vdim"])
-        v = rms_norm(raw, None, eps)
+        k = rotate(normed(projected("k"), "k").reshape(T, G, m["dim"]), rot["dims"], rot["base"])
+        raw = projected("v").reshape(T, G, m["vdim"])
         own = (k, raw)
     else:
         k, raw = lent[m["kv_from"]]
-        v = rms_norm(raw, None, eps)
-    o = talking_attention(q, k, v, m["scale"], m.get("mask"), w[p + "talk"])
+    v = rms_norm(raw, None, eps) if m.get("norm_v", True) else raw
+    talk = w[p + "talk"] if p + "talk" in w else np.eye(H)
+    o = talking_attention(q, k, v, m["scale"], m.get("mask"), talk)
     return o.reshape(T, -1) @ w[p + "o"].T, own
 
 
