@@ -818,6 +818,150 @@ def time_cfg1_matvec(be, timed_region, copies=68):
     return ms * 1e3 / (5 * copies), wbytes + 4672 + 4 * m
 
 
+# ------------------------------------------------------------------ layered decoders beside the block-quantized one
+# layers of real models' sizes, four lightning and four attention layers (two of them on the layer's keys and values
+# before); the Llama session beside them has the same width, feed-forward, heads and layer count in Q4_K
+METULIX_SHAPES = {
+    "2b": dict(width=2048, ff=8192, heads=16, kv_heads=4, dim=128, vocab=32000, window=1024, keep=4, layers=8),
+    "8b": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, vocab=32000, window=1024, keep=4, layers=8),
+    "8b-full": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, vocab=32000, window=0, keep=0, layers=8),
+}
+
+
+def build_metulix_session(be, sh, n_ctx, seed0=7000):
+    """Random weights (N(0, 1/K) in bf16, norm weights and convolution taps 1) -> (session, weight bytes, allocations)."""
+    import emel_cpp_b200 as eb
+    from emel_cpp_b200 import layered as ly
+    from emel_cpp_b200 import llama as el
+    W, H, G, D, ff = sh["width"], sh["heads"], sh["kv_heads"], sh["dim"], sh["ff"]
+    decay = [1.0 - 2.0 ** (-1.0 - 8.0 * h / H) for h in range(H)]
+    layers = []
+    for i in range(sh["layers"]):
+        if i % 2 == 0:
+            layers.append(ly.linear_layer(H, D, D, decay, n_ff=ff))
+        else:
+            layers.append(ly.attention_layer(H, G, D, D, D ** -0.5, conv_taps=3, rope_dim=D, rope_freq_base=20000.0, window=sh["window"],
+                                             keep_first=sh["keep"], kv_from=i - 2 if i % 4 == 3 else -1, n_ff=ff))
+    sess = ly.Session(be, ly.config(len(layers), W, sh["vocab"], n_ctx, 1e-6), layers)
+    allocs, weight_bytes = [], 0
+    ones = be.alloc(4 * 65536)
+    assert be.to_device(ones, np.ones(65536, np.float32))
+    allocs.append(ones)
+
+    def mat(layer, role, rows, k):
+        nonlocal weight_bytes
+        d = be.alloc(2 * rows * k)
+        allocs.append(d)
+        assert be.synth_fill(d, eb.BF16, rows * k, seed0 + len(allocs), k ** -0.5, 0)
+        assert sess.bind_matrix_at(layer, role, d, rows, k, k), (layer, role, sess.last_error)
+        if role != el.TOKEN_EMBD:
+            weight_bytes += 2 * rows * k
+
+    def vec(layer, role, n, rows=1):
+        assert sess.bind_vector_at(layer, role, ones, n, rows), (layer, role)
+
+    mat(-1, el.TOKEN_EMBD, sh["vocab"], W)
+    mat(-1, el.OUTPUT, sh["vocab"], W)
+    vec(-1, el.OUTPUT_NORM, W)
+    for i, l in enumerate(layers):
+        mat(i, ly.MIX_IN, ly.in_rows(l), W)
+        mat(i, el.ATTN_OUT, W, H * D)
+        vec(i, el.ATTN_NORM, W)
+        if l.mixer == ly.MIXER_LINEAR:
+            vec(i, ly.MIX_NORM_OUT, H * D)
+        else:
+            vec(i, ly.MIX_CONV, 3, ly.in_rows(l))
+            vec(i, ly.MIX_NORM_Q, H * D)
+            if l.kv_from < 0:
+                vec(i, ly.MIX_NORM_K, G * D)
+            talk = be.alloc(4 * H * H)
+            allocs.append(talk)
+            assert be.to_device(talk, (np.eye(H) + 0.1 * np.random.default_rng(i).standard_normal((H, H))).astype(np.float32))
+            assert sess.bind_vector_at(i, ly.MIX_HEADS, talk, H, H)
+        mat(i, ly.FFN_IN, 2 * ff, W)
+        vec(i, ly.FFN_IN_BIAS, 2 * ff)
+        mat(i, el.FFN_DOWN, W, ff)
+        vec(i, ly.FFN_DOWN_BIAS, W)
+        vec(i, el.FFN_NORM, W)
+    assert be.sync()
+    return sess, weight_bytes, allocs
+
+
+def run_metulix(args):
+    """--workload metulix: prompt and decode throughput of layered decoders at the sizes of METULIX_SHAPES, each beside a Llama
+    session of equal width, feed-forward, heads and layer count.  A step = one decoded token."""
+    import torch
+    import emel_cpp_b200 as eb
+
+    rank, world, local = dist_setup(args.gpus)
+    torch.cuda.set_device(local)
+    dev = torch.device("cuda", local)
+    be = eb.Backend(local)
+    stream = torch.cuda.ExternalStream(be.stream(), device=dev)
+    peaks, peak_kind = measured_peaks()
+    steps, warmup = args.steps, args.warmup
+    prompt_len = args.prompt or 2048
+
+    def timed(fn):
+        be.sync()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(stream)
+        out = fn()
+        e1.record(stream)
+        be.sync()
+        e1.synchronize()
+        return e0.elapsed_time(e1), out
+
+    def measure(sess, weight_bytes, vocab):
+        p = np.random.Generator(np.random.PCG64(42)).integers(0, vocab, size=prompt_len, dtype=np.int32)
+        for _ in range(warmup):
+            assert sess.prefill(p, 0), sess.last_error
+        times = [timed(lambda: sess.prefill(p, 0))[0] for _ in range(5)]
+        ids = sess.generate(1, prompt_len, warmup)
+        ms, ids = timed(lambda: sess.generate(int(ids[-1]), prompt_len + warmup, steps))
+        launches = sess.launches_per_token()
+        d0 = be.diagnostics()
+
+        def loop():
+            t = int(ids[-1])
+            for i in range(steps):
+                t = sess.decode(t, prompt_len + warmup + steps + i)
+        ms_e, _ = timed(loop)
+        d1 = be.diagnostics()
+        return {"prefill_tok_s": round(prompt_len / (float(np.median(times)) * 1e-3), 1), "decode_tok_s": round(steps / (ms * 1e-3), 2),
+                "decode_e2e_tok_s": round(steps / (ms_e * 1e-3), 2), "ms_per_token": round(ms / steps, 5), "launches_per_token": launches,
+                "weight_bytes_per_token": int(weight_bytes), "weight_gbs": round(weight_bytes / (ms / steps * 1e-3) / 1e9, 1),
+                "weight_frac_of_hbm": round(weight_bytes / (ms / steps * 1e-3) / 1e9 / peaks["hbm_gbs"], 3)}, \
+            (d1["d2h_bytes"] - d0["d2h_bytes"]) // steps
+
+    n_ctx = ((prompt_len + warmup + 2 * steps + 63) // 64) * 64
+    out, d2h = {}, 0
+    with ClockSampler(local) as clk:
+        for name in args.sizes.split(","):
+            sh = METULIX_SHAPES[name]
+            sess, wb, allocs = build_metulix_session(be, sh, n_ctx)
+            res, d2h = measure(sess, wb, sh["vocab"])
+            sess.close()
+            for d in allocs:
+                be.free(d)
+            lsh = dict(n_layer=sh["layers"], n_embd=sh["width"], n_head=sh["heads"], n_head_kv=sh["kv_heads"], head_dim=sh["dim"], n_ff=sh["ff"],
+                       n_vocab=sh["vocab"])
+            sess, info = build_decode_session(be, lsh, eb.Q4_K, n_ctx, 0, 1)
+            other, _ = measure(sess, info["weight_bytes"], sh["vocab"])
+            release_decode_session(be, sess, info, 1)
+            out[name] = {"metulix": res, "llama_q4_k": other}
+    clocks = clk.summary()
+    head = out[args.sizes.split(",")[0]]["metulix"]
+    print(json.dumps({
+        "metric": "decode tok/s", "value": head["decode_tok_s"], "unit": "tok/s", "n_gpus": world, "steps": steps, "warmup": warmup,
+        "ms_per_step": head["ms_per_token"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16 operands and KV, f32 accumulation, residual stream and state", "data": "synthetic",
+        "config": {"workload": "metulix layers beside Llama layers of equal size", "prompt_tokens": prompt_len, "sizes": args.sizes,
+                   "l2_policy": "inputs larger than L2: the weights of a token or prompt batch"},
+        "sizes": out, "e2e": {"value": head["decode_e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 8, "d2h_bytes_per_step": d2h},
+        "gpu_launches": head["launches_per_token"] * steps, "peak_source": f"of {peak_kind}", "clocks": clocks}), flush=True)
+
+
 def run_decode_batch(args):
     """--batch B > 1: B sequences decoded together (BASELINE configuration 5's batch-16 decode, or the 8B shape).
     Every sequence gets its own random prompt of the configured length; a step = one token for each sequence."""
@@ -1395,7 +1539,7 @@ def main():
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "decode_70b", "gemv_q4_k", "gemv_q8_0", "prefill_q4_k", "load_gguf"])
+    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "decode_70b", "gemv_q4_k", "gemv_q8_0", "prefill_q4_k", "load_gguf", "metulix"])
     ap.add_argument("--layers", type=int, default=16, help="load_gguf: layers in the synthetic file (122.7 MB each)")
     ap.add_argument("--prompt", type=int, default=None, help="prompt length override for the decode workloads")
     ap.add_argument("--ncols", type=int, default=1)
@@ -1415,6 +1559,7 @@ def main():
     ap.add_argument("--one-kernel", action="store_true",
                     help="decode workloads: run the headline through the one-kernel step (every layer of a token in one "
                          "persistent kernel) instead of the launch chain")
+    ap.add_argument("--sizes", default="2b,8b,8b-full", help="metulix: which of METULIX_SHAPES, with commas between them")
     ap.add_argument("--mix", action="store_true",
                     help="decode workloads: attn_v and ffn_down of every other layer as Q6_K instead of Q4_K")
     args = ap.parse_args()
@@ -1422,7 +1567,12 @@ def main():
     MIX_Q6_K = args.mix
     args.warmup = max(3, args.warmup)
     decode = args.workload.startswith("decode")
-    if args.workload == "prefill_q4_k":
+    if args.workload == "metulix":
+        if args.impl == "reference":
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no layered decoder of this design"}), flush=True)
+        else:
+            run_metulix(args)
+    elif args.workload == "prefill_q4_k":
         (run_reference_prefill if args.impl == "reference" else run_prefill)(args)
     elif args.workload == "load_gguf":
         (run_reference_load if args.impl == "reference" else run_load)(args)

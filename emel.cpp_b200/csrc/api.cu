@@ -1078,6 +1078,7 @@ uint32_t emelb_synth_fill(emelb_ctx* c, void* dev, int32_t type, uint64_t elems,
   cudaSetDevice(c->device);
   cudaError_t e;
   if (type == T_F32) e = launch_fill_normal(static_cast<float*>(dev), elems, seed, sigma, offset, c->stream);
+  else if (type == T_BF16) e = launch_fill_normal_bf16(dev, elems, seed, sigma, offset, c->stream);
   else if (is_native_quant(type) && elems % block_elems(type) == 0)
     e = launch_encode_normal(type, static_cast<uint8_t*>(dev), elems, seed, sigma, offset, c->stream);
   else return EMELB_INVALID_REQUEST;

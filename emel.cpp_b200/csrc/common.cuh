@@ -10,7 +10,7 @@
 namespace emelb {
 
 // dtype codes, src/emel/kernel/events.hpp:78-123
-enum : int { T_F32 = 0, T_F16 = 1, T_Q4_0 = 2, T_Q8_0 = 8, T_Q4_K = 12, T_Q6_K = 14, T_Q8_K = 15, T_I32 = 26 };
+enum : int { T_F32 = 0, T_F16 = 1, T_Q4_0 = 2, T_Q8_0 = 8, T_Q4_K = 12, T_Q6_K = 14, T_Q8_K = 15, T_I32 = 26, T_BF16 = 30 };
 
 constexpr int QK_K = 256;
 constexpr int QK32 = 32;

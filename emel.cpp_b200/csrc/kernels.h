@@ -293,6 +293,7 @@ cudaError_t launch_llama_token(const TokenArgs& a, int sm_count, TokenLaunchStat
 
 // synth.cu — synthetic N(0, sigma) data generated and block-encoded on the device
 cudaError_t launch_fill_normal(float* out, uint64_t n, uint64_t seed, float sigma, uint64_t offset, cudaStream_t st);
+cudaError_t launch_fill_normal_bf16(void* out, uint64_t n, uint64_t seed, float sigma, uint64_t offset, cudaStream_t st);
 cudaError_t launch_encode_normal(int type, uint8_t* out, uint64_t elems, uint64_t seed, float sigma, uint64_t offset,
                                  cudaStream_t st);
 

@@ -3,6 +3,7 @@
 // GGUF block formats (the reference has no K-quant encoder; any encoder that
 // emits valid blocks serves, since every consumer reads the same bytes).  Used
 // to fill benchmark-sized weight matrices (tens of GB) without a host pass.
+#include <cuda_bf16.h>
 #include "common.cuh"
 #include "kernels.h"
 
@@ -29,6 +30,11 @@ __device__ __forceinline__ float normal_at(uint64_t seed, uint64_t idx) {
 __global__ void fill_normal_kernel(float* out, uint64_t n, uint64_t seed, float sigma, uint64_t offset) {
   for (uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (uint64_t)gridDim.x * blockDim.x)
     out[i] = sigma * normal_at(seed, offset + i);
+}
+
+__global__ void fill_normal_bf16_kernel(__nv_bfloat16* out, uint64_t n, uint64_t seed, float sigma, uint64_t offset) {
+  for (uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (uint64_t)gridDim.x * blockDim.x)
+    out[i] = __float2bfloat16_rn(sigma * normal_at(seed, offset + i));
 }
 
 __device__ __forceinline__ uint16_t f2h_bits(float f) { return __half_as_ushort(__float2half_rn(f)); }
@@ -153,6 +159,13 @@ cudaError_t launch_fill_normal(float* out, uint64_t n, uint64_t seed, float sigm
   uint64_t blocks = (n + 255) / 256;
   if (blocks > 65535) blocks = 65535;
   fill_normal_kernel<<<(unsigned)blocks, 256, 0, st>>>(out, n, seed, sigma, offset);
+  return cudaGetLastError();
+}
+
+cudaError_t launch_fill_normal_bf16(void* out, uint64_t n, uint64_t seed, float sigma, uint64_t offset, cudaStream_t st) {
+  uint64_t blocks = (n + 255) / 256;
+  if (blocks > 65535) blocks = 65535;
+  fill_normal_bf16_kernel<<<(unsigned)blocks, 256, 0, st>>>(static_cast<__nv_bfloat16*>(out), n, seed, sigma, offset);
   return cudaGetLastError();
 }
 
