@@ -195,8 +195,9 @@ class Port(_Lib):
             return bool(self.f("can_run_mul_mat")(C.byref(op)))
         raise ValueError(code)
 
-    def mul_mat(self, op):
-        return bool(self.f("mul_mat")(C.byref(op)))
+    def mul_mat(self, op, route="scalar"):
+        """route "blocks": the x86 AVX2 route's f32 order, one value per block."""
+        return bool(self.f("mul_mat" if route == "scalar" else "mul_mat_blocks")(C.byref(op)))
 
     def mul_mat_argmax(self, op):
         return bool(self.f("mul_mat_argmax")(C.byref(op)))
@@ -344,7 +345,7 @@ class LConfig(C.Structure):
 class CpuLlama:
     """The reference generator's decode loop restated on the CPU.  `kernels` picks who does the
     matrix products and attention: "ref-avx2" / "ref-scalar" (the reference's own kernels from
-    oracle/_ref) or "port" (emel_oracle.c)."""
+    oracle/_ref), "port" (emel_oracle.c) or "port-blocks" (the same with the products in the AVX2 route's order)."""
 
     def __init__(self, cfg: dict, kernels: str = "port"):
         lib = port().lib
@@ -356,7 +357,7 @@ class CpuLlama:
         elif kernels == "ref-scalar":
             mm, fa = r.lib.ref_mul_mat_scalar, r.lib.ref_flash_attn_scalar
         else:
-            mm, fa = lib.orc_mul_mat, lib.orc_flash_attn
+            mm, fa = lib.orc_mul_mat_blocks if kernels == "port-blocks" else lib.orc_mul_mat, lib.orc_flash_attn
         self.cfg = LConfig(cfg["n_layer"], cfg["n_embd"], cfg["n_head"], cfg["n_head_kv"], cfg["head_dim"], cfg["n_ff"],
                            cfg["n_vocab"], cfg["n_ctx"], cfg.get("rope_dim", cfg["head_dim"]), cfg.get("rope_neox", 0),
                            cfg.get("kv_block", 16), cfg.get("rope_freq_base", 500000.0), cfg.get("rms_eps", 1e-5))

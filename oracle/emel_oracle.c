@@ -334,7 +334,46 @@ static float dot_q4_0_q8_0(const blk_q4_0* lhs, const blk_q8_0* rhs, uint64_t nb
   return sumf;
 }
 
+/* The x86 AVX2 route's f32 order (src/emel/kernel/x86_64/actions.hpp:859-866, 876-896): the block integers are exact in
+ * any order, and each block adds one value to the row sum.  The scalar order above spreads a block over eight lanes. */
+static _Thread_local int block_order = 0;
+
+static float block_dot_q4_k(const blk_q4_k* lhs, const blk_q8_k* rhs, uint64_t nblk) {
+  float sum = 0.0f;
+  for (uint64_t b = 0; b < nblk; ++b) {
+    uint8_t sc[8], mn[8];
+    for (int j = 0; j < 8; ++j) scale_min_k4(j, lhs[b].scales, &sc[j], &mn[j]);
+    int32_t isum = 0, msum = 0;
+    for (int j = 0; j < QK_K; ++j) {
+      const int sub = j / 32;
+      const uint8_t byte = lhs[b].qs[(sub / 2) * 32 + j % 32];
+      isum += (int32_t)sc[sub] * (int32_t)(sub % 2 ? byte >> 4 : byte & 0x0f) * (int32_t)rhs[b].qs[j];
+    }
+    for (int g = 0; g < 16; ++g) msum += (int32_t)rhs[b].bsums[g] * (int32_t)mn[g / 2];
+    const float d = orc_fp16_to_fp32(lhs[b].d) * rhs[b].d, dmin = orc_fp16_to_fp32(lhs[b].dmin) * rhs[b].d;
+    sum += fmaf(d, (float)isum, -(dmin * (float)msum));
+  }
+  return sum;
+}
+
+static float block_dot_q6_k(const blk_q6_k* lhs, const blk_q8_k* rhs, uint64_t nblk) {
+  float sum = 0.0f;
+  for (uint64_t b = 0; b < nblk; ++b) {
+    int32_t isum = 0;
+    for (int j = 0; j < QK_K; ++j) {
+      const int half = j / 128, quarter = j % 128 / 32, l = j % 32;
+      const uint8_t low = lhs[b].ql[64 * half + 32 * (quarter % 2) + l], high = lhs[b].qh[32 * half + l];
+      const int q = ((quarter < 2 ? low & 0x0f : low >> 4) | (((high >> (2 * quarter)) & 3) << 4)) - 32;
+      isum += (int32_t)lhs[b].scales[j / 16] * q * (int32_t)rhs[b].qs[j];
+    }
+    sum += orc_fp16_to_fp32(lhs[b].d) * rhs[b].d * (float)isum;
+  }
+  return sum;
+}
+
 float orc_row_dot(int type, const void* lhs, const void* rhs, uint64_t nblk) {
+  if (block_order && type == T_Q4_K) return block_dot_q4_k((const blk_q4_k*)lhs, (const blk_q8_k*)rhs, nblk);
+  if (block_order && type == T_Q6_K) return block_dot_q6_k((const blk_q6_k*)lhs, (const blk_q8_k*)rhs, nblk);
   switch (type) {
     case T_Q4_K: return dot_q4_k_q8_k((const blk_q4_k*)lhs, (const blk_q8_k*)rhs, nblk);
     case T_Q6_K: return dot_q6_k_q8_k((const blk_q6_k*)lhs, (const blk_q8_k*)rhs, nblk);
@@ -449,6 +488,13 @@ int orc_mul_mat(const o_op* r) {
     free(q8);
   }
   return 1;
+}
+
+int orc_mul_mat_blocks(const o_op* r) {
+  block_order = 1;
+  const int ok = orc_mul_mat(r);
+  block_order = 0;
+  return ok;
 }
 
 /* src/emel/kernel/detail.hpp:3573-3731: strict > over ascending rows, so the

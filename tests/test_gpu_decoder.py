@@ -29,7 +29,7 @@ def build_model(be, port, cfg, types, seed):
     """Encodes N(0, 0.02) weights on the host, uploads them, binds both decoders."""
     c = el.config(**cfg)
     sess = el.Session(be, c)
-    kernels = "ref-avx2" if ob.ref() is not None else "port"
+    kernels = "ref-avx2" if ob.ref() is not None else "port-blocks"
     cpu = ob.CpuLlama(cfg, kernels)
     shapes = el.matrix_shapes(c)
     tid = _NEXT_TENSOR_ID

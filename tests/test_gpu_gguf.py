@@ -59,7 +59,7 @@ def test_decode_from_gguf_file_matches_reference_loop(be, port, tmp_path, types)
     image, plan = model_file(port, 21, types)
     path = tmp_path / "tiny-llama.gguf"
     path.write_bytes(image)
-    kernels = "ref-avx2" if ob.ref() is not None else "port"
+    kernels = "ref-avx2" if ob.ref() is not None else "port-blocks"
     cpu = ob.CpuLlama(CFG, kernels)
     host = np.frombuffer(image, np.uint8)
     with gguf.File(str(path)) as f:

@@ -39,10 +39,9 @@ def gpu_mul_mat(be, t, w, k, m, x, n=1):
 
 
 def cpu_mul_mat(lib, t, w, k, m, x, n=1, **kw):
-    """The reference's x86 route (AVX2/FMA) where oracle/_ref is present, else the C port."""
+    """The reference's x86 route (AVX2/FMA) where oracle/_ref is present, else the C port in that route's order."""
     y = np.zeros((m, n), np.float32)
-    if isinstance(lib, ob.Ref):
-        kw.setdefault("route", "avx2")
+    kw.setdefault("route", "avx2" if isinstance(lib, ob.Ref) else "blocks")
     assert lib.mul_mat(ob.mul_mat_op(w, t, k, m, x, n, y), **kw)
     return y
 
