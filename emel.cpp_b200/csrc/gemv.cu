@@ -198,6 +198,11 @@ cudaError_t launch_type(GemvArgs a, int ncols, bool argmax, bool fast, int sm_co
 
 }  // namespace
 
+cudaError_t launch_argmax_finish(const float* part_val, const int* part_idx, int parts, float* out_val, int* out_idx, cudaStream_t st) {
+  argmax_finish_kernel<<<1, 256, 0, st>>>(part_val, part_idx, parts, out_val, out_idx);
+  return cudaGetLastError();
+}
+
 cudaError_t launch_argmax_f32(const float* x, int n, float* out_val, int* out_idx, cudaStream_t st) {
   argmax_f32_kernel<<<1, 1024, 0, st>>>(x, n, out_val, out_idx);
   return cudaGetLastError();

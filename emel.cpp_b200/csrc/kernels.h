@@ -134,6 +134,8 @@ cudaError_t launch_gemm_q4k_mma(const GemvArgs& a, int ncols, int sm_count, cuda
 cudaError_t launch_gemv_stream2(int type, const GemvArgs& a, int ncols, bool argmax, int sm_count, cudaStream_t st,
                                 int* launches, int* grid_out);
 
+// per-block candidates -> the highest value and, on ties, the lowest row
+cudaError_t launch_argmax_finish(const float* part_val, const int* part_idx, int parts, float* out_val, int* out_idx, cudaStream_t st);
 cudaError_t launch_argmax_f32(const float* x, int n, float* out_val, int* out_idx, cudaStream_t st);
 
 // quantize.cu — built with -fmad=false: every float op rounds as written

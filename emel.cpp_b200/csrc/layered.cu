@@ -71,6 +71,7 @@ struct Layered {
   void *xb = nullptr, *projb = nullptr, *q = nullptr, *mix = nullptr, *h = nullptr, *nb = nullptr;
   XMaps xb_x{}, nb_x{};
   // attention scratch
+  float* lin_local = nullptr;
   float *scores = nullptr, *stats = nullptr, *part = nullptr;
   uint64_t scores_floats = 0, stats_floats = 0, part_floats = 0;
   float* trace_out = nullptr;
@@ -161,9 +162,9 @@ MixAttnArgs mix_args(const Layered* m, const LayerS& l, const void* q) {
   return a;
 }
 
-LinAttnArgs lin_args(const LayerS& l, int64_t ldx, float* out) {
+LinAttnArgs lin_args(const Layered* m, const LayerS& l, int64_t ldx, float* out) {
   const emelb_layer_config& g = l.cfg;
-  return LinAttnArgs{ldx, g.n_head, g.key_dim, g.value_dim, l.decay, l.state, out};
+  return LinAttnArgs{ldx, g.n_head, g.key_dim, g.value_dim, l.decay, l.state, out, m->lin_local};
 }
 
 bool check(Layered* m, LayeredRun& r, cudaError_t e, int launches = 1) {
@@ -214,9 +215,9 @@ void rows_through_layers(Layered* m, LayeredRun& r, const int* tokens, const Row
       T* proj = static_cast<T*>(m->projb);
       linear(m, r, l.w.in, l.w.in_map, xb, ldx, m->xb_x, n, nullptr, ACT_SILU_SIGMOID, l.gate_at(), reinterpret_cast<float*>(m->projb),
              m->f32 ? nullptr : static_cast<bf16*>(m->projb), ldp);
-      const LinAttnArgs a = lin_args(l, ldp, m->lin);
+      const LinAttnArgs a = lin_args(m, l, ldp, m->lin);
       if (!m->f32 && rows.prompt && linear_attention_prompt_supported(a))
-        check(m, r, launch_linear_attention_prompt(a, reinterpret_cast<const bf16*>(proj), rows, r.st));
+        check(m, r, launch_linear_attention_prompt(a, reinterpret_cast<const bf16*>(proj), rows, m->c->sm_count, r.st, &r.launches), 0);
       else
         check(m, r, launch_linear_attention_rows<T>(a, proj, rows, r.st));
       check(m, r, launch_rms_gate<T>(m->lin, l.w.norm_out, proj + l.gate_at(), ldp, m->cfg.rms_eps, n, od, mix, ldo, r.st));
@@ -241,7 +242,7 @@ void rows_through_layers(Layered* m, LayeredRun& r, const int* tokens, const Row
 
 // the fused one-token chain; T = type of the key / value cache
 template <class T>
-void step_through_layers(Layered* m, LayeredRun& r, int seq, const int* state, float* logits) {
+void step_through_layers(Layered* m, LayeredRun& r, int seq, const int* state, float* logits, int* argmax_parts) {
   const int sms = m->c->sm_count;
   const bool pdl = (m->c->pdl & 1) != 0;
   const Rows rows{1, false, seq, state + 1};
@@ -250,7 +251,7 @@ void step_through_layers(Layered* m, LayeredRun& r, int seq, const int* state, f
   auto vec = [&](const Bf16Matrix& w, const float* bias, int act, int split, VecArgs v, float* out) {
     v.eps = m->cfg.rms_eps;
     v.out = out;
-    check(m, r, launch_linear_vec(LinearArgs{w, bias, act, split, 1}, v, sms, pdl, r.st));
+    check(m, r, launch_linear_vec(LinearArgs{w, bias, act, split, 1}, v, sms, pdl, r.st, v.part_val ? argmax_parts : nullptr));
   };
   // a product of the residual stream: the norm and sum of the sublayer before it run in its prologue
   auto stream = [&](const Bf16Matrix& w, const float* bias, int act, int split, float* out) {
@@ -283,7 +284,7 @@ void step_through_layers(Layered* m, LayeredRun& r, int seq, const int* state, f
       check(m, r, (launch_mix_attention_rows<T, float>(mix_args(m, l, m->vq), rows, m->vmix, l.out_dim(), sms, r.st, &r.launches)), 0);
     } else {
       stream(l.w.in, nullptr, ACT_SILU_SIGMOID, l.gate_at(), m->vproj);
-      check(m, r, launch_linear_attention_rows<float>(lin_args(l, 0, m->vmix), m->vproj, rows, r.st));
+      check(m, r, launch_linear_attention_rows<float>(lin_args(m, l, 0, m->vmix), m->vproj, rows, r.st));
       out.pro = PRO_RMS_GATE;
       out.norm_w = l.w.norm_out;
       out.gate = m->vproj + l.gate_at();
@@ -306,6 +307,10 @@ void step_through_layers(Layered* m, LayeredRun& r, int seq, const int* state, f
   v.y = m->vy;
   v.norm_w = pending;
   v.norm2_w = m->final_norm;
+  if (argmax_parts) {
+    v.part_val = m->c->part_val;
+    v.part_idx = m->c->part_idx;
+  }
   vec(m->head, nullptr, ACT_NONE, 0, v, logits);
 }
 
@@ -352,7 +357,7 @@ Layered* layered_create(emelb_ctx* c, const emelb_llama_config& cfg, const emelb
   bool ok = true;
   std::map<std::pair<int, float>, std::pair<const float*, const float*>> tables;
   int max_in = 0, max_out = 0, max_ff = 0, max_q = 0;
-  uint64_t scores = 0, stats = 0, part = 0;
+  uint64_t scores = 0, stats = 0, part = 0, lin_state = 0;
   for (int i = 0; i < cfg.n_layer; ++i) {
     LayerS& l = m->layers[i];
     l.cfg = layers[i];
@@ -363,6 +368,7 @@ Layered* layered_create(emelb_ctx* c, const emelb_llama_config& cfg, const emelb
     max_out = std::max(max_out, l.out_dim());
     max_ff = std::max(max_ff, l.cfg.n_ff);
     if (!l.attention()) {
+      lin_state = std::max<uint64_t>(lin_state, (uint64_t)l.cfg.n_head * l.cfg.key_dim * l.cfg.value_dim);
       ok = ok && alloc_n(m->owned, &l.decay, l.cfg.n_head);
       ok = ok && ctx_cuda_ok(c, cudaMemcpy(l.decay, layers[i].decay, 4 * (size_t)l.cfg.n_head, cudaMemcpyHostToDevice));
       continue;
@@ -398,10 +404,12 @@ Layered* layered_create(emelb_ctx* c, const emelb_llama_config& cfg, const emelb
   for (int i = 0; i < 2; ++i) ok = ok && alloc_n(m->owned, &m->vx[i], cfg.n_embd);
   ok = ok && alloc_n(m->owned, &m->vy, cfg.n_embd) && alloc_n(m->owned, &m->vproj, max_in) && alloc_n(m->owned, &m->vmix, max_out);
   if (max_ff > 0) ok = ok && alloc_n(m->owned, &m->vh, max_ff);
+  if (lin_state > 0 && !f32) ok = ok && alloc_n(m->owned, &m->lin_local, kLinAttnMaxSegments * lin_state);
   if (scores > 0) {
     ok = ok && alloc(m->owned, &m->vq, 4 * (size_t)max_q);
     m->scores_floats = std::max<uint64_t>(scores, 16u << 20);
-    m->stats_floats = std::max<uint64_t>(stats, 1u << 20);
+    // prompts keep one {max, sum} pair per 64 columns of a strip's scores
+    m->stats_floats = std::max<uint64_t>(stats, m->scores_floats / 32);
     m->part_floats = std::max<uint64_t>(part, 4u << 20);
     ok = ok && alloc_n(m->owned, &m->scores, m->scores_floats) && alloc_n(m->owned, &m->stats, m->stats_floats) &&
          alloc_n(m->owned, &m->part, m->part_floats);
@@ -542,6 +550,13 @@ uint32_t layered_bind(Layered* m, int layer, int role, const emelb_view* t) {
   if (!dev) return EMELB_INVALID_REQUEST;
   if (vec) {
     if (t->type != EMELB_F32 || t->nb[0] != 4 || (M > 1 && (int64_t)t->nb[1] != 4 * K)) return EMELB_INVALID_REQUEST;
+    if (role == EMELB_T_MIX_CONV) {
+      // kept tap by tap, so that neighbouring channels are read together
+      float* taps = const_cast<float*>(l->w.conv);
+      if (!taps && !alloc_n(m->owned, &taps, (size_t)(K * M))) return EMELB_INTERNAL_ERROR;
+      if (!ctx_cuda_ok(m->c, launch_transpose(static_cast<const float*>(dev), (int)M, (int)K, taps, m->c->stream))) return EMELB_INTERNAL_ERROR;
+      dev = taps;
+    }
     *vec = static_cast<const float*>(dev);
     return EMELB_OK;
   }
@@ -572,9 +587,9 @@ bool layered_bound(const Layered* m) {
   return ok;
 }
 
-void layered_step(Layered* m, LayeredRun& r, int seq, const int* state, float* logits) {
-  if (m->f32) step_through_layers<float>(m, r, seq, state, logits);
-  else step_through_layers<bf16>(m, r, seq, state, logits);
+void layered_step(Layered* m, LayeredRun& r, int seq, const int* state, float* logits, int* argmax_parts) {
+  if (m->f32) step_through_layers<float>(m, r, seq, state, logits, argmax_parts);
+  else step_through_layers<bf16>(m, r, seq, state, logits, argmax_parts);
 }
 
 void layered_rows(Layered* m, LayeredRun& r, const int* tokens, const Rows& rows, int pos0) {

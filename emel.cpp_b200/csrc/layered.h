@@ -57,8 +57,11 @@ struct VecArgs {
   int64_t table_ld;
   const int* token;
   float* out;
+  float* part_val;         // optional: each block's highest output and the lowest row that has it (kMaxArgmaxParts)
+  int* part_idx;
 };
-cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_count, bool pdl, cudaStream_t st);
+// parts (optional): blocks launched
+cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_count, bool pdl, cudaStream_t st, int* parts = nullptr);
 // f32 operands on the CUDA cores
 cudaError_t launch_linear_f32(const LinearArgs& a, const float* x, int64_t ldx, float* y, int64_t ldy, cudaStream_t st);
 
@@ -92,9 +95,9 @@ cudaError_t launch_glu_rows(const float* gu, int rows, int ff, float* out, int64
 struct AttnInArgs {
   const float* proj;       // {rows, channels}: q | k | v, or q alone
   int channels;
-  const float* conv;       // [channels][taps]; null: no convolution
+  const float* conv;       // [taps][channels]; null: no convolution
   int taps;
-  float* conv_state;       // [sequence][channels][taps - 1]
+  float* conv_state;       // [sequence][taps - 1][channels]
   const float *norm_q, *norm_k;   // null: no norm
   int norm_v;
   float eps;
@@ -144,11 +147,14 @@ struct LinAttnArgs {
   const float* decay;      // device, [heads]
   float* state;            // [sequence][heads][dim][vdim]
   float* out;              // {rows, heads * vdim}
+  float* local;            // scratch of kLinAttnMaxSegments states (null: prompts run as one segment)
 };
+constexpr int kLinAttnMaxSegments = 8;
 template <class T>
 cudaError_t launch_linear_attention_rows(const LinAttnArgs& a, const T* x, const Rows& rows, cudaStream_t st);
 bool linear_attention_prompt_supported(const LinAttnArgs& a);
-cudaError_t launch_linear_attention_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, cudaStream_t st);
+cudaError_t launch_linear_attention_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, int sm_count, cudaStream_t st,
+                                           int* launches);
 
 // ---- layered.cu: the model object
 struct Layered;
@@ -167,7 +173,8 @@ bool layered_reserve_rows(Layered* m, int rows);
 int layered_row_capacity(const Layered* m);
 void layered_set_trace(Layered* m, float* out, int max_tokens);
 // one token of sequence seq; state = {token, position, ...} on the device; logits null: none
-void layered_step(Layered* m, LayeredRun& r, int seq, const int* state, float* logits);
+// argmax_parts (optional): with logits, the context's argmax candidates are written too; their count
+void layered_step(Layered* m, LayeredRun& r, int seq, const int* state, float* logits, int* argmax_parts = nullptr);
 // rows through every layer; pos0: host copy of the first position (prompts)
 void layered_rows(Layered* m, LayeredRun& r, const int* tokens, const Rows& rows, int pos0);
 // final norm and output product of the given rows of the last layered_rows call (index null: all), {n, n_vocab}

@@ -65,6 +65,8 @@ __global__ void __launch_bounds__(kCols * kGroups) linear_attention_rows_kernel(
 //   S'   = decay^n S + sum_j decay^(n-1-j) k_j v_j^T
 // q, k and v are bf16; every f32 factor that meets them (the state, the decayed scores, the decayed values) is fed as
 // two bf16 operands, high part and remainder, so the recurrence keeps f32 accuracy.
+// Long prompts are cut into segments of whole chunks that run side by side: a first launch (STATES) leaves what each
+// segment but the last adds to the state in `local`, the second starts every segment from the sum of those before it.
 // One block = one head x kVS value columns, four warps: 16 query rows each for the outputs, every fourth 16-row tile of
 // the state, which lives in accumulator fragments between the chunks.
 constexpr int kChunk = 64, kVS = 32, kMmaThreads = 128;
@@ -77,8 +79,11 @@ struct ChunkSmem {
   float pw[kChunk + 1];
 };
 
-template <int D>
-__global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(const LinAttnArgs a, const __nv_bfloat16* __restrict__ x, const Rows rows) {
+// local: [segment][head][D][vdim]; with several segments its last entry holds the state the prompt starts from, since
+// the sequence's own is overwritten while other segments may not have started
+template <int D, bool STATES>
+__global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(const LinAttnArgs a, const __nv_bfloat16* __restrict__ x, const Rows rows,
+                                                                              const int segment, const int segments) {
   extern __shared__ __align__(16) unsigned char raw[];
   using Smem = ChunkSmem<D>;
   Smem& sm = *reinterpret_cast<Smem*>(raw);
@@ -87,29 +92,32 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
   const int h = blockIdx.x, v0 = blockIdx.y * kVS;
   const float decay = a.decay[h];
   float* state = a.state + ((int64_t)rows.seq0 * a.heads + h) * D * a.vdim;
+  auto local = [&](int seg) { return a.local + ((int64_t)seg * a.heads + h) * D * a.vdim; };
+  const int seg = blockIdx.z, row_begin = seg * segment, row_end = min(rows.n, row_begin + segment);
   const __nv_bfloat16 *xq = x + h * D, *xk = x + (a.heads + h) * D, *xv = x + 2 * a.heads * D + h * a.vdim + v0;
 
   auto issue = [&](int c0, int buf) {
     for (int i = tid; i < kChunk * (D / 8); i += kMmaThreads) {
       const int r = i / (D / 8), c = i % (D / 8) * 8;
-      const bool live = c0 + r < rows.n;
+      const bool live = c0 + r < row_end;
       const int64_t at = (int64_t)(live ? c0 + r : 0) * a.ldx + c;
-      cp16_zfill(&sm.q[buf][r][c], xq + at, live);
+      if (!STATES) cp16_zfill(&sm.q[buf][r][c], xq + at, live);
       cp16_zfill(&sm.k[buf][r][c], xk + at, live);
     }
     for (int i = tid; i < kChunk * (kVS / 8); i += kMmaThreads) {
       const int r = i / (kVS / 8), c = i % (kVS / 8) * 8;
-      const bool live = c0 + r < rows.n && v0 + c < a.vdim;
+      const bool live = c0 + r < row_end && v0 + c < a.vdim;
       cp16_zfill(&sm.v[buf][r][c], live ? xv + (int64_t)(c0 + r) * a.ldx + c : xq, live);
     }
     asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
-  issue(0, 0);
+  issue(row_begin, 0);
   for (int i = tid; i <= kChunk; i += kMmaThreads) sm.pw[i] = powf(decay, (float)i);
 
   // state rows 16 (warp + 4 mt) + g (+8), columns 8 nt + 2t (+1)
   float S[MT][NT][4];
   const bool carried = rows.pos[0] > 0;
+  const float across = powf(decay, (float)segment);   // one whole segment's decay
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -117,7 +125,25 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = 16 * (warp + 4 * mt) + g + 8 * (e >> 1), c = 8 * nt + 2 * t + (e & 1);
-        S[mt][nt][e] = carried && r < D && v0 + c < a.vdim ? state[(int64_t)r * a.vdim + v0 + c] : 0.0f;
+        const bool mine = r < D && v0 + c < a.vdim;
+        const int64_t at = (int64_t)r * a.vdim + v0 + c;
+        float v = 0.0f;
+        if (STATES) {
+          if (mine && seg == 0) {
+            v = carried ? state[at] : 0.0f;
+            local(segments - 1)[at] = v;
+          }
+        } else if (mine) {
+          if (seg > 0) {
+            v = local(0)[at];   // the first segment's includes the state the prompt starts from
+            for (int p = 1; p < seg; ++p) v = fmaf(across, v, local(p)[at]);
+          } else if (segments > 1) {
+            v = local(segments - 1)[at];
+          } else if (carried) {
+            v = state[at];
+          }
+        }
+        S[mt][nt][e] = v;
       }
   auto publish = [&]() {
 #pragma unroll
@@ -135,12 +161,12 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
         }
     }
   };
-  publish();
+  if (!STATES) publish();
 
   int buf = 0;
-  for (int c0 = 0; c0 < rows.n; c0 += kChunk, buf ^= 1) {
-    const int n = min(kChunk, rows.n - c0);
-    if (c0 + kChunk < rows.n) {
+  for (int c0 = row_begin; c0 < row_end; c0 += kChunk, buf ^= 1) {
+    const int n = min(kChunk, row_end - c0);
+    if (c0 + kChunk < row_end) {
       issue(c0 + kChunk, buf ^ 1);
       asm volatile("cp.async.wait_group 1;\n" ::: "memory");
     } else {
@@ -148,7 +174,7 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
     }
     __syncthreads();
     const int r0 = 16 * warp;   // this warp's query rows
-    if (r0 < n) {
+    if (!STATES && r0 < n) {
       float s[kChunk / 8][4] = {}, o[NT][4] = {};
       const int ktiles = warp + 1;   // keys up to this warp's last row, 16 at a time
 #pragma unroll
@@ -208,7 +234,7 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int i = c0 + r0 + g + 8 * half;
-        if (i >= rows.n) continue;
+        if (i >= row_end) continue;
         float* out = a.out + ((int64_t)i * a.heads + h) * a.vdim + v0;
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
@@ -255,8 +281,10 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
       }
     }
     __syncthreads();   // every warp is done with this chunk and with the old state
-    publish();
+    if (!STATES) publish();
   }
+  if (!STATES && seg != segments - 1) return;
+  float* dst = STATES ? local(seg) : state;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -264,16 +292,30 @@ __global__ void __launch_bounds__(kMmaThreads) linear_attention_prompt_kernel(co
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = 16 * (warp + 4 * mt) + g + 8 * (e >> 1), c = 8 * nt + 2 * t + (e & 1);
-        if (r < D && v0 + c < a.vdim) state[(int64_t)r * a.vdim + v0 + c] = S[mt][nt][e];
+        if (r < D && v0 + c < a.vdim) dst[(int64_t)r * a.vdim + v0 + c] = S[mt][nt][e];
       }
 }
 
 template <int D>
-cudaError_t launch_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, cudaStream_t st) {
+cudaError_t launch_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, int sm_count, cudaStream_t st, int* launches) {
   const int smem = (int)sizeof(ChunkSmem<D>);
-  const cudaError_t e = cudaFuncSetAttribute(linear_attention_prompt_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  cudaError_t e = cudaFuncSetAttribute(linear_attention_prompt_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_attention_prompt_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return e;
-  linear_attention_prompt_kernel<D><<<dim3(a.heads, (a.vdim + kVS - 1) / kVS), kMmaThreads, smem, st>>>(a, x, rows);
+  const int tiles = (a.vdim + kVS - 1) / kVS;
+  // segments of at least 256 tokens while two blocks per SM have room for them
+  int segments = 2 * sm_count / (a.heads * tiles);
+  if (segments > kLinAttnMaxSegments) segments = kLinAttnMaxSegments;
+  if (segments > rows.n / 256) segments = rows.n / 256;
+  if (segments < 2 || !a.local) segments = 1;
+  const int chunks = (rows.n + kChunk - 1) / kChunk, segment = (chunks + segments - 1) / segments * kChunk;
+  segments = (rows.n + segment - 1) / segment;
+  if (segments > 1) {
+    linear_attention_prompt_kernel<D, true><<<dim3(a.heads, tiles, segments - 1), kMmaThreads, smem, st>>>(a, x, rows, segment, segments);
+    *launches += 1;
+  }
+  linear_attention_prompt_kernel<D, false><<<dim3(a.heads, tiles, segments), kMmaThreads, smem, st>>>(a, x, rows, segment, segments);
+  *launches += 1;
   return cudaGetLastError();
 }
 
@@ -283,16 +325,17 @@ bool linear_attention_prompt_supported(const LinAttnArgs& a) {
   return a.dim % 16 == 0 && a.dim <= 128 && a.vdim % 8 == 0 && a.ldx % 8 == 0;
 }
 
-cudaError_t launch_linear_attention_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, cudaStream_t st) {
+cudaError_t launch_linear_attention_prompt(const LinAttnArgs& a, const __nv_bfloat16* x, const Rows& rows, int sm_count, cudaStream_t st,
+                                           int* launches) {
   switch (a.dim / 16) {
-    case 1: return launch_prompt<16>(a, x, rows, st);
-    case 2: return launch_prompt<32>(a, x, rows, st);
-    case 3: return launch_prompt<48>(a, x, rows, st);
-    case 4: return launch_prompt<64>(a, x, rows, st);
-    case 5: return launch_prompt<80>(a, x, rows, st);
-    case 6: return launch_prompt<96>(a, x, rows, st);
-    case 7: return launch_prompt<112>(a, x, rows, st);
-    case 8: return launch_prompt<128>(a, x, rows, st);
+    case 1: return launch_prompt<16>(a, x, rows, sm_count, st, launches);
+    case 2: return launch_prompt<32>(a, x, rows, sm_count, st, launches);
+    case 3: return launch_prompt<48>(a, x, rows, sm_count, st, launches);
+    case 4: return launch_prompt<64>(a, x, rows, sm_count, st, launches);
+    case 5: return launch_prompt<80>(a, x, rows, sm_count, st, launches);
+    case 6: return launch_prompt<96>(a, x, rows, sm_count, st, launches);
+    case 7: return launch_prompt<112>(a, x, rows, sm_count, st, launches);
+    case 8: return launch_prompt<128>(a, x, rows, sm_count, st, launches);
     default: return cudaErrorInvalidValue;
   }
 }

@@ -127,6 +127,8 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
   }
   __syncthreads();
 
+  float best = 0.0f;
+  int best_row = -1;
   for (; task < tasks; task += stride) {
     float acc[RW];
 #pragma unroll
@@ -173,9 +175,40 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
           if (a.bias) y += a.bias[row];
           if (a.act == ACT_SILU_SIGMOID) y = row < a.act_split ? siluf_(y) : sigmoidf_(y);
           v.out[row] = y;
+          if (best_row < 0 || y > best) {   // rows of a lane ascend
+            best = y;
+            best_row = row;
+          }
         }
       }
     }
+  }
+  if (!v.part_val) return;
+  __shared__ float bv[kVecWarps];
+  __shared__ int bi[kVecWarps];
+  auto better = [](float x, int i, float y, int j) { return i >= 0 && (j < 0 || x > y || (x == y && i < j)); };
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float x = __shfl_xor_sync(0xffffffffu, best, o);
+    const int i = __shfl_xor_sync(0xffffffffu, best_row, o);
+    if (better(x, i, best, best_row)) {
+      best = x;
+      best_row = i;
+    }
+  }
+  if (lane == 0) {
+    bv[warp] = best;
+    bi[warp] = best_row;
+  }
+  __syncthreads();
+  if (tid == 0) {
+    for (int w = 1; w < kVecWarps; ++w)
+      if (better(bv[w], bi[w], best, best_row)) {
+        best = bv[w];
+        best_row = bi[w];
+      }
+    v.part_val[blockIdx.x] = best_row >= 0 ? best : -INFINITY;
+    v.part_idx[blockIdx.x] = best_row >= 0 ? best_row : 0x7fffffff;
   }
 }
 
@@ -224,7 +257,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearArgs a, con
 
 }  // namespace
 
-cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_count, bool pdl, cudaStream_t st) {
+cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_count, bool pdl, cudaStream_t st, int* parts) {
   const int chunks = (a.w.K + 7) / 8, smem = 32 * chunks;
   if (smem > 200 * 1024) return cudaErrorInvalidValue;
   const bool glu = a.act == ACT_GLU;
@@ -241,6 +274,7 @@ cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_coun
   per_sm = per_sm > 4 ? 4 : per_sm;
   int grid = (tasks + kVecWarps - 1) / kVecWarps;
   if (grid > sm_count * per_sm) grid = sm_count * per_sm;
+  if (parts) *parts = grid;
   return launch_kernel(kern, dim3(grid), dim3(kVecThreads), (size_t)smem, st, pdl, a, v);
 }
 

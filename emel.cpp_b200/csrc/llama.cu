@@ -827,13 +827,14 @@ struct Enqueue {
   // a layered session's step: the same modes, state words and follow-ups
   void layered_token_step(Mode mode) {
     LayeredRun run{st};
-    layered_step(s->layered, run, s->cur_seq, s->state, mode == MODE_PREFILL ? nullptr : s->logits);
+    int parts = 0;
+    layered_step(s->layered, run, s->cur_seq, s->state, mode == MODE_PREFILL ? nullptr : s->logits, mode == MODE_ARGMAX ? &parts : nullptr);
     launches += run.launches;
     ok = ok && run.ok;
     if (mode != MODE_ARGMAX || !ok) return;
-    check(launch_argmax_columns(s->logits, s->cfg.n_vocab, 1, s->c->part_val, s->c->part_idx, s->c->best_idx, st));
+    check(launch_argmax_finish(s->c->part_val, s->c->part_idx, parts, s->c->best_val, s->c->best_idx, st));
     check(launch_step_advance(s->state, s->c->best_idx, s->tokens_dev, st));
-    launches += 3;
+    launches += 2;
   }
 
   void token_step(Mode mode) {

@@ -301,9 +301,11 @@ template cudaError_t launch_mix_attention_rows<__nv_bfloat16, __nv_bfloat16>(con
 
 // ---- prompts on the tensor cores (mma.sync bf16).  A strip of consecutive query rows at a time, so that the scores of
 // every head stay in the L2 cache between three launches:
-//   scores   q . k * scale of 64 rows x 64 key columns, all heads of a key/value head per block
-//   mix      per row: softmax of every head over its visible columns, heads mixed in f32; each weight is left as two
-//            bf16 parts (high, remainder) in the place of its score, invisible columns as zero
+//   scores   q . k * scale of 64 rows x 64 key columns of one head, and the {max, sum of exponentials} of each row's
+//            visible columns in the tile
+//   mix      per row: softmax of every head over its visible columns, then talk x weights on the tensor cores, both
+//            fed as two bf16 parts (high, remainder); each mixed weight is left in two such parts in the place of its
+//            score, invisible columns as zero
 //   values   weights x value rows, both parts
 // Column c of a strip is key c for c < kk (kept tokens below the strip's first window), else key lo + c - kk.
 namespace {
@@ -329,140 +331,197 @@ __device__ __forceinline__ bool tile_visible(const Strip& s, int i0, int c0, int
   return k0 < keep || window <= 0 || p0 - k1 < window;
 }
 
+// the visible columns of a strip's row i: [0, kept) and [w0, w1]
+struct RowSpan {
+  int kept, w0, w1;
+  __device__ __forceinline__ bool sees(int c) const { return c < kept || (c >= w0 && c <= w1); }
+};
+__device__ __forceinline__ RowSpan row_span(const Strip& s, int i, int window, int keep) {
+  const int pos = s.pos0 + i, lo = window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
+  return RowSpan{min(keep, lo), s.kk + lo - s.lo, s.kk + pos - s.lo};
+}
+
 __global__ void __launch_bounds__(kMmaThreads) mix_prompt_scores_kernel(const MixAttnArgs a, const int seq, const Strip s) {
   extern __shared__ __align__(16) unsigned char raw[];
   const int D = a.dim_pad, row_halves = D + 8;
   __nv_bfloat16* qt = reinterpret_cast<__nv_bfloat16*>(raw);      // [64][D + 8]
   __nv_bfloat16* kt = qt + kQT * row_halves;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-  const int c0 = blockIdx.x * kCT, i0 = blockIdx.y * kQT, kh = blockIdx.z, n_rep = a.heads / a.kv_heads;
+  const int c0 = blockIdx.x * kCT, i0 = blockIdx.y * kQT, h = blockIdx.z, kh = h / (a.heads / a.kv_heads);
   if (!tile_visible(s, i0, c0, a.window, a.keep_first)) return;
   const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
   const __nv_bfloat16* k = static_cast<const __nv_bfloat16*>(a.k) + ((int64_t)seq * a.kv_heads + kh) * a.capacity * D;
-  const int chunks = D / 8;
-  for (int i = tid; i < kCT * chunks; i += kMmaThreads) {
-    const int r = i / chunks, c = i % chunks * 8;
-    const bool live = c0 + r < s.cols;
-    cp16_zfill(kt + r * row_halves + c, k + (live ? (int64_t)strip_key(s, c0 + r) * D + c : 0), live);
+  // two threads per row
+  for (int c = (tid & 1) * 8; c < D; c += 16) {
+    const int r = tid >> 1;
+    const bool kl = c0 + r < s.cols, ql = i0 + r < s.rows;
+    cp16_zfill(kt + r * row_halves + c, k + (kl ? (int64_t)strip_key(s, c0 + r) * D + c : 0), kl);
+    cp16_zfill(qt + r * row_halves + c, q + (ql ? ((int64_t)(s.row0 + i0 + r) * a.heads + h) * D + c : 0), ql);
   }
-  for (int rep = 0; rep < n_rep; ++rep) {
-    const int h = kh * n_rep + rep;
-    for (int i = tid; i < kQT * chunks; i += kMmaThreads) {
-      const int r = i / chunks, c = i % chunks * 8;
-      const bool live = i0 + r < s.rows;
-      cp16_zfill(qt + r * row_halves + c, q + (live ? ((int64_t)(s.row0 + i0 + r) * a.heads + h) * D + c : 0), live);
-    }
-    asm volatile("cp.async.commit_group;\n" ::: "memory");
-    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-    __syncthreads();
-    float acc[kCT / 8][4] = {};
-    for (int kk = 0; kk < D / 16; ++kk) {
-      uint32_t qa[4];
-      ldsm(qa, qt + (16 * warp + (lane & 15)) * row_halves + 16 * kk + (lane >> 4) * 8);
+  asm volatile("cp.async.commit_group;\n" ::: "memory");
+  asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+  __syncthreads();
+  float acc[kCT / 8][4] = {};
+  for (int kk = 0; kk < D / 16; ++kk) {
+    uint32_t qa[4];
+    ldsm(qa, qt + (16 * warp + (lane & 15)) * row_halves + 16 * kk + (lane >> 4) * 8);
 #pragma unroll
-      for (int nt = 0; nt < kCT / 16; ++nt) {
-        uint32_t b[4];
-        ldsm(b, kt + (16 * nt + (lane & 7) + (lane >> 4) * 8) * row_halves + 16 * kk + ((lane >> 3) & 1) * 8);
-        mma_bf16_16816(acc[2 * nt], qa, b[0], b[1]);
-        mma_bf16_16816(acc[2 * nt + 1], qa, b[2], b[3]);
+    for (int nt = 0; nt < kCT / 16; ++nt) {
+      uint32_t b[4];
+      ldsm(b, kt + (16 * nt + (lane & 7) + (lane >> 4) * 8) * row_halves + 16 * kk + ((lane >> 3) & 1) * 8);
+      mma_bf16_16816(acc[2 * nt], qa, b[0], b[1]);
+      mma_bf16_16816(acc[2 * nt + 1], qa, b[2], b[3]);
+    }
+  }
+  // every row of the tile sees every column: the last row's window starts at or before it, the first row's ends after it
+  const bool inside = row_span(s, min(i0 + kQT, s.rows) - 1, a.window, a.keep_first).w0 <= c0 && row_span(s, i0, a.window, a.keep_first).w1 >= c0 + kCT - 1;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int i = i0 + 16 * warp + g + 8 * half;
+    const RowSpan span = row_span(s, i, a.window, a.keep_first);
+    float* out = a.scores + ((int64_t)i * a.heads + h) * s.cols_pad + c0;
+    float m = -INFINITY, sum = 0.0f;
+#pragma unroll
+    for (int nt = 0; nt < kCT / 8; ++nt) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        float& v = acc[nt][2 * half + e];
+        v *= a.scale;
       }
-    }
+      if (i < s.rows) *reinterpret_cast<float2*>(out + 8 * nt + 2 * t) = make_float2(acc[nt][2 * half], acc[nt][2 * half + 1]);
+      if (!inside) {
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int i = i0 + 16 * warp + g + 8 * half;
-      if (i >= s.rows) continue;
-      float* out = a.scores + ((int64_t)i * a.heads + h) * s.cols_pad + c0;
-#pragma unroll
-      for (int nt = 0; nt < kCT / 8; ++nt)
-        *reinterpret_cast<float2*>(out + 8 * nt + 2 * t) = make_float2(acc[nt][2 * half] * a.scale, acc[nt][2 * half + 1] * a.scale);
+        for (int e = 0; e < 2; ++e)
+          if (!span.sees(c0 + 8 * nt + 2 * t + e)) acc[nt][2 * half + e] = -INFINITY;
+      }
+      m = fmaxf(m, fmaxf(acc[nt][2 * half], acc[nt][2 * half + 1]));
     }
-    __syncthreads();   // the query tile is replaced
+    m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));   // the four lanes of a row
+    m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
+    const float base = m == -INFINITY ? 0.0f : m;
+#pragma unroll
+    for (int nt = 0; nt < kCT / 8; ++nt)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) sum += __expf(acc[nt][2 * half + e] - base);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+    if (t == 0 && i < s.rows) reinterpret_cast<float2*>(a.stats)[((int64_t)i * a.heads + h) * (s.cols_pad / kCT) + blockIdx.x] = make_float2(m, sum);
   }
 }
 
 constexpr int kMixThreads = 256;
 
-// one block per row; HM >= heads
+// one block per row; heads padded to HM, a multiple of 16
 template <int HM>
 __global__ void __launch_bounds__(kMixThreads) mix_prompt_weights_kernel(const MixAttnArgs a, const Strip s) {
-  __shared__ __align__(16) float talk[HM * HM];
+  constexpr int kRow = HM + 8, MT = HM / 16;
+  __shared__ __align__(16) __nv_bfloat16 talk_hi[HM][kRow], talk_lo[HM][kRow];
   __shared__ float mx[HM], inv[HM];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, H = a.heads;
-  const int i = blockIdx.x, pos = s.pos0 + i;
-  const int lo = a.window > 0 && pos - a.window + 1 > 0 ? pos - a.window + 1 : 0;
-  const int kept = min(a.keep_first, lo);                 // columns [0, kept) and [w0, w1]
-  const int w0 = s.kk + lo - s.lo, w1 = s.kk + pos - s.lo, n = kept + w1 - w0 + 1;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, H = a.heads;
+  const int i = blockIdx.x, tiles = s.cols_pad / kCT, q_tile = i / kQT * kQT;
+  const RowSpan span = row_span(s, i, a.window, a.keep_first);
   float* sc = a.scores + (int64_t)i * H * s.cols_pad;
   for (int x = tid; x < HM * HM; x += kMixThreads) {
-    const int h = x / HM, g = x % HM;
-    talk[x] = h < H && g < H ? (a.talk ? a.talk[h * H + g] : (h == g ? 1.0f : 0.0f)) : 0.0f;
+    const int h = x / HM, k = x % HM;
+    const float v = h < H && k < H ? (a.talk ? a.talk[h * H + k] : (h == k ? 1.0f : 0.0f)) : 0.0f;
+    const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+    talk_hi[h][k] = hi;
+    talk_lo[h][k] = __float2bfloat16_rn(v - __bfloat162float(hi));
   }
-  for (int h = warp; h < H; h += kMixThreads / 32) {
-    const float* row = sc + (int64_t)h * s.cols_pad;
-    float m = -INFINITY;
-    for (int c = lane; c < n; c += 32) m = fmaxf(m, row[c < kept ? c : w0 + c - kept]);
+  for (int h = warp; h < HM; h += kMixThreads / 32) {
+    const float2* st = reinterpret_cast<const float2*>(a.stats) + ((int64_t)i * H + h) * tiles;
+    float m = -INFINITY, sum = 0.0f;
+    for (int b = lane; h < H && b < tiles; b += 32)
+      if (tile_visible(s, q_tile, b * kCT, a.window, a.keep_first)) {
+        const float2 v = st[b];
+        const float to = fmaxf(m, v.x);
+        if (to > -INFINITY) sum = sum * __expf(m - to) + v.y * __expf(v.x - to);
+        m = to;
+      }
+    float M = m;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-    float sum = 0.0f;
-    for (int c = lane; c < n; c += 32) sum += expf(row[c < kept ? c : w0 + c - kept] - m);
-    sum = warp_sum(sum);
+    for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+    sum = warp_sum(m > -INFINITY ? sum * __expf(m - M) : 0.0f);
     if (lane == 0) {
-      mx[h] = m;
-      inv[h] = 1.0f / sum;
+      mx[h] = h < H ? M : 0.0f;
+      inv[h] = h < H ? 1.0f / sum : 0.0f;
     }
   }
   __syncthreads();
-  const int q_tile = i / kQT * kQT;
-  for (int c = tid; c < s.cols_pad; c += kMixThreads) {
-    float* col = sc + c;
-    if (!(c < kept || (c >= w0 && c <= w1))) {
-      if (tile_visible(s, q_tile, c / kCT * kCT, a.window, a.keep_first))
-        for (int h = 0; h < H; ++h) reinterpret_cast<uint32_t*>(col)[(int64_t)h * s.cols_pad] = 0u;
-      continue;
-    }
-    float p[HM];
+  // 8 columns per turn and warp: weights of all heads as the B operand (k = head, n = column), mixed ones as C
+  for (int c0 = 8 * warp; c0 < s.cols_pad; c0 += 8 * (kMixThreads / 32)) {
+    if (!tile_visible(s, q_tile, c0 / kCT * kCT, a.window, a.keep_first)) continue;
+    const int c = c0 + g;
+    const bool sees = span.sees(c);
+    float p[MT][4];
 #pragma unroll
-    for (int h = 0; h < HM; ++h) p[h] = h < H ? expf(col[(int64_t)h * s.cols_pad] - mx[h]) * inv[h] : 0.0f;
-#pragma unroll 4
-    for (int h = 0; h < H; ++h) {
-      float w = 0.0f;
+    for (int kt = 0; kt < MT; ++kt)
 #pragma unroll
-      for (int g = 0; g < HM; g += 4) {
-        const float4 tk = *reinterpret_cast<const float4*>(talk + h * HM + g);
-        w = fmaf(tk.x, p[g], w);
-        w = fmaf(tk.y, p[g + 1], w);
-        w = fmaf(tk.z, p[g + 2], w);
-        w = fmaf(tk.w, p[g + 3], w);
+      for (int e = 0; e < 4; ++e) {
+        const int h = 16 * kt + 2 * t + (e & 1) + 8 * (e >> 1);
+        p[kt][e] = sees && h < H ? sc[(int64_t)h * s.cols_pad + c] : 0.0f;
       }
-      const __nv_bfloat16 hi = __float2bfloat16_rn(w), rest = __float2bfloat16_rn(w - __bfloat162float(hi));
-      reinterpret_cast<uint32_t*>(col)[(int64_t)h * s.cols_pad] = (uint32_t)__bfloat16_as_ushort(hi) | (uint32_t)__bfloat16_as_ushort(rest) << 16;
+    uint32_t hi[MT][2], lo[MT][2];
+#pragma unroll
+    for (int kt = 0; kt < MT; ++kt) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int h = 16 * kt + 2 * t + (e & 1) + 8 * (e >> 1);
+        p[kt][e] = sees && h < H ? __expf(p[kt][e] - mx[h]) * inv[h] : 0.0f;
+      }
+      split2(p[kt][0], p[kt][1], hi[kt][0], lo[kt][0]);
+      split2(p[kt][2], p[kt][3], hi[kt][1], lo[kt][1]);
+    }
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      float w[4] = {};
+#pragma unroll
+      for (int kt = 0; kt < MT; ++kt) {
+        uint32_t th[4], tl[4];
+        ldsm(th, &talk_hi[16 * mt + (lane & 15)][16 * kt + (lane >> 4) * 8]);
+        ldsm(tl, &talk_lo[16 * mt + (lane & 15)][16 * kt + (lane >> 4) * 8]);
+        mma_bf16_16816(w, th, hi[kt][0], hi[kt][1]);
+        mma_bf16_16816(w, th, lo[kt][0], lo[kt][1]);
+        mma_bf16_16816(w, tl, hi[kt][0], hi[kt][1]);
+      }
+      // every lane's scores of these columns are in its operands by now: their places are free
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int h = 16 * mt + g + 8 * half;
+        if (h >= H) continue;
+        uint32_t wh, wl;
+        split2(w[2 * half], w[2 * half + 1], wh, wl);
+        *reinterpret_cast<uint2*>(sc + (int64_t)h * s.cols_pad + c0 + 2 * t) = make_uint2(__byte_perm(wh, wl, 0x5410), __byte_perm(wh, wl, 0x7632));
+      }
     }
   }
 }
 
-// grid (query tiles, heads, blocks of 8 NT value columns)
+// grid (query tiles, heads, blocks of 8 NT value columns).  Eight warps: 16 query rows each, twice -- the second four
+// warps take the second half of every key tile, and the halves are added at the end
+constexpr int kValuesThreads = 256, kValuesStages = 3;
 template <int NT>
 struct ValuesSmem {
   static constexpr int kWRow = kCT + 4, kVRow = 8 * NT + 8;
-  uint32_t w[2][kQT][kWRow];
-  __nv_bfloat16 v[2][kCT][kVRow];
+  uint32_t w[kValuesStages][kQT][kWRow];
+  __nv_bfloat16 v[kValuesStages][kCT][kVRow];
 };
 template <int NT>
-__global__ void __launch_bounds__(kMmaThreads) mix_prompt_values_kernel(const MixAttnArgs a, const int seq, const Strip s, __nv_bfloat16* __restrict__ out,
+__global__ void __launch_bounds__(kValuesThreads) mix_prompt_values_kernel(const MixAttnArgs a, const int seq, const Strip s, __nv_bfloat16* __restrict__ out,
                                                                         int64_t ldo) {
   extern __shared__ __align__(16) unsigned char raw[];
   ValuesSmem<NT>& sm = *reinterpret_cast<ValuesSmem<NT>*>(raw);
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, half_of_keys = tid >> 7, g = lane >> 2, t = lane & 3;
   const int i0 = blockIdx.x * kQT, h = blockIdx.y, v0 = blockIdx.z * 8 * NT, n_rep = a.heads / a.kv_heads;
   const uint32_t* w = reinterpret_cast<const uint32_t*>(a.scores);
   const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(a.v) + ((int64_t)seq * a.kv_heads + h / n_rep) * a.capacity * a.vdim_pad;
   auto issue = [&](int c0, int buf) {
-    for (int i = tid; i < kQT * (kCT / 4); i += kMmaThreads) {
+    for (int i = tid; i < kQT * (kCT / 4); i += kValuesThreads) {
       const int r = i / (kCT / 4), c = i % (kCT / 4) * 4;
       const bool live = i0 + r < s.rows;
       cp16_zfill(&sm.w[buf][r][c], w + (live ? ((int64_t)(i0 + r) * a.heads + h) * s.cols_pad + c0 + c : 0), live);
     }
-    for (int i = tid; i < kCT * NT; i += kMmaThreads) {
+    for (int i = tid; i < kCT * NT; i += kValuesThreads) {
       const int r = i / NT, c = i % NT * 8;
       const bool live = c0 + r < s.cols && v0 + c < a.vdim_pad;
       cp16_zfill(&sm.v[buf][r][c], v + (live ? (int64_t)strip_key(s, c0 + r) * a.vdim_pad + v0 + c : 0), live);
@@ -474,19 +533,29 @@ __global__ void __launch_bounds__(kMmaThreads) mix_prompt_values_kernel(const Mi
     return c0;
   };
   float acc[NT][4] = {};
-  int c0 = next(0), buf = 0;
-  if (c0 < s.cols_pad) issue(c0, 0);
-  while (c0 < s.cols_pad) {
-    const int c1 = next(c0 + kCT);
-    if (c1 < s.cols_pad) {
-      issue(c1, buf ^ 1);
-      asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+  // a ring of three tiles, two of them on their way while one is worked on
+  int ahead = next(0), work = 0, fill = 0, pending = 0;
+  auto feed = [&]() {
+    if (ahead < s.cols_pad) {
+      issue(ahead, fill);
+      fill = fill == kValuesStages - 1 ? 0 : fill + 1;
+      ahead = next(ahead + kCT);
+      ++pending;
     } else {
-      asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+      asm volatile("cp.async.commit_group;\n" ::: "memory");   // empty, so that the count below holds
     }
-    __syncthreads();
+  };
+  feed();
+  feed();
+  for (; pending > 0; --pending) {
+    asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+    __syncthreads();   // the tile has landed, and the one worked on before it is free
+    feed();
+    const int buf = work;
+    work = work == kValuesStages - 1 ? 0 : work + 1;
 #pragma unroll
-    for (int kk = 0; kk < kCT / 16; ++kk) {
+    for (int kh = 0; kh < kCT / 32; ++kh) {
+      const int kk = 2 * half_of_keys + kh;
       uint32_t hi[4], lo[4];
 #pragma unroll
       for (int part = 0; part < 4; ++part) {
@@ -504,10 +573,22 @@ __global__ void __launch_bounds__(kMmaThreads) mix_prompt_values_kernel(const Mi
         mma_bf16_16816(acc[2 * np + 1], lo, b[2], b[3]);
       }
     }
-    __syncthreads();
-    c0 = c1;
-    buf ^= 1;
   }
+  __syncthreads();
+  // add the halves through shared memory 
+  float* sum = reinterpret_cast<float*>(raw) + (tid & 127);
+  static_assert(sizeof(ValuesSmem<NT>) >= 4 * 128 * 4 * NT, "room for one half's accumulators");
+  if (half_of_keys == 1)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sum[128 * (4 * nt + e)] = acc[nt][e];
+  __syncthreads();
+  if (half_of_keys == 1) return;
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[nt][e] += sum[128 * (4 * nt + e)];
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int i = i0 + 16 * warp + g + 8 * half;
@@ -528,7 +609,7 @@ cudaError_t launch_prompt_values(const MixAttnArgs& a, int seq, const Strip& s, 
   const int smem = (int)sizeof(ValuesSmem<NT>);
   const cudaError_t e = cudaFuncSetAttribute(mix_prompt_values_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return e;
-  mix_prompt_values_kernel<NT><<<dim3((s.rows + kQT - 1) / kQT, a.heads, (a.vdim_pad + 8 * NT - 1) / (8 * NT)), kMmaThreads, smem, st>>>(a, seq, s, out, ldo);
+  mix_prompt_values_kernel<NT><<<dim3((s.rows + kQT - 1) / kQT, a.heads, (a.vdim_pad + 8 * NT - 1) / (8 * NT)), kValuesThreads, smem, st>>>(a, seq, s, out, ldo);
   return cudaGetLastError();
 }
 
@@ -550,7 +631,7 @@ Strip make_strip(const MixAttnArgs& a, int row0, int rows, int pos0) {
 bool mix_attention_prompt_supported(const MixAttnArgs& a) {
   // one tile of query rows must fit the scratch
   const uint64_t widest = ((uint64_t)a.max_visible + 2 * kQT + kCT) * a.heads * kQT;
-  return a.heads <= 64 && a.dim_pad % 16 == 0 && a.dim_pad <= 256 && widest <= a.scores_floats;
+  return a.heads <= 64 && a.dim_pad % 16 == 0 && a.dim_pad <= 256 && widest <= a.scores_floats && widest / 32 <= a.stats_floats;
 }
 
 cudaError_t launch_mix_attention_prompt(const MixAttnArgs& a, const Rows& rows, int pos0, __nv_bfloat16* out, int64_t ldo, cudaStream_t st,
@@ -565,20 +646,18 @@ cudaError_t launch_mix_attention_prompt(const MixAttnArgs& a, const Rows& rows, 
     while (n < rows.n - r0 && n < 256) {
       const int more = rows.n - r0 < n + kQT ? rows.n - r0 : n + kQT;
       const Strip t = make_strip(a, r0, more, pos0 + r0);
-      if ((uint64_t)t.rows * a.heads * t.cols_pad > a.scores_floats) break;
+      if ((uint64_t)t.rows * a.heads * t.cols_pad > a.scores_floats || (uint64_t)t.rows * a.heads * t.cols_pad / 32 > a.stats_floats) break;
       n = more;
       s = t;
     }
-    mix_prompt_scores_kernel<<<dim3(s.cols_pad / kCT, (n + kQT - 1) / kQT, a.kv_heads), kMmaThreads, smem, st>>>(a, rows.seq0, s);
-    if (a.heads <= 8) mix_prompt_weights_kernel<8><<<n, kMixThreads, 0, st>>>(a, s);
-    else if (a.heads <= 16) mix_prompt_weights_kernel<16><<<n, kMixThreads, 0, st>>>(a, s);
+    mix_prompt_scores_kernel<<<dim3(s.cols_pad / kCT, (n + kQT - 1) / kQT, a.heads), kMmaThreads, smem, st>>>(a, rows.seq0, s);
+    if (a.heads <= 16) mix_prompt_weights_kernel<16><<<n, kMixThreads, 0, st>>>(a, s);
     else if (a.heads <= 32) mix_prompt_weights_kernel<32><<<n, kMixThreads, 0, st>>>(a, s);
     else mix_prompt_weights_kernel<64><<<n, kMixThreads, 0, st>>>(a, s);
     e = cudaGetLastError();
     if (e != cudaSuccess) break;
     if (a.vdim_pad <= 32) e = launch_prompt_values<4>(a, rows.seq0, s, out, ldo, st);
-    else if (a.vdim_pad <= 64) e = launch_prompt_values<8>(a, rows.seq0, s, out, ldo, st);
-    else e = launch_prompt_values<16>(a, rows.seq0, s, out, ldo, st);
+    else e = launch_prompt_values<8>(a, rows.seq0, s, out, ldo, st);
     *launches += 3;
     r0 += n;
   }

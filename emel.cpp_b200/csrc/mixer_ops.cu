@@ -21,6 +21,7 @@ __device__ __forceinline__ __nv_bfloat16 to<__nv_bfloat16>(float x) { return __f
 __device__ __forceinline__ float from(float x) { return x; }
 __device__ __forceinline__ float from(__nv_bfloat16 x) { return __bfloat162float(x); }
 
+template <int WARPS = kWarps>
 __device__ __forceinline__ float block_sum(float v, float* scratch) {
   v = warp_sum(v);
   __syncthreads();
@@ -28,9 +29,12 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   __syncthreads();
   float t = 0.0f;
 #pragma unroll
-  for (int w = 0; w < kWarps; ++w) t += scratch[w];
+  for (int w = 0; w < WARPS; ++w) t += scratch[w];
   return t;
 }
+
+__device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
 
 template <class T>
 __global__ void embed_rows_bf16_kernel(const __nv_bfloat16* __restrict__ table, int64_t ld, const int* __restrict__ tokens, int width,
@@ -108,11 +112,31 @@ __global__ void glu_rows_kernel(const float* __restrict__ gu, int ff, float* __r
   out[r * ldo + i] = g / (1.0f + expf(-g)) * u;
 }
 
-// One block = one row of the queries (part 0), keys (1) or values (2).
-template <class T>
-__global__ void __launch_bounds__(kThreads) attn_in_kernel(const AttnInArgs a, const Rows rows) {
-  extern __shared__ float s[];
-  __shared__ float scratch[kWarps];
+// V = 1 or 4 consecutive channels
+template <int V>
+struct Chan { float f[V]; };
+template <int V>
+__device__ __forceinline__ Chan<V> load_chan(const float* p) {
+  Chan<V> c;
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    c.f[0] = v.x; c.f[1] = v.y; c.f[2] = v.z; c.f[3] = v.w;
+  } else {
+    c.f[0] = *p;
+  }
+  return c;
+}
+template <int V>
+__device__ __forceinline__ void store_chan(float* p, const Chan<V>& c) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(c.f[0], c.f[1], c.f[2], c.f[3]);
+  else *p = c.f[0];
+}
+
+// One block = one row of the queries (part 0), keys (1) or values (2), V channels per thread and turn.
+template <class T, int THREADS, int V>
+__global__ void __launch_bounds__(THREADS) attn_in_kernel(const AttnInArgs a, const Rows rows) {
+  extern __shared__ __align__(16) float s[];
+  __shared__ float scratch[THREADS / 32];
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
@@ -121,35 +145,43 @@ __global__ void __launch_bounds__(kThreads) attn_in_kernel(const AttnInArgs a, c
   const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
   const int n = part == 0 ? nq : part == 1 ? nk : nv, off = part == 0 ? 0 : part == 1 ? nq : nq + nk;
   const int hist = a.taps - 1;
+  float* state = a.conv_state + (int64_t)seq * hist * a.channels;
 
   float ss = 0.0f;
-  for (int i = tid; i < n; i += kThreads) {
+  for (int i = tid * V; i < n; i += THREADS * V) {
     const int c = off + i;
-    const float u = a.proj[(int64_t)r * a.channels + c];
-    float y = u;
+    const Chan<V> u = load_chan<V>(a.proj + (int64_t)r * a.channels + c);
+    Chan<V> y = u;
     if (a.conv) {
-      const float* w = a.conv + (int64_t)c * a.taps;
-      float* st = a.conv_state + ((int64_t)seq * a.channels + c) * hist;
-      y = w[hist] * u;
-      for (int b = 1; b <= hist; ++b) {   // b tokens back
-        float past = 0.0f;
-        if (pos - b >= 0) past = rows.prompt && r - b >= 0 ? a.proj[(int64_t)(r - b) * a.channels + c] : st[hist - (rows.prompt ? b - r : b)];
-        y = fmaf(w[hist - b], past, y);
+      const Chan<V> wl = load_chan<V>(a.conv + (int64_t)hist * a.channels + c);
+#pragma unroll
+      for (int e = 0; e < V; ++e) y.f[e] = wl.f[e] * u.f[e];
+      for (int b = 1; b <= hist && b <= pos; ++b) {   // b tokens back
+        const Chan<V> past = rows.prompt && r - b >= 0 ? load_chan<V>(a.proj + (int64_t)(r - b) * a.channels + c)
+                                                       : load_chan<V>(state + (int64_t)(hist - (rows.prompt ? b - r : b)) * a.channels + c);
+        const Chan<V> w = load_chan<V>(a.conv + (int64_t)(hist - b) * a.channels + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y.f[e] = fmaf(w.f[e], past.f[e], y.f[e]);
       }
       if (!rows.prompt) {
-        for (int j = 0; j + 1 < hist; ++j) st[j] = pos - hist + 1 + j >= 0 ? st[j + 1] : 0.0f;
-        if (hist > 0) st[hist - 1] = u;
+        for (int j = 0; j + 1 < hist; ++j) {
+          Chan<V> next = load_chan<V>(state + (int64_t)(j + 1) * a.channels + c);
+          if (pos - hist + 1 + j < 0) next = Chan<V>{};
+          store_chan<V>(state + (int64_t)j * a.channels + c, next);
+        }
+        if (hist > 0) store_chan<V>(state + (int64_t)(hist - 1) * a.channels + c, u);
       }
     }
-    s[i] = y;
-    ss = fmaf(y, y, ss);
+    store_chan<V>(s + i, y);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(y.f[e], y.f[e], ss);
   }
 
   if (part == 2) {
     __syncthreads();
     // a warp per value head
     T* cache = static_cast<T*>(a.v);
-    for (int h = tid >> 5; h < a.kv_heads; h += kWarps) {
+    for (int h = tid >> 5; h < a.kv_heads; h += THREADS / 32) {
       const float* v = s + h * a.vdim;
       float inv = 1.0f;
       if (a.norm_v) {
@@ -158,17 +190,18 @@ __global__ void __launch_bounds__(kThreads) attn_in_kernel(const AttnInArgs a, c
         inv = 1.0f / sqrtf(warp_sum(t) / a.vdim + a.eps);
       }
       T* row = cache + (((int64_t)seq * a.kv_heads + h) * a.capacity + pos) * a.vdim_pad;
-      for (int d = tid & 31; d < a.vdim_pad; d += 32) row[d] = to<T>(d < a.vdim ? v[d] * inv : 0.0f);
+      for (int d = 2 * (tid & 31); d < a.vdim_pad; d += 64)
+        store_pair(row + d, d < a.vdim ? v[d] * inv : 0.0f, d + 1 < a.vdim ? v[d + 1] * inv : 0.0f);
     }
     return;
   }
   const float* nw = part == 0 ? a.norm_q : a.norm_k;
-  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / n + a.eps);   // also orders the writes of s
+  const float inv = 1.0f / sqrtf(block_sum<THREADS / 32>(ss, scratch) / n + a.eps);   // also orders the writes of s
   const int heads = part == 0 ? a.heads : a.kv_heads;
   auto normed = [&](int i) { return nw ? s[i] * inv * nw[i] : s[i]; };
   const int half_pad = a.dim_pad / 2;
-  for (int idx = tid; idx < heads * half_pad; idx += kThreads) {
-    const int h = idx / half_pad, p = idx % half_pad, d = 2 * p;
+  for (int idx = tid; idx < heads * half_pad; idx += THREADS) {
+    const int h = idx / half_pad, p = idx - h * half_pad, d = 2 * p;
     float x0 = d < a.dim ? normed(h * a.dim + d) : 0.0f, x1 = d + 1 < a.dim ? normed(h * a.dim + d + 1) : 0.0f;
     if (d < a.rope_dim) {
       const int64_t t = (int64_t)pos * (a.rope_dim / 2) + p;
@@ -179,22 +212,21 @@ __global__ void __launch_bounds__(kThreads) attn_in_kernel(const AttnInArgs a, c
     }
     T* row = part == 0 ? static_cast<T*>(a.q) + ((int64_t)r * a.heads + h) * a.dim_pad
                        : static_cast<T*>(a.k) + (((int64_t)seq * a.kv_heads + h) * a.capacity + pos) * a.dim_pad;
-    row[d] = to<T>(x0);
-    row[d + 1] = to<T>(x1);
+    store_pair(row + d, x0, x1);
   }
 }
 
 __global__ void conv_state_kernel(const AttnInArgs a, const Rows rows) {
   const int c = blockIdx.x * kThreads + threadIdx.x, hist = a.taps - 1;
   if (c >= a.channels) return;
-  float* st = a.conv_state + ((int64_t)rows.seq0 * a.channels + c) * hist;
+  float* st = a.conv_state + (int64_t)rows.seq0 * hist * a.channels + c;
   // entry j holds the row hist - j before the next one; an old entry moves down by rows.n >= 1 places
   for (int j = 0; j < hist; ++j) {
     const int r = rows.n - hist + j;
     float v = 0.0f;
     if (r >= 0) v = a.proj[(int64_t)r * a.channels + c];
-    else if (rows.pos[0] + r >= 0) v = st[hist + r];
-    st[j] = v;
+    else if (rows.pos[0] + r >= 0) v = st[(int64_t)(hist + r) * a.channels];
+    st[(int64_t)j * a.channels] = v;
   }
 }
 
@@ -257,15 +289,24 @@ cudaError_t launch_glu_rows(const float* gu, int rows, int ff, float* out, int64
   return cudaGetLastError();
 }
 
+namespace {
+template <class T, int THREADS, int V>
+cudaError_t launch_attn_in_sized(const AttnInArgs& a, const Rows& rows, size_t smem, cudaStream_t st) {
+  const cudaError_t e = allow_smem(attn_in_kernel<T, THREADS, V>, smem);
+  if (e != cudaSuccess) return e;
+  attn_in_kernel<T, THREADS, V><<<dim3(rows.n, a.own_kv ? 3 : 1), THREADS, smem, st>>>(a, rows);
+  return cudaGetLastError();
+}
+}  // namespace
+
 template <class T>
 cudaError_t launch_attn_in(const AttnInArgs& a, const Rows& rows, cudaStream_t st) {
-  int n = a.heads * a.dim;
-  if (a.own_kv && a.kv_heads * a.vdim > n) n = a.kv_heads * a.vdim;
-  const size_t smem = 4 * (size_t)n;
-  const cudaError_t e = allow_smem(attn_in_kernel<T>, smem);
-  if (e != cudaSuccess) return e;
-  attn_in_kernel<T><<<dim3(rows.n, a.own_kv ? 3 : 1), kThreads, smem, st>>>(a, rows);
-  return cudaGetLastError();
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+  const size_t smem = 4 * (size_t)(a.own_kv && nv > nq ? nv : nq);
+  const bool quads = nq % 4 == 0 && (!a.own_kv || (nk % 4 == 0 && nv % 4 == 0));
+  // few rows: a wide block each
+  if (rows.n <= 16) return quads ? launch_attn_in_sized<T, 1024, 4>(a, rows, smem, st) : launch_attn_in_sized<T, 1024, 1>(a, rows, smem, st);
+  return quads ? launch_attn_in_sized<T, kThreads, 4>(a, rows, smem, st) : launch_attn_in_sized<T, kThreads, 1>(a, rows, smem, st);
 }
 template cudaError_t launch_attn_in<float>(const AttnInArgs&, const Rows&, cudaStream_t);
 template cudaError_t launch_attn_in<__nv_bfloat16>(const AttnInArgs&, const Rows&, cudaStream_t);

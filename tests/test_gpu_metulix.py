@@ -390,3 +390,16 @@ def test_trace_runner(cases, tmp_path, f32):
         got = np.fromfile(tmp_path / f"{step}.f32", "<f4").reshape(len(rows), -1)
         assert mm.row_errors(got, c.logits[rows]).max() < 1.5 * TOL[f32], step
     assert not (tmp_path / "1.f32").exists()
+
+
+@BOTH
+def test_long_prompts(be, tmp_path, f32):
+    """Prompts of several key strips and several segments of the linear state, whole, cut and continued."""
+    cfg = mm.model(96, 60, [mm.lightning(2, 48, 40, [0.999, 0.97], ff=64), mm.attention(4, 2, 32, 32, 0.5, conv=3, rot=(32, 5000.0), window=330, keep=7),
+                            mm.lightning(3, 32, 72, [0.9995, 0.6, 1.0]), mm.attention(4, 2, 32, 32, 0.5, conv=2, rot=(32, 5000.0), kv_from=1)])
+    cfg["layers"][3]["mixer"].pop("mask", None)     # the borrowing layer sees everything
+    c = Case(cfg, tmp_path / "m", 1150, 41)
+    s = c.session(be, f32, n_ctx=1152)
+    for sizes in ([1150], [700, 449, 1], [1, 600, 549], [511, 3, 636]):
+        assert_close(mm.row_errors(feed(s, c.tokens, sizes), c.logits), f32, sizes)
+    s.close()
