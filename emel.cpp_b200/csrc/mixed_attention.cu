@@ -373,13 +373,16 @@ __global__ void __launch_bounds__(kMmaThreads) mix_prompt_scores_kernel(const Mi
       mma_bf16_16816(acc[2 * nt + 1], qa, b[2], b[3]);
     }
   }
+  // the scores leave through shared memory, whole rows of the tile at a time
+  constexpr int kTileRow = kCT + 4;
+  float* tile = reinterpret_cast<float*>(raw);
+  __syncthreads();
   // every row of the tile sees every column: the last row's window starts at or before it, the first row's ends after it
   const bool inside = row_span(s, min(i0 + kQT, s.rows) - 1, a.window, a.keep_first).w0 <= c0 && row_span(s, i0, a.window, a.keep_first).w1 >= c0 + kCT - 1;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int i = i0 + 16 * warp + g + 8 * half;
     const RowSpan span = row_span(s, i, a.window, a.keep_first);
-    float* out = a.scores + ((int64_t)i * a.heads + h) * s.cols_pad + c0;
     float m = -INFINITY, sum = 0.0f;
 #pragma unroll
     for (int nt = 0; nt < kCT / 8; ++nt) {
@@ -388,7 +391,7 @@ __global__ void __launch_bounds__(kMmaThreads) mix_prompt_scores_kernel(const Mi
         float& v = acc[nt][2 * half + e];
         v *= a.scale;
       }
-      if (i < s.rows) *reinterpret_cast<float2*>(out + 8 * nt + 2 * t) = make_float2(acc[nt][2 * half], acc[nt][2 * half + 1]);
+      *reinterpret_cast<float2*>(tile + (16 * warp + g + 8 * half) * kTileRow + 8 * nt + 2 * t) = make_float2(acc[nt][2 * half], acc[nt][2 * half + 1]);
       if (!inside) {
 #pragma unroll
         for (int e = 0; e < 2; ++e)
@@ -407,26 +410,56 @@ __global__ void __launch_bounds__(kMmaThreads) mix_prompt_scores_kernel(const Mi
     sum += __shfl_xor_sync(0xffffffffu, sum, 2);
     if (t == 0 && i < s.rows) reinterpret_cast<float2*>(a.stats)[((int64_t)i * a.heads + h) * (s.cols_pad / kCT) + blockIdx.x] = make_float2(m, sum);
   }
+  __syncwarp();   // a warp stores the 16 rows it wrote
+#pragma unroll
+  for (int x = lane; x < 16 * (kCT / 4); x += 32) {
+    const int r = 16 * warp + x / (kCT / 4), c = x % (kCT / 4) * 4;
+    if (i0 + r < s.rows)
+      *reinterpret_cast<float4*>(a.scores + ((int64_t)(i0 + r) * a.heads + h) * s.cols_pad + c0 + c) = *reinterpret_cast<const float4*>(tile + r * kTileRow + c);
+  }
 }
 
 constexpr int kMixThreads = 256;
 
-// one block per row; heads padded to HM, a multiple of 16
+// grid (rows, shares of the column tiles); heads padded to HM, a multiple of 16
+template <int HM>
+struct WeightsSmem {
+  static constexpr int kTalkRow = HM + 8, kTileRow = kCT + 4, kStages = 3;
+  float tile[kStages][HM][kTileRow];            // 64 columns of every head's scores, then of the mixed weights
+  __nv_bfloat16 talk_hi[HM][kTalkRow], talk_lo[HM][kTalkRow];
+  float mx[HM], inv[HM];
+};
 template <int HM>
 __global__ void __launch_bounds__(kMixThreads) mix_prompt_weights_kernel(const MixAttnArgs a, const Strip s) {
-  constexpr int kRow = HM + 8, MT = HM / 16;
-  __shared__ __align__(16) __nv_bfloat16 talk_hi[HM][kRow], talk_lo[HM][kRow];
-  __shared__ float mx[HM], inv[HM];
+  constexpr int MT = HM / 16;
+  static_assert(kMixThreads / 32 * 8 == kCT, "eight columns per warp");
+  extern __shared__ __align__(16) unsigned char raw[];
+  WeightsSmem<HM>& sm = *reinterpret_cast<WeightsSmem<HM>*>(raw);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, H = a.heads;
   const int i = blockIdx.x, tiles = s.cols_pad / kCT, q_tile = i / kQT * kQT;
   const RowSpan span = row_span(s, i, a.window, a.keep_first);
   float* sc = a.scores + (int64_t)i * H * s.cols_pad;
+  auto next = [&](int b) {
+    while (b < tiles && !tile_visible(s, q_tile, b * kCT, a.window, a.keep_first)) b += gridDim.y;
+    return b;
+  };
+  auto issue = [&](int b, int buf) {
+    if (b < tiles)
+      for (int x = tid; x < H * (kCT / 4); x += kMixThreads) {
+        const int h = x / (kCT / 4), c = x % (kCT / 4) * 4;
+        cp16_zfill(&sm.tile[buf][h][c], sc + (int64_t)h * s.cols_pad + b * kCT + c, true);
+      }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  int b0 = next(blockIdx.y), b1 = next(b0 + gridDim.y), buf = 0;
+  issue(b0, 0);
+  issue(b1, 1);
   for (int x = tid; x < HM * HM; x += kMixThreads) {
     const int h = x / HM, k = x % HM;
     const float v = h < H && k < H ? (a.talk ? a.talk[h * H + k] : (h == k ? 1.0f : 0.0f)) : 0.0f;
     const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-    talk_hi[h][k] = hi;
-    talk_lo[h][k] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    sm.talk_hi[h][k] = hi;
+    sm.talk_lo[h][k] = __float2bfloat16_rn(v - __bfloat162float(hi));
   }
   for (int h = warp; h < HM; h += kMixThreads / 32) {
     const float2* st = reinterpret_cast<const float2*>(a.stats) + ((int64_t)i * H + h) * tiles;
@@ -443,58 +476,73 @@ __global__ void __launch_bounds__(kMixThreads) mix_prompt_weights_kernel(const M
     for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
     sum = warp_sum(m > -INFINITY ? sum * __expf(m - M) : 0.0f);
     if (lane == 0) {
-      mx[h] = h < H ? M : 0.0f;
-      inv[h] = h < H ? 1.0f / sum : 0.0f;
+      sm.mx[h] = h < H ? M : 0.0f;
+      sm.inv[h] = h < H ? 1.0f / sum : 0.0f;
     }
   }
   __syncthreads();
-  // 8 columns per turn and warp: weights of all heads as the B operand (k = head, n = column), mixed ones as C
-  for (int c0 = 8 * warp; c0 < s.cols_pad; c0 += 8 * (kMixThreads / 32)) {
-    if (!tile_visible(s, q_tile, c0 / kCT * kCT, a.window, a.keep_first)) continue;
-    const int c = c0 + g;
-    const bool sees = span.sees(c);
-    float p[MT][4];
-#pragma unroll
-    for (int kt = 0; kt < MT; ++kt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int h = 16 * kt + 2 * t + (e & 1) + 8 * (e >> 1);
-        p[kt][e] = sees && h < H ? sc[(int64_t)h * s.cols_pad + c] : 0.0f;
-      }
+  // 8 columns per warp: weights of all heads as the B operand (k = head, n = column), mixed ones as C
+  while (b0 < tiles) {
+    asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+    __syncthreads();   // this tile has landed; the one before it has been stored
+    const int b2 = next(b1 + gridDim.y);
+    issue(b2, buf == 0 ? 2 : buf - 1);
+    float (*tile)[WeightsSmem<HM>::kTileRow] = sm.tile[buf];
+    const int c0 = 8 * warp;
+    const bool sees = span.sees(b0 * kCT + c0 + g);
     uint32_t hi[MT][2], lo[MT][2];
 #pragma unroll
     for (int kt = 0; kt < MT; ++kt) {
+      float p[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int h = 16 * kt + 2 * t + (e & 1) + 8 * (e >> 1);
-        p[kt][e] = sees && h < H ? __expf(p[kt][e] - mx[h]) * inv[h] : 0.0f;
+        p[e] = sees && h < H ? __expf(tile[h][c0 + g] - sm.mx[h]) * sm.inv[h] : 0.0f;
       }
-      split2(p[kt][0], p[kt][1], hi[kt][0], lo[kt][0]);
-      split2(p[kt][2], p[kt][3], hi[kt][1], lo[kt][1]);
+      split2(p[0], p[1], hi[kt][0], lo[kt][0]);
+      split2(p[2], p[3], hi[kt][1], lo[kt][1]);
     }
+    __syncwarp();
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       float w[4] = {};
 #pragma unroll
       for (int kt = 0; kt < MT; ++kt) {
         uint32_t th[4], tl[4];
-        ldsm(th, &talk_hi[16 * mt + (lane & 15)][16 * kt + (lane >> 4) * 8]);
-        ldsm(tl, &talk_lo[16 * mt + (lane & 15)][16 * kt + (lane >> 4) * 8]);
+        ldsm(th, &sm.talk_hi[16 * mt + (lane & 15)][16 * kt + (lane >> 4) * 8]);
+        ldsm(tl, &sm.talk_lo[16 * mt + (lane & 15)][16 * kt + (lane >> 4) * 8]);
         mma_bf16_16816(w, th, hi[kt][0], hi[kt][1]);
         mma_bf16_16816(w, th, lo[kt][0], lo[kt][1]);
         mma_bf16_16816(w, tl, hi[kt][0], hi[kt][1]);
       }
-      // every lane's scores of these columns are in its operands by now: their places are free
+      // every lane's scores of the warp's columns are in its operands by now: their places are free
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int h = 16 * mt + g + 8 * half;
         if (h >= H) continue;
         uint32_t wh, wl;
         split2(w[2 * half], w[2 * half + 1], wh, wl);
-        *reinterpret_cast<uint2*>(sc + (int64_t)h * s.cols_pad + c0 + 2 * t) = make_uint2(__byte_perm(wh, wl, 0x5410), __byte_perm(wh, wl, 0x7632));
+        *reinterpret_cast<uint2*>(&tile[h][c0 + 2 * t]) = make_uint2(__byte_perm(wh, wl, 0x5410), __byte_perm(wh, wl, 0x7632));
       }
     }
+    __syncthreads();
+    for (int x = tid; x < H * (kCT / 4); x += kMixThreads) {
+      const int h = x / (kCT / 4), c = x % (kCT / 4) * 4;
+      *reinterpret_cast<float4*>(sc + (int64_t)h * s.cols_pad + b0 * kCT + c) = *reinterpret_cast<const float4*>(&tile[h][c]);
+    }
+    b0 = b1;
+    b1 = b2;
+    buf = buf == 2 ? 0 : buf + 1;
   }
+}
+
+template <int HM>
+cudaError_t launch_prompt_weights(const MixAttnArgs& a, const Strip& s, cudaStream_t st) {
+  const int smem = (int)sizeof(WeightsSmem<HM>), tiles = s.cols_pad / kCT;
+  const cudaError_t e = cudaFuncSetAttribute(mix_prompt_weights_kernel<HM>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return e;
+  mix_prompt_weights_kernel<HM><<<dim3(s.rows, tiles > 12 ? 3 : tiles > 6 ? 2 : 1), kMixThreads, smem, st>>>(a, s);
+  return cudaGetLastError();
 }
 
 // grid (query tiles, heads, blocks of 8 NT value columns).  Eight warps: 16 query rows each, twice -- the second four
@@ -636,7 +684,8 @@ bool mix_attention_prompt_supported(const MixAttnArgs& a) {
 
 cudaError_t launch_mix_attention_prompt(const MixAttnArgs& a, const Rows& rows, int pos0, __nv_bfloat16* out, int64_t ldo, cudaStream_t st,
                                         int* launches) {
-  const int smem = 2 * kQT * (a.dim_pad + 8) * 2;
+  int smem = 2 * kQT * (a.dim_pad + 8) * 2;
+  if (smem < kQT * (kCT + 4) * 4) smem = kQT * (kCT + 4) * 4;
   cudaError_t e = cudaSuccess;
   if (smem > 48 * 1024) e = cudaFuncSetAttribute(mix_prompt_scores_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   for (int r0 = 0; e == cudaSuccess && r0 < rows.n;) {
@@ -651,10 +700,9 @@ cudaError_t launch_mix_attention_prompt(const MixAttnArgs& a, const Rows& rows, 
       s = t;
     }
     mix_prompt_scores_kernel<<<dim3(s.cols_pad / kCT, (n + kQT - 1) / kQT, a.heads), kMmaThreads, smem, st>>>(a, rows.seq0, s);
-    if (a.heads <= 16) mix_prompt_weights_kernel<16><<<n, kMixThreads, 0, st>>>(a, s);
-    else if (a.heads <= 32) mix_prompt_weights_kernel<32><<<n, kMixThreads, 0, st>>>(a, s);
-    else mix_prompt_weights_kernel<64><<<n, kMixThreads, 0, st>>>(a, s);
     e = cudaGetLastError();
+    if (e != cudaSuccess) break;
+    e = a.heads <= 16 ? launch_prompt_weights<16>(a, s, st) : a.heads <= 32 ? launch_prompt_weights<32>(a, s, st) : launch_prompt_weights<64>(a, s, st);
     if (e != cudaSuccess) break;
     if (a.vdim_pad <= 32) e = launch_prompt_values<4>(a, rows.seq0, s, out, ldo, st);
     else e = launch_prompt_values<8>(a, rows.seq0, s, out, ldo, st);
