@@ -99,7 +99,7 @@ struct GemmParams {
 template <int BN, bool GLU>
 struct Tile {
   static constexpr int kStageBytes = (GLU ? 2 : 1) * kWeightTile + BN * kBK * 2;
-  static constexpr int kStages = BN == 128 && !GLU ? 3 : 4;
+  static constexpr int kStages = kStageBytes > 40 * 1024 ? 2 : BN == 128 ? 3 : 4;   // two CTAs per SM: one computes while the other stores
   static constexpr int kTmemCols = (GLU ? 2 : 1) * BN < 32 ? 32 : (GLU ? 2 : 1) * BN;
   static constexpr int kBox = BN >= 128 ? 128 : kGemmTokenBox;   // rows per TMA copy of x
   static constexpr int kSmem = kStages * kStageBytes + 1024 + 256;
@@ -260,8 +260,8 @@ cudaError_t launch_gemm_bf16(const LinearArgs& a, const TmaMap& wmap, const XMap
   }
   if (R <= 16) return launch_tile<16, false>(wmap, x.narrow, p, st);
   if (R <= 64) return launch_tile<64, false>(wmap, x.narrow, p, st);
-  // 256-row tiles once they fill the SMs
-  if (((p.M + kBM - 1) / kBM) * ((R + 255) / 256) >= 120) return launch_tile<256, false>(wmap, x.wide, p, st);
+  // 256-row tiles once there are more of them than SMs
+  if (((p.M + kBM - 1) / kBM) * ((R + 255) / 256) >= 180) return launch_tile<256, false>(wmap, x.wide, p, st);
   return launch_tile<128, false>(wmap, x.wide, p, st);
 }
 
