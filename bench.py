@@ -840,7 +840,7 @@ def build_metulix_session(be, sh, n_ctx, seed0=7000):
         if i % 2 == 0:
             layers.append(ly.linear_layer(H, D, D, decay, n_ff=ff))
         else:
-            layers.append(ly.attention_layer(H, G, D, D, D ** -0.5, conv_taps=3, rope_dim=D, rope_freq_base=20000.0, window=sh["window"],
+            layers.append(ly.attention_layer(H, G, D, D, D ** -0.5, conv_taps=3, rope_dim=D, rope_freq_base=10000.0, window=sh["window"],
                                              keep_first=sh["keep"], kv_from=i - 2 if i % 4 == 3 else -1, n_ff=ff))
     sess = ly.Session(be, ly.config(len(layers), W, sh["vocab"], n_ctx, 1e-6), layers)
     allocs, weight_bytes = [], 0
