@@ -35,6 +35,8 @@ SOURCES = {
     "mixer_ops.cu": [],
     "mixed_attention.cu": [],
     "lightning.cu": [],
+    "latent_attention.cu": [],
+    "delta.cu": [],
     "layered.cu": [],
     "llama.cu": [],
     "comm.cu": [],

@@ -10,6 +10,7 @@
 #include <cudaTypedefs.h>
 #include <cuda_runtime.h>
 
+#include "act.cuh"
 #include "common.cuh"
 #include "layered.h"
 
@@ -94,6 +95,10 @@ struct GemmParams {
   __nv_bfloat16* yb;
   int64_t ldy;
   int* status;
+  float out_scale, softcap;
+  int tail;                // first feature stored as f32 at tail_y
+  float* tail_y;
+  int64_t tail_ld;
 };
 
 template <int BN, bool GLU>
@@ -185,7 +190,7 @@ __global__ void __launch_bounds__(kThreads) gemm_bf16_kernel(const __grid_consta
       const bool live = f < p.M;
       const float b0 = live && p.bias ? p.bias[f] : 0.0f, b1 = GLU && live && p.bias ? p.bias[p.M + f] : 0.0f;
       const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
-      const bool sigm = p.act == ACT_SILU_SIGMOID;
+      const bool sigm = p.act == ACT_SILU_SIGMOID, gelu = p.act == ACT_GLU_GELU, cap = p.act == ACT_SOFTCAP, tail = f >= p.tail;
       for (int c = 0; c < BN && t0 + c < p.rows; c += 8) {
         uint32_t v[8], u[8];
         tmem_ld8(lane_base + c, v);
@@ -195,13 +200,16 @@ __global__ void __launch_bounds__(kThreads) gemm_bf16_kernel(const __grid_consta
         for (int j = 0; j < 8; ++j) {
           float o = __uint_as_float(v[j]) + b0;
           if (GLU) {
-            o = o / (1.0f + expf(-o)) * (__uint_as_float(u[j]) + b1);
+            o = (gelu ? gelu_tanhf_(o) : siluf_(o)) * (__uint_as_float(u[j]) + b1);
           } else if (sigm) {
-            const float sg = 1.0f / (1.0f + expf(-o));
+            const float sg = sigmoidf_(o);
             o = f < p.act_split ? o * sg : sg;
+          } else if (cap) {
+            o = softcapf_(o * p.out_scale, p.softcap);
           }
           if (live && t0 + c + j < p.rows) {
-            if (p.yb) p.yb[(int64_t)(t0 + c + j) * p.ldy + f] = __float2bfloat16_rn(o);
+            if (tail) p.tail_y[(int64_t)(t0 + c + j) * p.tail_ld + f - p.tail] = o;
+            else if (p.yb) p.yb[(int64_t)(t0 + c + j) * p.ldy + f] = __float2bfloat16_rn(o);
             else p.y[(int64_t)(t0 + c + j) * p.ldy + f] = o;
           }
         }
@@ -250,8 +258,9 @@ bool encode_bf16_map(TmaMap* map, const __nv_bfloat16* base, int64_t rows, int64
 
 cudaError_t launch_gemm_bf16(const LinearArgs& a, const TmaMap& wmap, const XMaps& x, float* y, __nv_bfloat16* yb, int64_t ldy, int* status,
                              cudaStream_t st) {
-  const bool glu = a.act == ACT_GLU;
-  GemmParams p{glu ? a.w.M / 2 : a.w.M, a.w.K, a.rows, a.bias, a.act, a.act_split, y, yb, ldy, status};
+  const bool glu = is_glu(a.act);
+  GemmParams p{glu ? a.w.M / 2 : a.w.M, a.w.K, a.rows, a.bias, a.act, a.act_split, y, yb, ldy, status,
+               a.out_scale, a.softcap, a.tail, a.tail_y, a.tail_ld};
   const int R = a.rows;
   if (glu) {
     if (R <= 16) return launch_tile<16, true>(wmap, x.narrow, p, st);

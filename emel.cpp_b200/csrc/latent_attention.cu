@@ -1,0 +1,349 @@
+// Softmax attention whose keys and values are projections of one cached latent per token (and, optionally, a rotated key
+// part all heads share).  A cache row is [latent (rank), zeros to rank_pad, rotated part, zeros to width].
+//
+// Row by row (decoding, batches, f32 sessions, short portions) keys and values are never formed:
+//   in     latent norm, rotation, cache row; the query against the key rows of its head: q . (U c) = (U^T q) . c
+//   attn   per key range and eight heads: scores, online softmax, weighted latents
+//   out    ranges merged, value rows of the head times the weighted latent, output gate
+#include <math.h>
+
+#include "act.cuh"
+#include "common.cuh"
+#include "layered.h"
+#include "mma_bf16.cuh"
+
+namespace emelb {
+namespace {
+
+constexpr int kThreads = 128;
+constexpr int kHG = 8;          // heads per block of the attention launch
+constexpr int kKeys = 64;       // keys per tile
+constexpr int kCols = 512;      // latent columns per block of the attention launch
+constexpr int kSlice = 64;      // latent columns per block of the query launch
+constexpr int kOutTile = 32;    // values per block of the out launch
+constexpr int kMaxSplits = 32;
+
+__device__ __forceinline__ float from(float x) { return x; }
+__device__ __forceinline__ float from(__nv_bfloat16 x) { return __bfloat162float(x); }
+template <class T> __device__ __forceinline__ T to(float x);
+template <> __device__ __forceinline__ float to<float>(float x) { return x; }
+template <> __device__ __forceinline__ __nv_bfloat16 to<__nv_bfloat16>(float x) { return __float2bfloat16_rn(x); }
+
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 v = *reinterpret_cast<const uint4*>(p);
+  const float2 a = unpack2(v.x), b = unpack2(v.y), c = unpack2(v.z), d = unpack2(v.w);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
+}
+__device__ __forceinline__ void load4(const float* p, float (&f)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack2(v.x), b = unpack2(v.y);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+
+__device__ __forceinline__ int row_pos(const Rows& r, int i) { return r.prompt ? r.pos[0] + i : r.pos[i]; }
+__device__ __forceinline__ int row_seq(const Rows& r, int i) { return r.prompt ? r.seq0 : r.seq0 + i; }
+__device__ __forceinline__ int first_key(int pos, int window) { return window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0; }
+
+// pair p of a rotated vector of n dimensions: its two places
+__device__ __forceinline__ void pair_of(int p, int n, int half, int& i, int& j) {
+  i = half ? p : 2 * p;
+  j = half ? p + n / 2 : 2 * p + 1;
+}
+
+// one block: the cache row of row r
+template <class TC>
+__device__ void store_latent(const LatentArgs& a, int r, int pos, int seq) {
+  __shared__ float scratch[kThreads / 32];
+  const float* x = a.down + (int64_t)r * a.ldd;
+  TC* row = static_cast<TC*>(a.cache) + ((int64_t)seq * a.capacity + pos) * a.width;
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < a.rank; i += kThreads) ss = fmaf(x[i], x[i], ss);
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float inv = 1.0f / sqrtf((scratch[0] + scratch[1] + scratch[2] + scratch[3]) / a.rank + a.eps);
+  for (int i = threadIdx.x; i < a.rank_pad; i += kThreads) row[i] = to<TC>(i < a.rank ? x[i] * inv * a.norm[i] : 0.0f);
+  const float* k = x + a.rank;
+  for (int p = threadIdx.x; p < a.rot / 2; p += kThreads) {
+    int i, j;
+    pair_of(p, a.rot, a.rope_half, i, j);
+    const float c = a.rope_cos[(int64_t)pos * (a.rot / 2) + p], s = a.rope_sin[(int64_t)pos * (a.rot / 2) + p];
+    row[a.rank_pad + i] = to<TC>(k[i] * c - k[j] * s);
+    row[a.rank_pad + j] = to<TC>(k[j] * c + k[i] * s);
+  }
+  for (int i = a.rank_pad + a.rot + threadIdx.x; i < a.width; i += kThreads) row[i] = to<TC>(0.0f);
+}
+
+// grid (column slices + 1, heads, rows): slices of U^T q of one head; the last slice rotates the head's query and, for
+// head 0, stores the cache row
+template <class TC, class TP>
+__global__ void __launch_bounds__(kThreads) latent_in_kernel(const LatentArgs a, const Rows rows, int row0) {
+  extern __shared__ float qs[];            // [dim], then the warps' partial columns
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.y, r = row0 + blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const TP* q = static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp + h * (a.dim + a.rot);
+  float* out = a.qlat + ((int64_t)blockIdx.z * a.heads + h) * a.width;
+  if (blockIdx.x == gridDim.x - 1) {
+    const int pos = row_pos(rows, r);
+    for (int p = tid; p < a.rot / 2; p += kThreads) {
+      int i, j;
+      pair_of(p, a.rot, a.rope_half, i, j);
+      const float c = a.rope_cos[(int64_t)pos * (a.rot / 2) + p], s = a.rope_sin[(int64_t)pos * (a.rot / 2) + p];
+      const float u = from(q[a.dim + i]), v = from(q[a.dim + j]);
+      out[a.rank_pad + i] = u * c - v * s;
+      out[a.rank_pad + j] = v * c + u * s;
+    }
+    for (int i = a.rank_pad + a.rot + tid; i < a.width; i += kThreads) out[i] = 0.0f;
+    if (h == 0) store_latent<TC>(a, r, pos, row_seq(rows, r));
+    return;
+  }
+  float* part = qs + a.dim;                // [warps][kSlice]
+  for (int i = tid; i < a.dim; i += kThreads) qs[i] = from(q[i]);
+  __syncthreads();
+  const int c = blockIdx.x * kSlice + 2 * lane;   // two columns per lane; rows of `up` are readable to a multiple of 8
+  float s0 = 0.0f, s1 = 0.0f;
+  if (c < a.rank_pad) {
+    const __nv_bfloat16* w = a.up.w + (int64_t)h * a.dim * a.up.ld + c;
+#pragma unroll 8
+    for (int d = warp; d < a.dim; d += kThreads / 32) {
+      const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(w + (int64_t)d * a.up.ld));
+      s0 = fmaf(qs[d], x.x, s0);
+      s1 = fmaf(qs[d], x.y, s1);
+    }
+  }
+  part[warp * kSlice + 2 * lane] = s0;
+  part[warp * kSlice + 2 * lane + 1] = s1;
+  __syncthreads();
+  const int col = blockIdx.x * kSlice + tid;
+  if (tid < kSlice && col < a.rank_pad) {
+    float s = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kThreads / 32; ++w) s += part[w * kSlice + tid];
+    out[col] = col < a.rank ? s : 0.0f;
+  }
+}
+
+// sums of N = 32 values over the warp's lanes; lane i returns with the sum of value i
+__device__ __forceinline__ float transpose_sum(float (&v)[32]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float give = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
+  }
+  return v[0];
+}
+
+// grid (ranges x column blocks, head groups, rows)
+template <class TC>
+__global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs a, const Rows rows, int row0, int splits) {
+  extern __shared__ __align__(16) float sm[];
+  float* qs = sm;                          // [kHG][width]
+  float* p = qs + kHG * a.width;           // [kHG][kKeys] scores, then weights
+  __shared__ float m_run[kHG], l_run[kHG], fix[kHG];
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int split = blockIdx.x % splits, col0 = blockIdx.x / splits * kCols, h0 = blockIdx.y * kHG, r = row0 + blockIdx.z;
+  const int pos = row_pos(rows, r), lo = first_key(pos, a.window), n = pos - lo + 1;
+  const int L = (n + splits - 1) / splits, k0 = min(n, split * L), k1 = min(n, k0 + L);
+  const TC* cache = static_cast<const TC*>(a.cache) + ((int64_t)row_seq(rows, r) * a.capacity + lo) * a.width;
+  const float* q = a.qlat + ((int64_t)blockIdx.z * a.heads + h0) * a.width;
+  for (int i = tid; i < kHG * a.width; i += kThreads) qs[i] = h0 + i / a.width < a.heads ? q[i] : 0.0f;
+  if (tid < kHG) {
+    m_run[tid] = -INFINITY;
+    l_run[tid] = 0.0f;
+  }
+  const int col = col0 + 4 * tid;
+  const bool mine = col < a.rank_pad;
+  float acc[kHG][4] = {};
+  for (int t0 = k0; t0 < k1; t0 += kKeys) {
+    const int nt = min(kKeys, k1 - t0);
+    __syncthreads();
+    // scores: four keys of a warp at a time, lanes across the row
+    for (int kb = 4 * warp; kb < nt; kb += 4 * (kThreads / 32)) {
+      const TC* kp[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) kp[u] = cache + (int64_t)(t0 + min(kb + u, nt - 1)) * a.width;
+      float s[4 * kHG] = {};
+      for (int c = 8 * lane; c < a.width; c += 256) {
+        float kf[4][8];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) load8(kp[u] + c, kf[u]);
+#pragma unroll
+        for (int h = 0; h < kHG; ++h) {
+          float qf[8];
+          load8(qs + h * a.width + c, qf);
+#pragma unroll
+          for (int u = 0; u < 4; ++u)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s[4 * h + u] = fmaf(qf[e], kf[u][e], s[4 * h + u]);
+        }
+      }
+      const float sum = transpose_sum(s);
+      if (kb + (lane & 3) < nt) p[(lane >> 2) * kKeys + kb + (lane & 3)] = sum * a.scale;
+    }
+    __syncthreads();
+    for (int h = warp; h < kHG; h += kThreads / 32) {
+      const float s0 = lane < nt ? p[h * kKeys + lane] : -INFINITY, s1 = lane + 32 < nt ? p[h * kKeys + lane + 32] : -INFINITY;
+      float m = fmaxf(s0, s1);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      const float before = m_run[h];
+      m = fmaxf(m, before);
+      const float w0 = expf(s0 - m), w1 = expf(s1 - m);
+      p[h * kKeys + lane] = w0;
+      p[h * kKeys + lane + 32] = w1;
+      const float l = warp_sum(w0 + w1), f = expf(before - m);
+      if (lane == 0) {
+        m_run[h] = m;
+        l_run[h] = l_run[h] * f + l;
+        fix[h] = f;
+      }
+    }
+    __syncthreads();
+    if (mine) {
+#pragma unroll
+      for (int h = 0; h < kHG; ++h)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[h][e] *= fix[h];
+      for (int k = 0; k < nt; k += 4) {
+        float v[4][4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) load4(cache + (int64_t)(t0 + min(k + u, nt - 1)) * a.width + col, v[u]);   // weights past nt are 0
+#pragma unroll
+        for (int h = 0; h < kHG; ++h) {
+          const float4 w = *reinterpret_cast<const float4*>(p + h * kKeys + k);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[h][e] = fmaf(w.w, v[3][e], fmaf(w.z, v[2][e], fmaf(w.y, v[1][e], fmaf(w.x, v[0][e], acc[h][e]))));
+        }
+      }
+    }
+  }
+  __syncthreads();
+  if (mine)
+#pragma unroll
+    for (int h = 0; h < kHG; ++h)
+      if (h0 + h < a.heads)
+        *reinterpret_cast<float4*>(a.part + (((int64_t)blockIdx.z * splits + split) * a.heads + h0 + h) * a.rank_pad + col) =
+            make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
+  if (col0 == 0 && tid < kHG && h0 + tid < a.heads)
+    reinterpret_cast<float2*>(a.stats)[((int64_t)blockIdx.z * splits + split) * a.heads + h0 + tid] = make_float2(m_run[tid], l_run[tid]);
+}
+
+// grid (value tiles, heads, rows)
+template <class TP, class TO>
+__global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a, const Rows rows, int row0, int splits, TO* __restrict__ out, int64_t ldo) {
+  extern __shared__ __align__(16) float o[];    // [rank_pad]
+  __shared__ float weight[kMaxSplits];
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, r = row0 + blockIdx.z;
+  if (warp == 0) {
+    const float2 s = lane < splits ? reinterpret_cast<const float2*>(a.stats)[((int64_t)blockIdx.z * splits + lane) * a.heads + h] : make_float2(-INFINITY, 0.0f);
+    float m = s.x;
+#pragma unroll
+    for (int k = 16; k > 0; k >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, k));
+    const float f = s.x > -INFINITY ? expf(s.x - m) : 0.0f;
+    weight[lane] = f / warp_sum(f * s.y);
+  }
+  __syncthreads();
+  const float* part = a.part + ((int64_t)blockIdx.z * splits * a.heads + h) * a.rank_pad;
+  for (int c = 4 * tid; c < a.rank_pad; c += 4 * kThreads) {
+    float4 t = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int s = 0; s < splits; ++s) {
+      const float w = weight[s];
+      if (w == 0.0f) continue;
+      const float4 v = *reinterpret_cast<const float4*>(part + (int64_t)s * a.heads * a.rank_pad + c);
+      t.x = fmaf(w, v.x, t.x);
+      t.y = fmaf(w, v.y, t.y);
+      t.z = fmaf(w, v.z, t.z);
+      t.w = fmaf(w, v.w, t.w);
+    }
+    *reinterpret_cast<float4*>(o + c) = t;
+  }
+  __syncthreads();
+  const TP* gate = a.gate_at ? static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp + a.gate_at + h * a.vdim : nullptr;
+  const int e0 = blockIdx.x * kOutTile, e1 = min(a.vdim, e0 + kOutTile);
+  for (int e = e0 + warp; e < e1; e += kThreads / 32) {
+    const __nv_bfloat16* w = a.up.w + ((int64_t)a.heads * a.dim + (int64_t)h * a.vdim + e) * a.up.ld;
+    float s = 0.0f;
+    for (int c = 8 * lane; c < a.rank_pad; c += 256) {
+      float wf[8], of[8];
+      load8(w + c, wf);
+      load8(o + c, of);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s = fmaf(wf[i], of[i], s);
+    }
+    s = warp_sum(s);
+    if (lane == 0) {
+      if (gate) s *= sigmoidf_(from(gate[e]));
+      out[(int64_t)r * ldo + h * a.vdim + e] = to<TO>(s);
+    }
+  }
+}
+
+}  // namespace
+
+template <class TC, class TP, class TO>
+cudaError_t launch_latent_rows(const LatentArgs& a, const Rows& rows, TO* out, int64_t ldo, int sm_count, bool pdl, cudaStream_t st, int* launches) {
+  const int groups = (a.heads + kHG - 1) / kHG, blocks = (a.rank_pad + kCols - 1) / kCols;
+  // about one tile of keys per range at least, two blocks per SM at most
+  int splits = 1;
+  if (rows.n <= kLatentRows) {
+    splits = (a.max_visible + kKeys - 1) / kKeys;
+    const int fill = (2 * sm_count + groups * blocks - 1) / (groups * blocks);
+    splits = splits > fill ? fill : splits;
+    splits = splits > kMaxSplits ? kMaxSplits : splits;
+  }
+  const size_t s_in = 4 * ((size_t)a.dim + kThreads / 32 * kSlice), s_attn = 4 * (size_t)kHG * (a.width + kKeys), s_out = 4 * (size_t)a.rank_pad;
+  if (s_in > 48 * 1024 || s_attn > 200 * 1024 || s_out > 200 * 1024) return cudaErrorInvalidValue;
+  cudaError_t e = cudaSuccess;
+  if (s_attn > 40 * 1024) e = cudaFuncSetAttribute(latent_attn_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s_attn);
+  if (e == cudaSuccess && s_out > 40 * 1024) e = cudaFuncSetAttribute(latent_out_kernel<TP, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s_out);
+  if (e != cudaSuccess) return e;
+  uint64_t fit = kLatentRows;
+  const uint64_t per_part = (uint64_t)splits * a.heads * a.rank_pad, per_stats = 2ull * splits * a.heads;
+  if (a.part_floats / per_part < fit) fit = a.part_floats / per_part;
+  if (a.stats_floats / per_stats < fit) fit = a.stats_floats / per_stats;
+  if (fit < 1) return cudaErrorInvalidValue;
+  for (int r0 = 0; r0 < rows.n; r0 += (int)fit) {
+    const int n = rows.n - r0 < (int)fit ? rows.n - r0 : (int)fit;
+    e = launch_kernel(latent_in_kernel<TC, TP>, dim3((a.rank_pad + kSlice - 1) / kSlice + 1, a.heads, n), dim3(kThreads), s_in, st, pdl, a, rows, r0);
+    if (e == cudaSuccess) e = launch_kernel(latent_attn_kernel<TC>, dim3(splits * blocks, groups, n), dim3(kThreads), s_attn, st, pdl, a, rows, r0, splits);
+    if (e == cudaSuccess)
+      e = launch_kernel(latent_out_kernel<TP, TO>, dim3((a.vdim + kOutTile - 1) / kOutTile, a.heads, n), dim3(kThreads), s_out, st, pdl, a, rows, r0, splits, out, ldo);
+    if (e != cudaSuccess) return e;
+    *launches += 3;
+  }
+  return cudaSuccess;
+}
+template cudaError_t launch_latent_rows<float, float, float>(const LatentArgs&, const Rows&, float*, int64_t, int, bool, cudaStream_t, int*);
+template cudaError_t launch_latent_rows<__nv_bfloat16, float, float>(const LatentArgs&, const Rows&, float*, int64_t, int, bool, cudaStream_t, int*);
+template cudaError_t launch_latent_rows<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(const LatentArgs&, const Rows&, __nv_bfloat16*, int64_t, int, bool,
+                                                                                     cudaStream_t, int*);
+
+bool latent_prompt_supported(const LatentArgs& a, int rows) {
+  (void)a; (void)rows;
+  return false;
+}
+cudaError_t launch_latent_prompt(const LatentArgs&, const TmaMap&, const Rows&, int, __nv_bfloat16*, int64_t, int*, cudaStream_t, int*) {
+  return cudaErrorInvalidValue;
+}
+
+}  // namespace emelb

@@ -3,6 +3,7 @@
 // rows in full f32.  f32 activations and accumulation in both.
 #include <cstdlib>
 
+#include "act.cuh"
 #include "common.cuh"
 #include "layered.h"
 
@@ -11,9 +12,6 @@ namespace {
 
 constexpr int kVecThreads = 256;
 constexpr int kVecWarps = kVecThreads / 32;
-
-__device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float siluf_(float z) { return z / (1.0f + expf(-z)); }
 
 __device__ __forceinline__ float block_sum(float v, float* scratch) {
   v = warp_sum(v);
@@ -40,29 +38,35 @@ struct SplitVec {
   __device__ __forceinline__ float& at(int i) const { return ((i & 4) ? hi : lo)[(i >> 3) * 4 + (i & 3)]; }
 };
 
-// A warp owns RW rows at a time (for ACT_GLU a gate row and its up row) and walks them in 16-byte chunks, U per lane
-// in flight; the first chunks are requested before the wait for the kernel in front.
-template <int RW, int U>
+// A warp owns RW rows at a time (for a GLU a gate row and its up row) and walks them in 16-byte chunks, U per lane
+// in flight; the first chunks are requested before the wait for the kernel in front.  DUAL: the tasks of a second matrix,
+// which meets the input with the other norm weight, follow those of the first.
+template <int RW, int U, bool DUAL>
 __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArgs a, const VecArgs v) {
   extern __shared__ __align__(16) float xs_raw[];
   __shared__ float scratch[kVecWarps];
   pdl_trigger();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int K = a.w.K, chunks = (K + 7) / 8;
-  const SplitVec xs{xs_raw, xs_raw + 4 * chunks};
-  const bool glu = a.act == ACT_GLU;
-  const int outs = glu ? a.w.M / 2 : a.w.M;
-  const int per_task = glu ? 1 : RW;
-  const int tasks = (outs + per_task - 1) / per_task;
+  const SplitVec xs{xs_raw, xs_raw + 4 * chunks}, xs2{xs_raw + 8 * chunks, xs_raw + 12 * chunks};
+  auto glu_of = [](int act) { return act == ACT_GLU || act == ACT_GLU_GELU; };
+  auto outs_of = [&](const Bf16Matrix& w, int act) { return glu_of(act) ? w.M / 2 : w.M; };
+  auto tasks_of = [&](int outs, int act) { return glu_of(act) ? outs : (outs + RW - 1) / RW; };
+  const int outs1 = outs_of(a.w, a.act), tasks1 = tasks_of(outs1, a.act);
+  const int outs2 = DUAL ? outs_of(v.w2, v.act2) : 0;
+  const int tasks = tasks1 + (DUAL ? tasks_of(outs2, v.act2) : 0);
   const int stride = gridDim.x * kVecWarps;
   int task = blockIdx.x * kVecWarps + warp;
 
-  auto row_of = [&](int t, int r) { return glu ? t + r * outs : min(t * RW + r, outs - 1); };
   uint4 w[RW][U];
   auto load = [&](int t, int c0) {
+    const bool second = DUAL && t >= tasks1;
+    const Bf16Matrix& m = second ? v.w2 : a.w;
+    const int outs = second ? outs2 : outs1, task_at = second ? t - tasks1 : t;
+    const bool glu = glu_of(second ? v.act2 : a.act);
 #pragma unroll
     for (int r = 0; r < RW; ++r) {
-      const uint4* p = reinterpret_cast<const uint4*>(a.w.w + (int64_t)row_of(t, r) * a.w.ld);
+      const uint4* p = reinterpret_cast<const uint4*>(m.w + (int64_t)(glu ? task_at + r * outs : min(task_at * RW + r, outs - 1)) * m.ld);
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int c = c0 + lane + 32 * u;
@@ -74,15 +78,45 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
   pdl_wait();
 
   // ---- the input vector
-  for (int i = K + tid; i < 8 * chunks; i += kVecThreads) xs.at(i) = 0.0f;
+  for (int i = K + tid; i < 8 * chunks; i += kVecThreads) {
+    xs.at(i) = 0.0f;
+    if (DUAL) xs2.at(i) = 0.0f;
+  }
   if (v.pro == PRO_PLAIN) {
     for (int i = tid; i < K; i += kVecThreads) xs.at(i) = v.x[i];
   } else if (v.pro == PRO_EMBED) {
     const __nv_bfloat16* row = v.table + (int64_t)*v.token * v.table_ld;
     for (int i = tid; i < K; i += kVecThreads) {
-      const float x = __bfloat162float(row[i]);
+      const float x = __bfloat162float(row[i]) + (v.step ? v.step[i] : 0.0f);
       xs.at(i) = x;
       if (blockIdx.x == 0) v.x_out[i] = x;
+    }
+  } else if (v.pro == PRO_PRENORM) {
+    const __nv_bfloat16* row = v.table ? v.table + (int64_t)*v.token * v.table_ld : nullptr;
+    float s = 0.0f, ss = 0.0f;
+    for (int i = tid; i < K; i += kVecThreads) {
+      float x = row ? __bfloat162float(row[i]) : v.x[i];
+      if (v.y) x += v.y[i];
+      if (v.step) x += v.step[i];
+      xs.at(i) = x;
+      s += x;
+      ss = fmaf(x, x, ss);
+      if (v.x_out && blockIdx.x == 0) v.x_out[i] = x;
+    }
+    float mean = 0.0f;
+    if (!v.rms) {
+      mean = block_sum(s, scratch) / K;
+      ss = 0.0f;
+      for (int i = tid; i < K; i += kVecThreads) {
+        const float d = xs.at(i) - mean;
+        ss = fmaf(d, d, ss);
+      }
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / K + v.eps);
+    for (int i = tid; i < K; i += kVecThreads) {
+      const float n = (xs.at(i) - mean) * inv;
+      xs.at(i) = n * v.norm_w[i];
+      if (DUAL) xs2.at(i) = n * v.norm2_w[i];
     }
   } else if (v.pro == PRO_RMS_GATE) {
     float ss = 0.0f;
@@ -100,7 +134,7 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
       xs.at(i) = y;
       s += y;
     }
-    const float mean = block_sum(s, scratch) / K;
+    const float mean = v.rms ? 0.0f : block_sum(s, scratch) / K;
     float ss = 0.0f;
     for (int i = tid; i < K; i += kVecThreads) {
       const float d = xs.at(i) - mean;
@@ -109,13 +143,13 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / K + v.eps);
     s = 0.0f;
     for (int i = tid; i < K; i += kVecThreads) {
-      const float x = v.x[i] + (xs.at(i) - mean) * inv * v.norm_w[i];
+      const float x = v.x[i] + (xs.at(i) - mean) * inv * v.norm_w[i] + (v.step ? v.step[i] : 0.0f);
       xs.at(i) = x;
       s += x;
       if (v.x_out && blockIdx.x == 0) v.x_out[i] = x;
     }
     if (v.pro == PRO_RESIDUAL_NORM) {
-      const float mean2 = block_sum(s, scratch) / K;
+      const float mean2 = v.rms ? 0.0f : block_sum(s, scratch) / K;
       ss = 0.0f;
       for (int i = tid; i < K; i += kVecThreads) {
         const float d = xs.at(i) - mean2;
@@ -130,6 +164,8 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
   float best = 0.0f;
   int best_row = -1;
   for (; task < tasks; task += stride) {
+    const bool second = DUAL && task >= tasks1;
+    const SplitVec in = second ? xs2 : xs;
     float acc[RW];
 #pragma unroll
     for (int r = 0; r < RW; ++r) acc[r] = 0.0f;
@@ -138,7 +174,7 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
       for (int u = 0; u < U; ++u) {
         const int c = c0 + lane + 32 * u;
         if (c < chunks) {
-          const float4 xl = *reinterpret_cast<const float4*>(xs.lo + 4 * c), xh = *reinterpret_cast<const float4*>(xs.hi + 4 * c);
+          const float4 xl = *reinterpret_cast<const float4*>(in.lo + 4 * c), xh = *reinterpret_cast<const float4*>(in.hi + 4 * c);
           const float x[8] = {xl.x, xl.y, xl.z, xl.w, xh.x, xh.y, xh.z, xh.w};
 #pragma unroll
           for (int r = 0; r < RW; ++r) {
@@ -157,24 +193,28 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
     }
 #pragma unroll
     for (int r = 0; r < RW; ++r) acc[r] = warp_sum(acc[r]);
-    if (glu) {
+    const int act = second ? v.act2 : a.act, outs = second ? outs2 : outs1, task_at = second ? task - tasks1 : task;
+    const float* bias = second ? v.bias2 : a.bias;
+    float* out = second ? v.out2 : v.out;
+    if (glu_of(act)) {
       if (lane == 0) {
         float g = acc[0], u = acc[RW - 1];
-        if (a.bias) {
-          g += a.bias[task];
-          u += a.bias[task + outs];
+        if (bias) {
+          g += bias[task_at];
+          u += bias[task_at + outs];
         }
-        v.out[task] = siluf_(g) * u;
+        out[task_at] = (act == ACT_GLU ? siluf_(g) : gelu_tanhf_(g)) * u;
       }
     } else {
 #pragma unroll
       for (int r = 0; r < RW; ++r) {
-        const int row = task * RW + r;
+        const int row = task_at * RW + r;
         if (lane == r && row < outs) {
           float y = acc[r];
-          if (a.bias) y += a.bias[row];
-          if (a.act == ACT_SILU_SIGMOID) y = row < a.act_split ? siluf_(y) : sigmoidf_(y);
-          v.out[row] = y;
+          if (bias) y += bias[row];
+          if (act == ACT_SILU_SIGMOID) y = row < a.act_split ? siluf_(y) : sigmoidf_(y);
+          if (act == ACT_SOFTCAP) y = softcapf_(y * a.out_scale, a.softcap);
+          out[row] = y;
           if (best_row < 0 || y > best) {   // rows of a lane ascend
             best = y;
             best_row = row;
@@ -251,6 +291,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearArgs a, con
       float o = acc[i][j];
       if (a.bias) o += a.bias[f];
       if (a.act == ACT_SILU_SIGMOID) o = f < a.act_split ? siluf_(o) : sigmoidf_(o);
+      if (a.act == ACT_SOFTCAP) o = softcapf_(o * a.out_scale, a.softcap);
       y[(int64_t)row * ldy + f] = o;
     }
 }
@@ -258,18 +299,20 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearArgs a, con
 }  // namespace
 
 cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_count, bool pdl, cudaStream_t st, int* parts) {
-  const int chunks = (a.w.K + 7) / 8, smem = 32 * chunks;
-  if (smem > 200 * 1024) return cudaErrorInvalidValue;
-  const bool glu = a.act == ACT_GLU;
-  const int outs = glu ? a.w.M / 2 : a.w.M;
+  const bool dual = v.w2.w != nullptr;
+  const int chunks = (a.w.K + 7) / 8, smem = (dual ? 64 : 32) * chunks;
+  if (smem > 200 * 1024 || (dual && (v.w2.K != a.w.K || v.pro != PRO_PRENORM || v.part_val))) return cudaErrorInvalidValue;
+  auto outs_of = [](const Bf16Matrix& w, int act) { return is_glu(act) ? w.M / 2 : w.M; };
+  const int outs = outs_of(a.w, a.act);
   // two rows per warp unless that leaves SMs without work
-  const bool pair = glu || outs >= sm_count * kVecWarps * 2;
-  auto kern = pair ? linear_vec_kernel<2, 4> : linear_vec_kernel<1, 8>;
+  const bool pair = dual || is_glu(a.act) || outs >= sm_count * kVecWarps * 2;
+  auto kern = dual ? linear_vec_kernel<2, 4, true> : pair ? linear_vec_kernel<2, 4, false> : linear_vec_kernel<1, 8, false>;
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return e;
   }
-  const int tasks = pair && !glu ? (outs + 1) / 2 : outs;
+  auto tasks_of = [&](int n, int act) { return pair && !is_glu(act) ? (n + 1) / 2 : n; };
+  const int tasks = tasks_of(outs, a.act) + (dual ? tasks_of(outs_of(v.w2, v.act2), v.act2) : 0);
   int per_sm = (200 * 1024) / (smem + 1024);
   per_sm = per_sm > 4 ? 4 : per_sm;
   int grid = (tasks + kVecWarps - 1) / kVecWarps;
@@ -279,7 +322,7 @@ cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_coun
 }
 
 cudaError_t launch_linear_f32(const LinearArgs& a, const float* x, int64_t ldx, float* y, int64_t ldy, cudaStream_t st) {
-  if (a.act == ACT_GLU) return cudaErrorInvalidValue;
+  if (is_glu(a.act)) return cudaErrorInvalidValue;
   const dim3 grid((a.w.M + kTile - 1) / kTile, (a.rows + kTile - 1) / kTile);
   linear_f32_kernel<<<grid, 256, 0, st>>>(a, x, ldx, y, ldy);
   return cudaGetLastError();

@@ -1155,13 +1155,23 @@ uint32_t emelb_llama_create(emelb_ctx* c, const emelb_llama_config* cfg, emelb_l
 }
 
 uint32_t emelb_llama_check_layers(const emelb_llama_config* cfg, const emelb_layer_config* layers) {
-  return cfg ? layered_check(*cfg, layers) : EMELB_INVALID_REQUEST;
+  return cfg ? layered_check(*cfg, layered_default_stack(), layers) : EMELB_INVALID_REQUEST;
+}
+
+uint32_t emelb_llama_check_stack(const emelb_llama_config* cfg, const emelb_stack_config* stack, const emelb_layer_config* layers) {
+  return cfg && stack ? layered_check(*cfg, *stack, layers) : EMELB_INVALID_REQUEST;
 }
 
 uint32_t emelb_llama_create_layers(emelb_ctx* c, const emelb_llama_config* cfg, const emelb_layer_config* layers, int32_t float32, emelb_llama** out) {
-  if (!c || !cfg || !out || (float32 != 0 && float32 != 1)) return EMELB_INVALID_REQUEST;
+  const emelb_stack_config stack = layered_default_stack();
+  return emelb_llama_create_stack(c, cfg, &stack, layers, float32, out);
+}
+
+uint32_t emelb_llama_create_stack(emelb_ctx* c, const emelb_llama_config* cfg, const emelb_stack_config* stack, const emelb_layer_config* layers,
+                                  int32_t float32, emelb_llama** out) {
+  if (!c || !cfg || !stack || !out || (float32 != 0 && float32 != 1)) return EMELB_INVALID_REQUEST;
   *out = nullptr;
-  if (layered_check(*cfg, layers) != EMELB_OK) return EMELB_INVALID_REQUEST;
+  if (layered_check(*cfg, *stack, layers) != EMELB_OK) return EMELB_INVALID_REQUEST;
   cudaSetDevice(c->device);
   emelb_llama* s = new (std::nothrow) emelb_llama();
   if (!s) return EMELB_INTERNAL_ERROR;
@@ -1169,7 +1179,7 @@ uint32_t emelb_llama_create_layers(emelb_ctx* c, const emelb_llama_config* cfg, 
   s->cfg = *cfg;
   s->cfg.shard_count = 1;
   s->seq_len.assign(1, 0);
-  s->layered = layered_create(c, s->cfg, layers, float32 == 1);
+  s->layered = layered_create(c, s->cfg, *stack, layers, float32 == 1);
   bool ok = s->layered != nullptr;
   ok = ok && dev_alloc(s, (void**)&s->logits, 4 * (size_t)cfg->n_vocab) && dev_alloc(s, (void**)&s->state, 4 * sizeof(int));
   ok = ok && dev_alloc(s, (void**)&s->tokens_dev, sizeof(int) * (size_t)(cfg->n_ctx + 8));

@@ -1,8 +1,9 @@
-// Row kernels of layered decoders between the products: embedding, residual + layer norm, gated RMS norm, GLU, and the
+// Row kernels of layered decoders between the products: embedding, residual + norm, gated RMS norm, GLU, and the
 // step from an attention layer's projections to its queries and cache rows (short convolution, query / key norm over
 // the whole projection, partial rotation, value norm, store).  f32 arithmetic throughout.
 #include <math.h>
 
+#include "act.cuh"
 #include "common.cuh"
 #include "layered.h"
 
@@ -37,22 +38,26 @@ __device__ __forceinline__ void store_pair(float* p, float a, float b) { *reinte
 __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
 
 template <class T>
-__global__ void embed_rows_bf16_kernel(const __nv_bfloat16* __restrict__ table, int64_t ld, const int* __restrict__ tokens, int width,
-                                       float* x, T* xb, int64_t ldb) {
+__global__ void embed_rows_bf16_kernel(const __nv_bfloat16* __restrict__ table, int64_t ld, const int* __restrict__ tokens,
+                                       const float* __restrict__ step, int width, float* x, T* xb, int64_t ldb) {
   const int r = blockIdx.x;
   const __nv_bfloat16* row = table + (int64_t)tokens[r] * ld;
   for (int i = threadIdx.x; i < width; i += kThreads) {
-    const float v = __bfloat162float(row[i]);
+    const float v = __bfloat162float(row[i]) + (step ? step[i] : 0.0f);
     x[(int64_t)r * width + i] = v;
     xb[(int64_t)r * ldb + i] = to<T>(v);
   }
 }
 
-// layer norm of the vector in shared memory: mean and 1 / sqrt(variance + eps), squared deviations in a second pass
-__device__ __forceinline__ void norm_stats(const float* s, int n, float eps, float* scratch, float& mean, float& inv) {
+// norm of the vector in shared memory: mean (0 for an RMS norm) and 1 / sqrt(mean square of the deviations + eps),
+// the deviations in a second pass
+__device__ __forceinline__ void norm_stats(const float* s, int n, int rms, float eps, float* scratch, float& mean, float& inv) {
   float t = 0.0f;
-  for (int i = threadIdx.x; i < n; i += kThreads) t += s[i];
-  mean = block_sum(t, scratch) / n;
+  mean = 0.0f;
+  if (!rms) {
+    for (int i = threadIdx.x; i < n; i += kThreads) t += s[i];
+    mean = block_sum(t, scratch) / n;
+  }
   t = 0.0f;
   for (int i = threadIdx.x; i < n; i += kThreads) {
     const float d = s[i] - mean;
@@ -62,32 +67,57 @@ __device__ __forceinline__ void norm_stats(const float* s, int n, float eps, flo
 }
 
 template <class T>
-__global__ void residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float eps, int width,
-                                     T* __restrict__ xb, int64_t ldb, float* keep) {
+__global__ void residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, int rms, float eps,
+                                     int width, T* __restrict__ xb, int64_t ldb, float* keep, const float* __restrict__ step) {
   extern __shared__ float s[];
   __shared__ float scratch[kWarps];
   const int64_t r = blockIdx.x;
   for (int i = threadIdx.x; i < width; i += kThreads) s[i] = y[r * width + i];
   float mean, inv;
-  norm_stats(s, width, eps, scratch, mean, inv);
+  norm_stats(s, width, rms, eps, scratch, mean, inv);
   for (int i = threadIdx.x; i < width; i += kThreads) {
-    const float v = x[r * width + i] + (s[i] - mean) * inv * w[i];
+    float v = x[r * width + i] + (s[i] - mean) * inv * w[i];
+    if (keep) keep[r * width + i] = v;
+    if (step) v += step[i];
     x[r * width + i] = v;
     xb[r * ldb + i] = to<T>(v);
-    if (keep) keep[r * width + i] = v;
   }
 }
 
 template <class T>
-__global__ void norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ index, const float* __restrict__ w, float eps, int width,
+__global__ void norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ index, const float* __restrict__ w, int rms, float eps, int width,
                                  T* __restrict__ out, int64_t ldo) {
   extern __shared__ float s[];
   __shared__ float scratch[kWarps];
   const int64_t r = blockIdx.x, src = index ? index[r] : r;
   for (int i = threadIdx.x; i < width; i += kThreads) s[i] = x[src * width + i];
   float mean, inv;
-  norm_stats(s, width, eps, scratch, mean, inv);
+  norm_stats(s, width, rms, eps, scratch, mean, inv);
   for (int i = threadIdx.x; i < width; i += kThreads) out[r * ldo + i] = to<T>((s[i] - mean) * inv * w[i]);
+}
+
+template <class T>
+__global__ void prenorm_rows_kernel(const PrenormArgs a) {
+  extern __shared__ float s[];
+  __shared__ float scratch[kWarps];
+  const int64_t r = blockIdx.x;
+  const __nv_bfloat16* row = a.table ? a.table + (int64_t)a.tokens[r] * a.table_ld : nullptr;
+  for (int i = threadIdx.x; i < a.width; i += kThreads) {
+    float v = row ? __bfloat162float(row[i]) : a.x[r * a.width + i];
+    if (a.y) v += a.y[r * a.width + i];
+    if (a.keep) a.keep[r * a.width + i] = v;
+    if (a.step) v += a.step[i];
+    a.x[r * a.width + i] = v;
+    s[i] = v;
+  }
+  if (!a.h1 && !a.h2) return;
+  float mean, inv;
+  norm_stats(s, a.width, a.rms, a.eps, scratch, mean, inv);
+  for (int i = threadIdx.x; i < a.width; i += kThreads) {
+    const float n = (s[i] - mean) * inv;
+    if (a.h1) static_cast<T*>(a.h1)[r * a.ldh + i] = to<T>(n * a.w1[i]);
+    if (a.h2) static_cast<T*>(a.h2)[r * a.ldh + i] = to<T>(n * a.w2[i]);
+  }
 }
 
 template <class T>
@@ -104,12 +134,12 @@ __global__ void rms_gate_kernel(const float* __restrict__ o, const float* __rest
   for (int i = threadIdx.x; i < width; i += kThreads) out[r * ldo + i] = to<T>(o[r * width + i] * inv * w[i] * from(gate[r * ldg + i]));
 }
 
-__global__ void glu_rows_kernel(const float* __restrict__ gu, int ff, float* __restrict__ out, int64_t ldo) {
+__global__ void glu_rows_kernel(const float* __restrict__ gu, int ff, int act, float* __restrict__ out, int64_t ldo) {
   const int64_t r = blockIdx.y;
   const int i = blockIdx.x * kThreads + threadIdx.x;
   if (i >= ff) return;
   const float g = gu[r * 2 * ff + i], u = gu[r * 2 * ff + ff + i];
-  out[r * ldo + i] = g / (1.0f + expf(-g)) * u;
+  out[r * ldo + i] = (act == ACT_GLU_GELU ? gelu_tanhf_(g) : siluf_(g)) * u;
 }
 
 // V = 1 or 4 consecutive channels
@@ -233,14 +263,15 @@ __global__ void conv_state_kernel(const AttnInArgs a, const Rows rows) {
 }  // namespace
 
 template <class T>
-cudaError_t launch_embed_rows_bf16(const __nv_bfloat16* table, int64_t ld, const int* tokens, int rows, int width, float* x, T* xb,
-                                   int64_t ldb, cudaStream_t st) {
-  embed_rows_bf16_kernel<T><<<rows, kThreads, 0, st>>>(table, ld, tokens, width, x, xb, ldb);
+cudaError_t launch_embed_rows_bf16(const __nv_bfloat16* table, int64_t ld, const int* tokens, const float* step, int rows, int width, float* x,
+                                   T* xb, int64_t ldb, cudaStream_t st) {
+  embed_rows_bf16_kernel<T><<<rows, kThreads, 0, st>>>(table, ld, tokens, step, width, x, xb, ldb);
   return cudaGetLastError();
 }
-template cudaError_t launch_embed_rows_bf16<float>(const __nv_bfloat16*, int64_t, const int*, int, int, float*, float*, int64_t, cudaStream_t);
-template cudaError_t launch_embed_rows_bf16<__nv_bfloat16>(const __nv_bfloat16*, int64_t, const int*, int, int, float*, __nv_bfloat16*, int64_t,
-                                                           cudaStream_t);
+template cudaError_t launch_embed_rows_bf16<float>(const __nv_bfloat16*, int64_t, const int*, const float*, int, int, float*, float*, int64_t,
+                                                   cudaStream_t);
+template cudaError_t launch_embed_rows_bf16<__nv_bfloat16>(const __nv_bfloat16*, int64_t, const int*, const float*, int, int, float*, __nv_bfloat16*,
+                                                           int64_t, cudaStream_t);
 
 namespace {
 template <class K>
@@ -250,29 +281,41 @@ cudaError_t allow_smem(K kern, size_t bytes) {
 }  // namespace
 
 template <class T>
-cudaError_t launch_residual_norm(float* x, const float* y, const float* w, float eps, int rows, int width, T* xb, int64_t ldb, float* keep,
-                                 cudaStream_t st) {
+cudaError_t launch_residual_norm(float* x, const float* y, const float* w, int rms, float eps, int rows, int width, T* xb, int64_t ldb, float* keep,
+                                 const float* step, cudaStream_t st) {
   const size_t smem = 4 * (size_t)width;
   const cudaError_t e = allow_smem(residual_norm_kernel<T>, smem);
   if (e != cudaSuccess) return e;
-  residual_norm_kernel<T><<<rows, kThreads, smem, st>>>(x, y, w, eps, width, xb, ldb, keep);
+  residual_norm_kernel<T><<<rows, kThreads, smem, st>>>(x, y, w, rms, eps, width, xb, ldb, keep, step);
   return cudaGetLastError();
 }
-template cudaError_t launch_residual_norm<float>(float*, const float*, const float*, float, int, int, float*, int64_t, float*, cudaStream_t);
-template cudaError_t launch_residual_norm<__nv_bfloat16>(float*, const float*, const float*, float, int, int, __nv_bfloat16*, int64_t, float*,
-                                                         cudaStream_t);
+template cudaError_t launch_residual_norm<float>(float*, const float*, const float*, int, float, int, int, float*, int64_t, float*, const float*,
+                                                 cudaStream_t);
+template cudaError_t launch_residual_norm<__nv_bfloat16>(float*, const float*, const float*, int, float, int, int, __nv_bfloat16*, int64_t, float*,
+                                                         const float*, cudaStream_t);
 
 template <class T>
-cudaError_t launch_norm_rows(const float* x, const int* index, const float* w, float eps, int rows, int width, T* out, int64_t ldo,
+cudaError_t launch_norm_rows(const float* x, const int* index, const float* w, int rms, float eps, int rows, int width, T* out, int64_t ldo,
                              cudaStream_t st) {
   const size_t smem = 4 * (size_t)width;
   const cudaError_t e = allow_smem(norm_rows_kernel<T>, smem);
   if (e != cudaSuccess) return e;
-  norm_rows_kernel<T><<<rows, kThreads, smem, st>>>(x, index, w, eps, width, out, ldo);
+  norm_rows_kernel<T><<<rows, kThreads, smem, st>>>(x, index, w, rms, eps, width, out, ldo);
   return cudaGetLastError();
 }
-template cudaError_t launch_norm_rows<float>(const float*, const int*, const float*, float, int, int, float*, int64_t, cudaStream_t);
-template cudaError_t launch_norm_rows<__nv_bfloat16>(const float*, const int*, const float*, float, int, int, __nv_bfloat16*, int64_t, cudaStream_t);
+template cudaError_t launch_norm_rows<float>(const float*, const int*, const float*, int, float, int, int, float*, int64_t, cudaStream_t);
+template cudaError_t launch_norm_rows<__nv_bfloat16>(const float*, const int*, const float*, int, float, int, int, __nv_bfloat16*, int64_t, cudaStream_t);
+
+template <class T>
+cudaError_t launch_prenorm_rows(const PrenormArgs& a, cudaStream_t st) {
+  const size_t smem = 4 * (size_t)a.width;
+  const cudaError_t e = allow_smem(prenorm_rows_kernel<T>, smem);
+  if (e != cudaSuccess) return e;
+  prenorm_rows_kernel<T><<<a.rows, kThreads, smem, st>>>(a);
+  return cudaGetLastError();
+}
+template cudaError_t launch_prenorm_rows<float>(const PrenormArgs&, cudaStream_t);
+template cudaError_t launch_prenorm_rows<__nv_bfloat16>(const PrenormArgs&, cudaStream_t);
 
 template <class T>
 cudaError_t launch_rms_gate(const float* o, const float* w, const T* gate, int64_t ldg, float eps, int rows, int width, T* out, int64_t ldo,
@@ -284,8 +327,8 @@ template cudaError_t launch_rms_gate<float>(const float*, const float*, const fl
 template cudaError_t launch_rms_gate<__nv_bfloat16>(const float*, const float*, const __nv_bfloat16*, int64_t, float, int, int, __nv_bfloat16*,
                                                     int64_t, cudaStream_t);
 
-cudaError_t launch_glu_rows(const float* gu, int rows, int ff, float* out, int64_t ldo, cudaStream_t st) {
-  glu_rows_kernel<<<dim3((ff + kThreads - 1) / kThreads, rows), kThreads, 0, st>>>(gu, ff, out, ldo);
+cudaError_t launch_glu_rows(const float* gu, int rows, int ff, int act, float* out, int64_t ldo, cudaStream_t st) {
+  glu_rows_kernel<<<dim3((ff + kThreads - 1) / kThreads, rows), kThreads, 0, st>>>(gu, ff, act, out, ldo);
   return cudaGetLastError();
 }
 

@@ -32,6 +32,8 @@ SIGNATURES = {
     "emelb_llama_prefill": [_P, C.POINTER(C.c_int32), C.c_int32, C.c_int32],
     "emelb_llama_check_layers": [C.POINTER(Config), _P],
     "emelb_llama_create_layers": [_P, C.POINTER(Config), _P, C.c_int32, C.POINTER(_P)],
+    "emelb_llama_check_stack": [C.POINTER(Config), _P, _P],
+    "emelb_llama_create_stack": [_P, C.POINTER(Config), _P, _P, C.c_int32, C.POINTER(_P)],
     "emelb_llama_prefill_logits": [_P, C.POINTER(C.c_int32), C.c_int32, C.c_int32, C.POINTER(C.c_int32), C.c_int32, _P],
     "emelb_llama_trace_layers": [_P, _P, C.c_int32],
     "emelb_llama_generate": [_P, C.c_int32, C.c_int32, C.c_int32, C.POINTER(C.c_int32)],

@@ -13,6 +13,11 @@ def _metulix(backend, path, n_ctx, float32):
     return metulix.load(backend, path, n_ctx=n_ctx or 4096, float32=float32)
 
 
+def _sugonex(backend, path, n_ctx, float32):
+    from emel_cpp_b200 import sugonex
+    return sugonex.load(backend, path, n_ctx=n_ctx or 4096, float32=float32)
+
+
 def _llama(backend, path, n_ctx, float32):
     from emel_cpp_b200 import gguf
     if float32:
@@ -21,7 +26,7 @@ def _llama(backend, path, n_ctx, float32):
         return gguf.load_llama(backend, f, n_ctx)
 
 
-ARCHITECTURES = {"Metulix": _metulix, "llama": _llama}
+ARCHITECTURES = {"Metulix": _metulix, "Sugonex": _sugonex, "llama": _llama}
 
 
 def architecture(path: str) -> str:

@@ -83,14 +83,22 @@ enum {
   EMELB_T_MIX_NORM_OUT = 17, /* f32, over the concatenated heads of a linear mixer */
   EMELB_T_FFN_IN = 18,       /* gate|up stacked by rows */
   EMELB_T_FFN_IN_BIAS = 19,  /* f32, gate|up */
-  EMELB_T_FFN_DOWN_BIAS = 20 /* f32 */
+  EMELB_T_FFN_DOWN_BIAS = 20, /* f32 */
+  EMELB_T_MIX_LATENT_NORM = 21, /* f32, kv_rank */
+  EMELB_T_MIX_LATENT_UP = 22,   /* {kv_rank, n_head * (key_dim + value_dim)}: the latent's key rows of every head, then its value rows */
+  EMELB_T_MIX_DECAY_LOG = 23,   /* f32, n_head: log of the delta rule's decay rate */
+  EMELB_T_MIX_STEP_BIAS = 24,   /* f32, n_head: bias inside the decay's softplus */
+  EMELB_T_LAYER_OUT = 25,       /* parallel layers: output projection and feed-forward's down projection side by side,
+                                   {n_head * value_dim rounded up to 8 (zeros there) + n_ff, n_embd} */
+  EMELB_T_LOOP_STEP = 26        /* model level, f32 {n_embd, loop_times}: added to the stream ahead of each pass */
 };
 
 typedef struct emelb_llama emelb_llama;
 
 /* ---- layered sessions: decoders described layer by layer.  Each layer is a sequence mixer and, optionally, a
- * gated feed-forward; both read the residual stream itself and the norm (layer norm, weight only) is applied to what
- * they return: x += norm1(mixer(x)), x += norm2(ff(x)).  Weights are bf16, vectors f32; the residual stream, norms,
+ * gated feed-forward.  How they meet the residual stream is the stack's arrangement (emelb_stack_config): by default
+ * both read the stream itself and the norm (layer norm, weight only) is applied to what they return: x += norm1(mixer(x)),
+ * x += norm2(ff(x)).  Weights are bf16, vectors f32; the residual stream, norms,
  * attention scores and weights, and recurrent state are f32.  A session of this kind works through the same entry
  * points as the block-quantized ones (prefill, decode, generate, the batch calls, sequences), with one difference:
  * its mixers carry state, so a call must continue a sequence at the position where the last one ended, or start it
@@ -100,9 +108,18 @@ enum {
                                 the whole projection, adjacent-pair RoPE on the first rope_dim dimensions, value norm
                                 per head, sliding window that keeps the sequence's first tokens, mixing of the
                                 heads' weights after the softmax; keys and values may be another layer's */
-  EMELB_MIXER_LINEAR = 1     /* linear attention with a fixed decay per head: S = decay S + k v^T, o = S^T q, with silu
+  EMELB_MIXER_LINEAR = 1,    /* linear attention with a fixed decay per head: S = decay S + k v^T, o = S^T q, with silu
                                 on q, k and v; heads RMS-normed together and gated by sigmoid(gate) */
+  EMELB_MIXER_LATENT = 2,    /* softmax attention whose keys and values are projections of one cached latent per token
+                                (kv_rank values, RMS norm) and, with rope_dim > 0, one rotated key part shared by all heads:
+                                head = key_dim unrotated + rope_dim rotated dimensions; sliding window; optional sigmoid gate
+                                on the concatenated heads.  MIX_IN rows: q | gate (out_gate) | latent | rotated key part */
+  EMELB_MIXER_DELTA = 3      /* gated delta rule: short causal convolution and silu on q, k, v; q and k unit vectors per head;
+                                S = g S, u = beta (v - S^T k), S += k u^T, o = S^T q / sqrt(key_dim) with one decay g and one
+                                step size beta per head and token; heads RMS-normed each and gated by silu(gate).  n_head_kv
+                                query / key heads, n_head value heads.  MIX_IN rows: q | k | v | gate | beta | decay */
 };
+enum { EMELB_FF_SILU = 0, EMELB_FF_GELU_TANH = 1 };
 typedef struct emelb_layer_config {
   int32_t mixer;
   int32_t n_head, n_head_kv; /* n_head_kv: attention only */
@@ -119,7 +136,28 @@ typedef struct emelb_layer_config {
   int32_t kv_from;           /* layer whose keys and values are used (-1: this layer's own) */
   int32_t n_ff;              /* 0: no feed-forward */
   const float* decay;        /* linear: n_head factors (read by the create call) */
+  int32_t rope_half;         /* latent: 1 = dimension i turns with i + rope_dim / 2, 0 = with its neighbour */
+  int32_t kv_rank;           /* latent: size of the latent */
+  int32_t out_gate;          /* latent: 1 = heads multiplied by sigmoid(gate) */
+  int32_t ff_act;            /* EMELB_FF_*: activation of the gate */
+  int32_t ff_bias;           /* 1 = biases on gate | up and down */
 } emelb_layer_config;
+
+/* what the layers of a stack have in common */
+enum {
+  EMELB_STACK_POST_NORM = 0, /* x += norm1(mixer(x)); x += norm2(ff(x)) */
+  EMELB_STACK_PARALLEL = 1   /* x += mixer(norm1(x)) + ff(norm2(x)), both of the same x */
+};
+enum { EMELB_NORM_LAYER = 0, EMELB_NORM_RMS = 1 };   /* of the stream; weight only */
+typedef struct emelb_stack_config {
+  int32_t arrangement;
+  int32_t norm;
+  int32_t loop_start, loop_stop, loop_times; /* layers loop_start .. loop_stop - 1 run loop_times times in a row with the same
+                                weights, each pass with its own cache and state; loop_times 0: every layer runs once */
+  int32_t loop_step;         /* 1 = EMELB_T_LOOP_STEP row t is added to the stream ahead of pass t */
+  float logit_scale;         /* logits = logit_scale * output product ... */
+  float logit_softcap;       /* ... then softcap * tanh(logits / softcap); 0: none */
+} emelb_stack_config;
 
 /* pure check of a configuration (no device needed): EMELB_OK or
  * EMELB_INVALID_REQUEST.  Beyond the plain range checks, a sharded layout
@@ -144,6 +182,11 @@ EMELB_API uint32_t emelb_llama_destroy(emelb_llama* s);
 EMELB_API uint32_t emelb_llama_check_layers(const emelb_llama_config* cfg, const emelb_layer_config* layers);
 EMELB_API uint32_t emelb_llama_create_layers(emelb_ctx* ctx, const emelb_llama_config* cfg,
                                              const emelb_layer_config* layers, int32_t float32, emelb_llama** out);
+/* the same with the stack described; emelb_llama_create_layers is post-norm with layer norm, no loop, plain logits */
+EMELB_API uint32_t emelb_llama_check_stack(const emelb_llama_config* cfg, const emelb_stack_config* stack,
+                                           const emelb_layer_config* layers);
+EMELB_API uint32_t emelb_llama_create_stack(emelb_ctx* ctx, const emelb_llama_config* cfg, const emelb_stack_config* stack,
+                                            const emelb_layer_config* layers, int32_t float32, emelb_llama** out);
 
 /* binds one tensor (replaces bind_tensor_rows / make_src_view,
  * src/emel/text/generator/detail.hpp:788-817, 1886-1919): a {K, M} view of
@@ -176,8 +219,8 @@ EMELB_API uint32_t emelb_llama_prefill(emelb_llama* s, const int32_t* tokens, in
 EMELB_API uint32_t emelb_llama_prefill_logits(emelb_llama* s, const int32_t* tokens, int32_t n, int32_t start_pos,
                                               const int32_t* want, int32_t n_want, float* logits_out);
 
-/* layered sessions: the residual stream after every layer for the tokens of the last prefill batch is copied to
- * `out` (device or host, {n_layer, tokens, n_embd} f32, tokens <= max_tokens) by the following prefill calls; null
+/* layered sessions: the residual stream after every layer run (a looped layer counts once per pass) for the tokens of the
+ * last prefill batch is copied to `out` (device or host, {layer runs, tokens, n_embd} f32, tokens <= max_tokens) by the following prefill calls; null
  * turns it off (diagnostics). */
 EMELB_API uint32_t emelb_llama_trace_layers(emelb_llama* s, float* out, int32_t max_tokens);
 
