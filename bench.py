@@ -828,9 +828,41 @@ METULIX_SHAPES = {
 }
 
 
+# the same sizes in Sugonex layers: delta, latent attention with a rotated part, delta, windowed latent attention, twice
+SUGONEX_SHAPES = {
+    "2b": dict(width=2048, ff=8192, heads=16, kv_heads=8, dim=128, rot=64, rank=512, taps=4, vocab=32000, window=1024, layers=8),
+    "8b": dict(width=4096, ff=14336, heads=32, kv_heads=16, dim=128, rot=64, rank=512, taps=4, vocab=32000, window=1024, layers=8),
+}
+
+
+class RandomWeights:
+    """Binds random matrices (N(0, 1/K) in bf16) and constant vectors to a layered session."""
+
+    def __init__(self, be, sess, seed0):
+        self.be, self.sess, self.seed0, self.allocs, self.weight_bytes = be, sess, seed0, [], 0
+        self.const = {}
+
+    def mat(self, layer, role, rows, k, also=()):
+        import emel_cpp_b200 as eb
+        from emel_cpp_b200 import llama as el
+        d = self.be.alloc(2 * rows * k)
+        self.allocs.append(d)
+        assert self.be.synth_fill(d, eb.BF16, rows * k, self.seed0 + len(self.allocs), k ** -0.5, 0)
+        for i, r in [(layer, role), *also]:
+            assert self.sess.bind_matrix_at(i, r, d, rows, k, k), (i, r, self.sess.last_error)
+        if role != el.TOKEN_EMBD or also:
+            self.weight_bytes += 2 * rows * k
+
+    def vec(self, layer, role, n, rows=1, value=1.0):
+        if value not in self.const:
+            self.const[value] = self.be.alloc(4 * 65536)
+            self.allocs.append(self.const[value])
+            assert self.be.to_device(self.const[value], np.full(65536, value, np.float32))
+        assert self.sess.bind_vector_at(layer, role, self.const[value], n, rows), (layer, role)
+
+
 def build_metulix_session(be, sh, n_ctx, seed0=7000):
-    """Random weights (N(0, 1/K) in bf16, norm weights and convolution taps 1) -> (session, weight bytes, allocations)."""
-    import emel_cpp_b200 as eb
+    """Random weights, norm weights and convolution taps 1 -> (session, weight bytes, allocations)."""
     from emel_cpp_b200 import layered as ly
     from emel_cpp_b200 import llama as el
     W, H, G, D, ff = sh["width"], sh["heads"], sh["kv_heads"], sh["dim"], sh["ff"]
@@ -843,23 +875,8 @@ def build_metulix_session(be, sh, n_ctx, seed0=7000):
             layers.append(ly.attention_layer(H, G, D, D, D ** -0.5, conv_taps=3, rope_dim=D, rope_freq_base=10000.0, window=sh["window"],
                                              keep_first=sh["keep"], kv_from=i - 2 if i % 4 == 3 else -1, n_ff=ff))
     sess = ly.Session(be, ly.config(len(layers), W, sh["vocab"], n_ctx, 1e-6), layers)
-    allocs, weight_bytes = [], 0
-    ones = be.alloc(4 * 65536)
-    assert be.to_device(ones, np.ones(65536, np.float32))
-    allocs.append(ones)
-
-    def mat(layer, role, rows, k):
-        nonlocal weight_bytes
-        d = be.alloc(2 * rows * k)
-        allocs.append(d)
-        assert be.synth_fill(d, eb.BF16, rows * k, seed0 + len(allocs), k ** -0.5, 0)
-        assert sess.bind_matrix_at(layer, role, d, rows, k, k), (layer, role, sess.last_error)
-        if role != el.TOKEN_EMBD:
-            weight_bytes += 2 * rows * k
-
-    def vec(layer, role, n, rows=1):
-        assert sess.bind_vector_at(layer, role, ones, n, rows), (layer, role)
-
+    r = RandomWeights(be, sess, seed0)
+    mat, vec = r.mat, r.vec
     mat(-1, el.TOKEN_EMBD, sh["vocab"], W)
     mat(-1, el.OUTPUT, sh["vocab"], W)
     vec(-1, el.OUTPUT_NORM, W)
@@ -875,7 +892,7 @@ def build_metulix_session(be, sh, n_ctx, seed0=7000):
             if l.kv_from < 0:
                 vec(i, ly.MIX_NORM_K, G * D)
             talk = be.alloc(4 * H * H)
-            allocs.append(talk)
+            r.allocs.append(talk)
             assert be.to_device(talk, (np.eye(H) + 0.1 * np.random.default_rng(i).standard_normal((H, H))).astype(np.float32))
             assert sess.bind_vector_at(i, ly.MIX_HEADS, talk, H, H)
         mat(i, ly.FFN_IN, 2 * ff, W)
@@ -884,15 +901,55 @@ def build_metulix_session(be, sh, n_ctx, seed0=7000):
         vec(i, ly.FFN_DOWN_BIAS, W)
         vec(i, el.FFN_NORM, W)
     assert be.sync()
-    return sess, weight_bytes, allocs
+    return sess, r.weight_bytes, r.allocs
 
 
-def run_metulix(args):
-    """--workload metulix: prompt and decode throughput of layered decoders at the sizes of METULIX_SHAPES, each beside a Llama
-    session of equal width, feed-forward, heads and layer count.  A step = one decoded token."""
+def build_sugonex_session(be, sh, n_ctx, seed0=7000):
+    """Random weights, norm weights and convolution taps 1, decay logs -3 -> (session, weight bytes, allocations)."""
+    from emel_cpp_b200 import layered as ly
+    from emel_cpp_b200 import llama as el
+    W, H, D, R, ff = sh["width"], sh["heads"], sh["dim"], sh["rank"], dict(n_ff=sh["ff"], ff_act=ly.FF_GELU_TANH)
+    layers = []
+    for i in range(sh["layers"]):
+        if i % 2 == 0:
+            layers.append(ly.delta_layer(H, sh["kv_heads"], D, D, sh["taps"], **ff))
+        elif i % 4 == 1:
+            layers.append(ly.latent_layer(H, D, D, R, (D + sh["rot"]) ** -0.5, rope_dim=sh["rot"], out_gate=True, **ff))
+        else:
+            layers.append(ly.latent_layer(H, D, D, R, D ** -0.5, window=sh["window"], **ff))
+    st = ly.stack(ly.STACK_PARALLEL, ly.NORM_RMS, loop=(0, 2, sh.get("times", 1)), loop_step=True, logit_scale=0.5, logit_softcap=30.0)
+    sess = ly.Session(be, ly.config(len(layers), W, sh["vocab"], n_ctx, 1e-6), layers, st=st)
+    r = RandomWeights(be, sess, seed0)
+    r.mat(-1, el.TOKEN_EMBD, sh["vocab"], W, also=[(-1, el.OUTPUT)])
+    r.vec(-1, el.OUTPUT_NORM, W)
+    r.vec(-1, ly.LOOP_STEP, W, st.loop_times, value=0.0)
+    for i, l in enumerate(layers):
+        r.mat(i, ly.MIX_IN, ly.in_rows(l), W)
+        if l.mixer == ly.MIXER_DELTA:
+            r.vec(i, ly.MIX_CONV, sh["taps"], 2 * l.n_head_kv * D + H * D)
+            r.vec(i, ly.MIX_DECAY_LOG, H, value=-3.0)
+            r.vec(i, ly.MIX_STEP_BIAS, H)
+            r.vec(i, ly.MIX_NORM_OUT, D)
+        else:
+            r.vec(i, ly.MIX_LATENT_NORM, R)
+            r.mat(i, ly.MIX_LATENT_UP, H * 2 * D, R)
+        r.mat(i, ly.FFN_IN, 2 * sh["ff"], W)
+        r.mat(i, ly.LAYER_OUT, W, H * D + sh["ff"])
+        r.vec(i, el.ATTN_NORM, W)
+        r.vec(i, el.FFN_NORM, W)
+    assert be.sync()
+    return sess, r.weight_bytes, r.allocs
+
+
+def run_layered(args):
+    """--workload metulix / sugonex: prompt and decode throughput of layered decoders at the sizes of METULIX_SHAPES /
+    SUGONEX_SHAPES, each beside another model of equal width, feed-forward, heads and layer count: Metulix beside a Llama session,
+    Sugonex beside Metulix.  A step = one decoded token."""
     import torch
     import emel_cpp_b200 as eb
 
+    sugonex = args.workload == "sugonex"
+    sizes = args.sizes or ("2b,8b" if sugonex else "2b,8b,8b-full")
     rank, world, local = dist_setup(args.gpus)
     torch.cuda.set_device(local)
     dev = torch.device("cuda", local)
@@ -934,16 +991,25 @@ def run_metulix(args):
                 "weight_frac_of_hbm": round(weight_bytes / (ms / steps * 1e-3) / 1e9 / peaks["hbm_gbs"], 3)}, \
             (d1["d2h_bytes"] - d0["d2h_bytes"]) // steps
 
+    def layered(build, sh):
+        sess, wb, allocs = build(be, sh, n_ctx)
+        res, d2h = measure(sess, wb, sh["vocab"])
+        sess.close()
+        for d in allocs:
+            be.free(d)
+        return res, d2h
+
     n_ctx = ((prompt_len + warmup + 2 * steps + 63) // 64) * 64
     out, d2h = {}, 0
     with ClockSampler(local) as clk:
-        for name in args.sizes.split(","):
+        for name in sizes.split(","):
+            if sugonex:
+                res, d2h = layered(build_sugonex_session, SUGONEX_SHAPES[name])
+                other, _ = layered(build_metulix_session, METULIX_SHAPES[name])
+                out[name] = {"sugonex": res, "metulix": other}
+                continue
             sh = METULIX_SHAPES[name]
-            sess, wb, allocs = build_metulix_session(be, sh, n_ctx)
-            res, d2h = measure(sess, wb, sh["vocab"])
-            sess.close()
-            for d in allocs:
-                be.free(d)
+            res, d2h = layered(build_metulix_session, sh)
             lsh = dict(n_layer=sh["layers"], n_embd=sh["width"], n_head=sh["heads"], n_head_kv=sh["kv_heads"], head_dim=sh["dim"], n_ff=sh["ff"],
                        n_vocab=sh["vocab"])
             sess, info = build_decode_session(be, lsh, eb.Q4_K, n_ctx, 0, 1)
@@ -951,13 +1017,13 @@ def run_metulix(args):
             release_decode_session(be, sess, info, 1)
             out[name] = {"metulix": res, "llama_q4_k": other}
     clocks = clk.summary()
-    head = out[args.sizes.split(",")[0]]["metulix"]
+    head = out[sizes.split(",")[0]][args.workload]
     print(json.dumps({
         "metric": "decode tok/s", "value": head["decode_tok_s"], "unit": "tok/s", "n_gpus": world, "steps": steps, "warmup": warmup,
         "ms_per_step": head["ms_per_token"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16 operands and KV, f32 accumulation, residual stream and state", "data": "synthetic",
-        "config": {"workload": "metulix layers beside Llama layers of equal size", "prompt_tokens": prompt_len, "sizes": args.sizes,
-                   "l2_policy": "inputs larger than L2: the weights of a token or prompt batch"},
+        "config": {"workload": f"{args.workload} layers beside {'Metulix' if sugonex else 'Llama'} layers of equal size", "prompt_tokens": prompt_len,
+                   "sizes": sizes, "l2_policy": "inputs larger than L2: the weights of a token or prompt batch"},
         "sizes": out, "e2e": {"value": head["decode_e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 8, "d2h_bytes_per_step": d2h},
         "gpu_launches": head["launches_per_token"] * steps, "peak_source": f"of {peak_kind}", "clocks": clocks}), flush=True)
 
@@ -1539,7 +1605,7 @@ def main():
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "decode_70b", "gemv_q4_k", "gemv_q8_0", "prefill_q4_k", "load_gguf", "metulix"])
+    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "decode_70b", "gemv_q4_k", "gemv_q8_0", "prefill_q4_k", "load_gguf", "metulix", "sugonex"])
     ap.add_argument("--layers", type=int, default=16, help="load_gguf: layers in the synthetic file (122.7 MB each)")
     ap.add_argument("--prompt", type=int, default=None, help="prompt length override for the decode workloads")
     ap.add_argument("--ncols", type=int, default=1)
@@ -1559,7 +1625,7 @@ def main():
     ap.add_argument("--one-kernel", action="store_true",
                     help="decode workloads: run the headline through the one-kernel step (every layer of a token in one "
                          "persistent kernel) instead of the launch chain")
-    ap.add_argument("--sizes", default="2b,8b,8b-full", help="metulix: which of METULIX_SHAPES, with commas between them")
+    ap.add_argument("--sizes", default="", help="metulix, sugonex: which of METULIX_SHAPES / SUGONEX_SHAPES, with commas between them")
     ap.add_argument("--mix", action="store_true",
                     help="decode workloads: attn_v and ffn_down of every other layer as Q6_K instead of Q4_K")
     args = ap.parse_args()
@@ -1567,11 +1633,11 @@ def main():
     MIX_Q6_K = args.mix
     args.warmup = max(3, args.warmup)
     decode = args.workload.startswith("decode")
-    if args.workload == "metulix":
+    if args.workload in ("metulix", "sugonex"):
         if args.impl == "reference":
             print(json.dumps({"impl": "reference", "unavailable": "the reference has no layered decoder of this design"}), flush=True)
         else:
-            run_metulix(args)
+            run_layered(args)
     elif args.workload == "prefill_q4_k":
         (run_reference_prefill if args.impl == "reference" else run_prefill)(args)
     elif args.workload == "load_gguf":

@@ -5,6 +5,10 @@
 //   in     latent norm, rotation, cache row; the query against the key rows of its head: q . (U c) = (U^T q) . c
 //   attn   per key range and eight heads: scores, online softmax, weighted latents
 //   out    ranges merged, value rows of the head times the weighted latent, output gate
+//
+// Prompts form keys and values of the visible positions once (one product with the stacked key and value rows) and run an
+// online-softmax kernel on the tensor cores (mma.sync bf16), 128 queries of a head per block.  Scores and weights are f32;
+// the weights meet the values as two bf16 operands, high part and remainder.
 #include <math.h>
 
 #include "act.cuh"
@@ -82,6 +86,23 @@ __device__ void store_latent(const LatentArgs& a, int r, int pos, int seq) {
     row[a.rank_pad + j] = to<TC>(k[j] * c + k[i] * s);
   }
   for (int i = a.rank_pad + a.rot + threadIdx.x; i < a.width; i += kThreads) row[i] = to<TC>(0.0f);
+}
+
+// grid (rows): cache row, and the row's queries rotated in place
+__global__ void __launch_bounds__(kThreads) latent_store_kernel(const LatentArgs a, const Rows rows) {
+  const int r = blockIdx.x, pos = row_pos(rows, r), pairs = a.rot / 2;
+  store_latent<__nv_bfloat16>(a, r, pos, row_seq(rows, r));
+  __nv_bfloat16* q = static_cast<__nv_bfloat16*>(a.proj) + (int64_t)r * a.ldp + a.dim;
+  for (int x = threadIdx.x; x < a.heads * pairs; x += kThreads) {
+    const int h = x / pairs, p = x - h * pairs;
+    int i, j;
+    pair_of(p, a.rot, a.rope_half, i, j);
+    const float c = a.rope_cos[(int64_t)pos * pairs + p], s = a.rope_sin[(int64_t)pos * pairs + p];
+    __nv_bfloat16* head = q + h * (a.dim + a.rot);
+    const float u = from(head[i]), v = from(head[j]);
+    head[i] = to<__nv_bfloat16>(u * c - v * s);
+    head[j] = to<__nv_bfloat16>(v * c + u * s);
+  }
 }
 
 // grid (column slices + 1, heads, rows): slices of U^T q of one head; the last slice rotates the head's query and, for
@@ -338,12 +359,202 @@ template cudaError_t launch_latent_rows<__nv_bfloat16, float, float>(const Laten
 template cudaError_t launch_latent_rows<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(const LatentArgs&, const Rows&, __nv_bfloat16*, int64_t, int, bool,
                                                                                      cudaStream_t, int*);
 
-bool latent_prompt_supported(const LatentArgs& a, int rows) {
-  (void)a; (void)rows;
-  return false;
+// ---- prompts
+namespace {
+
+constexpr int kQT = 128, kKT = 64, kPromptThreads = 256;
+constexpr int kPromptMinRows = 9;   // fewer rows go through the latents: forming every visible key costs more
+
+struct PromptShape {
+  int qrow, vrow;          // elements between rows of the query / key and value tiles
+  int smem;
+};
+PromptShape prompt_shape(const LatentArgs& a) {
+  PromptShape s;
+  s.qrow = (a.dim + a.rot + 15) / 16 * 16 + 8;
+  s.vrow = (a.vdim + 15) / 16 * 16 + 8;
+  s.smem = 2 * (kQT * s.qrow + 2 * kKT * (s.qrow + s.vrow));
+  return s;
 }
-cudaError_t launch_latent_prompt(const LatentArgs&, const TmaMap&, const Rows&, int, __nv_bfloat16*, int64_t, int*, cudaStream_t, int*) {
-  return cudaErrorInvalidValue;
+
+// grid (query tiles, heads).  NV: 8-column tiles of the values (vdim <= 8 NV).  key0: position of the first row of a.kv
+template <int NV>
+__global__ void __launch_bounds__(kPromptThreads) latent_prompt_kernel(const LatentArgs a, const Rows rows, const int key0, const PromptShape shape,
+                                                                       __nv_bfloat16* __restrict__ out, int64_t ldo) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int QR = shape.qrow, VR = shape.vrow, D = a.dim + a.rot;
+  __nv_bfloat16* qt = reinterpret_cast<__nv_bfloat16*>(raw);   // [kQT][QR]
+  __nv_bfloat16* kt = qt + kQT * QR;                           // [2][kKT][QR]
+  __nv_bfloat16* vt = kt + 2 * kKT * QR;                       // [2][kKT][VR]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int i0 = (gridDim.x - 1 - blockIdx.x) * kQT, h = blockIdx.y;   // tiles with the most keys first
+  const int pos0 = rows.pos[0], last = min(rows.n, i0 + kQT) - 1;
+  const int k_begin = first_key(pos0 + i0, a.window), k_end = pos0 + last + 1;
+  const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.proj) + (int64_t)i0 * a.ldp + h * D;
+  const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(a.cache) + (int64_t)rows.seq0 * a.capacity * a.width + a.rank_pad;
+  const __nv_bfloat16 *kb = a.kv + h * a.dim, *vb = a.kv + a.heads * a.dim + h * a.vdim;
+  const int kc = (QR - 8) / 8, vc = (VR - 8) / 8, dc = a.dim / 8, xc = D / 8, vlive = a.vdim / 8;
+  for (int i = tid; i < kQT * kc; i += kPromptThreads) {
+    const int r = i / kc, c = i - r * kc;
+    const bool live = i0 + r < rows.n && c < xc;
+    cp16_zfill(qt + r * QR + 8 * c, live ? q + (int64_t)r * a.ldp + 8 * c : q, live);
+  }
+  auto issue = [&](int key, int buf) {
+    for (int i = tid; i < kKT * kc; i += kPromptThreads) {
+      const int r = i / kc, c = i - r * kc;
+      const bool live = key + r < k_end && c < xc;
+      const __nv_bfloat16* p = c < dc ? kb + (int64_t)(key + r - key0) * a.kv_ld + 8 * c : cache + (int64_t)(key + r) * a.width + 8 * (c - dc);
+      cp16_zfill(kt + (buf * kKT + r) * QR + 8 * c, live ? p : a.kv, live);
+    }
+    for (int i = tid; i < kKT * vc; i += kPromptThreads) {
+      const int r = i / vc, c = i - r * vc;
+      const bool live = key + r < k_end && c < vlive;
+      cp16_zfill(vt + (buf * kKT + r) * VR + 8 * c, live ? vb + (int64_t)(key + r - key0) * a.kv_ld + 8 * c : a.kv, live);
+    }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  issue(k_begin, 0);
+
+  float o[NV][4] = {};
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+  const float scale = a.scale * 1.4426950408889634f;   // weights as powers of two
+  const int row0 = i0 + 16 * warp, p_lo = pos0 + row0;   // this warp's first query
+  int buf = 0;
+  for (int key = k_begin; key < k_end; key += kKT, buf ^= 1) {
+    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    __syncthreads();   // the tile has landed, the other buffer is free
+    if (key + kKT < k_end) issue(key + kKT, buf ^ 1);
+    // nothing of the tile is visible to the warp's rows
+    if (row0 >= rows.n || key > p_lo + 15 || key + kKT <= first_key(p_lo, a.window)) continue;
+    const __nv_bfloat16 *kk = kt + buf * kKT * QR, *vv = vt + buf * kKT * VR;
+    float s[kKT / 8][4] = {};
+#pragma unroll 4
+    for (int d = 0; d < QR - 8; d += 16) {
+      uint32_t qa[4];
+      ldsm(qa, qt + (16 * warp + (lane & 15)) * QR + d + (lane >> 4) * 8);
+#pragma unroll
+      for (int nt = 0; nt < kKT / 16; ++nt) {
+        uint32_t b[4];
+        ldsm(b, kk + (16 * nt + (lane & 7) + (lane >> 4) * 8) * QR + d + ((lane >> 3) & 1) * 8);
+        mma_bf16_16816(s[2 * nt], qa, b[0], b[1]);
+        mma_bf16_16816(s[2 * nt + 1], qa, b[2], b[3]);
+      }
+    }
+    const bool inside = key + kKT - 1 <= p_lo && key >= first_key(p_lo + 15, a.window);
+    float fix[2];
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int pos = p_lo + g + 8 * half, lo = first_key(pos, a.window);
+      float mx = m[half];
+#pragma unroll
+      for (int nt = 0; nt < kKT / 8; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float& x = s[nt][2 * half + e];
+          const int k = key + 8 * nt + 2 * t + e;
+          x = inside || (k <= pos && k >= lo) ? x * scale : -INFINITY;
+          mx = fmaxf(mx, x);
+        }
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));   // the four lanes of a row
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      const float base = mx == -INFINITY ? 0.0f : mx;
+      fix[half] = exp2f(m[half] - base);
+      m[half] = mx;
+      float sum = 0.0f;
+#pragma unroll
+      for (int nt = 0; nt < kKT / 8; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float& x = s[nt][2 * half + e];
+          x = exp2f(x - base);
+          sum += x;
+        }
+      l[half] = l[half] * fix[half] + sum;   // this lane's columns
+    }
+#pragma unroll
+    for (int nv = 0; nv < NV; ++nv)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[nv][e] *= fix[e >> 1];
+#pragma unroll
+    for (int k16 = 0; k16 < kKT / 16; ++k16) {
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) split2(s[2 * k16 + part][2 * half], s[2 * k16 + part][2 * half + 1], hi[2 * part + half], lo[2 * part + half]);
+#pragma unroll
+      for (int np = 0; np < NV / 2; ++np) {
+        if (16 * np >= a.vdim) break;
+        uint32_t b[4];
+        ldsm_trans(b, vv + (16 * k16 + (lane & 15)) * VR + 16 * np + (lane >> 4) * 8);
+        mma_bf16_16816(o[2 * np], hi, b[0], b[1]);
+        mma_bf16_16816(o[2 * np + 1], hi, b[2], b[3]);
+        mma_bf16_16816(o[2 * np], lo, b[0], b[1]);
+        mma_bf16_16816(o[2 * np + 1], lo, b[2], b[3]);
+      }
+    }
+  }
+  const __nv_bfloat16* gate = a.gate_at ? static_cast<const __nv_bfloat16*>(a.proj) + a.gate_at + h * a.vdim : nullptr;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    float sum = l[half];
+    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+    const int r = row0 + g + 8 * half;
+    if (r >= rows.n) continue;
+    const float inv = 1.0f / sum;
+    __nv_bfloat16* dst = out + (int64_t)r * ldo + h * a.vdim;
+#pragma unroll
+    for (int nv = 0; nv < NV; ++nv) {
+      const int c = 8 * nv + 2 * t;
+      if (c >= a.vdim) continue;
+      float x = o[nv][2 * half] * inv, y = o[nv][2 * half + 1] * inv;
+      if (gate) {
+        const float2 z = unpack2(*reinterpret_cast<const uint32_t*>(gate + (int64_t)r * a.ldp + c));
+        x *= sigmoidf_(z.x);
+        y *= sigmoidf_(z.y);
+      }
+      *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(x, y);
+    }
+  }
+}
+
+template <int NV>
+cudaError_t launch_prompt_tiles(const LatentArgs& a, const Rows& rows, int key0, __nv_bfloat16* out, int64_t ldo, cudaStream_t st) {
+  const PromptShape s = prompt_shape(a);
+  const cudaError_t e = cudaFuncSetAttribute(latent_prompt_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, s.smem);
+  if (e != cudaSuccess) return e;
+  latent_prompt_kernel<NV><<<dim3((rows.n + kQT - 1) / kQT, a.heads), kPromptThreads, s.smem, st>>>(a, rows, key0, s, out, ldo);
+  return cudaGetLastError();
+}
+
+}  // namespace
+
+bool latent_prompt_supported(const LatentArgs& a, int rows) {
+  return rows >= kPromptMinRows && a.dim % 8 == 0 && a.rot % 8 == 0 && a.vdim % 8 == 0 && a.vdim <= 256 && a.dim + a.rot <= 256 && a.ldp % 8 == 0 && a.kv &&
+         prompt_shape(a).smem <= 227 * 1024;
+}
+
+cudaError_t launch_latent_prompt(const LatentArgs& a, const TmaMap& upmap, const Rows& rows, int pos0, __nv_bfloat16* out, int64_t ldo, int* status,
+                                 cudaStream_t st, int* launches) {
+  latent_store_kernel<<<rows.n, kThreads, 0, st>>>(a, rows);
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) return e;
+  const int key0 = a.window > 0 && pos0 - a.window + 1 > 0 ? pos0 - a.window + 1 : 0, keys = pos0 + rows.n - key0;
+  if (keys > a.kv_rows) return cudaErrorInvalidValue;
+  // keys and values of the visible positions
+  const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(a.cache) + ((int64_t)rows.seq0 * a.capacity + key0) * a.width;
+  XMaps x;
+  if (!encode_bf16_map(&x.narrow, base, keys, a.rank, a.width, kGemmTokenBox) || !encode_bf16_map(&x.wide, base, keys, a.rank, a.width, 128))
+    return cudaErrorInvalidValue;
+  e = launch_gemm_bf16(LinearArgs{a.up, nullptr, ACT_NONE, 0, keys}, upmap, x, nullptr, a.kv, a.kv_ld, status, st);
+  if (e != cudaSuccess) return e;
+  if (a.vdim <= 32) e = launch_prompt_tiles<4>(a, rows, key0, out, ldo, st);
+  else if (a.vdim <= 64) e = launch_prompt_tiles<8>(a, rows, key0, out, ldo, st);
+  else if (a.vdim <= 128) e = launch_prompt_tiles<16>(a, rows, key0, out, ldo, st);
+  else e = launch_prompt_tiles<32>(a, rows, key0, out, ldo, st);
+  *launches += 3;
+  return e;
 }
 
 }  // namespace emelb

@@ -332,7 +332,7 @@ void mixer_rows(Layered* m, LayeredRun& r, const LayerS& l, const RunS& run, con
       check(m, r, (launch_latent_rows<T, T, T>(a, rows, out, ldo, m->c->sm_count, false, r.st, &r.launches)), 0);
   } else {
     const DeltaArgs a = delta_args(m, l, run, proj, ldp, tail, tail_ld);
-    if (rows.prompt) check(m, r, launch_delta_prompt<T>(a, rows, out, ldo, r.st, &r.launches), 0);
+    if (rows.prompt) check(m, r, launch_delta_prompt<T>(a, rows, out, ldo, m->c->sm_count, r.st, &r.launches), 0);
     else check(m, r, (launch_delta_step<T, T>(a, rows, out, ldo, false, r.st)));
   }
 }

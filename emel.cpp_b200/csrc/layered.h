@@ -255,7 +255,7 @@ template <class TP, class TO>
 cudaError_t launch_delta_step(const DeltaArgs& a, const Rows& rows, TO* out, int64_t ldo, bool pdl, cudaStream_t st);
 // a prompt: convolution and scalars, the recurrence (token by token, or chunks on the tensor cores), norm and gate
 template <class T>
-cudaError_t launch_delta_prompt(const DeltaArgs& a, const Rows& rows, T* out, int64_t ldo, cudaStream_t st, int* launches);
+cudaError_t launch_delta_prompt(const DeltaArgs& a, const Rows& rows, T* out, int64_t ldo, int sm_count, cudaStream_t st, int* launches);
 bool delta_chunks_supported(const DeltaArgs& a);
 size_t delta_chunk_floats();                 // scratch per (chunk, head)
 int delta_chunks(int rows);
