@@ -3,9 +3,10 @@
 // (sequence, head) is f32 and stays in HBM between calls; a sequence that starts at position 0 starts from zero whatever
 // the memory holds.
 //
-// One token: everything from the projections to the gated heads is one launch, a block per (head, row).
+// One token: everything from the projections to the gated heads is one launch, a cluster per (head, row).
 // Prompts: convolution and the tokens' scalars; the recurrence; norm and gate.  1 / |q| and 1 / |k| stay f32 factors
 // beside the convolved vectors, so that the vectors themselves can be bf16 operands.
+#include <cooperative_groups.h>
 #include <math.h>
 
 #include "act.cuh"
@@ -26,77 +27,136 @@ constexpr float kUnitEps = 1e-6f;   // inside the root of the unit norms
 
 __device__ __forceinline__ float log_decay(const DeltaArgs& a, int h, float x) { return -expf(a.decay_log[h]) * softplusf_(x + a.step_bias[h]); }
 
-// ---- one token
-constexpr int kStepThreads = 512, kStepCols = 128, kStepGroups = kStepThreads / kStepCols;
-
-// grid (heads, rows).  RPT: state rows a thread keeps in registers between its two uses (0: read twice)
-template <class TP, class TO, int RPT>
-__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaArgs a, const Rows rows, TO* __restrict__ out, int64_t ldo) {
-  extern __shared__ float sm[];
-  float* q = sm;                          // [dim]
-  float* k = q + a.dim;                   // [dim]
-  float* v = k + a.dim;                   // [vdim], later the outputs
-  float* red = v + a.vdim;                // [2][kStepGroups][kStepCols]
-  __shared__ float scal[3];               // 1 / |q| / sqrt(dim), 1 / |k|, q . k (unscaled)
-  __shared__ float total[kStepThreads / 32];
-  pdl_trigger();
-  const int h = blockIdx.x, r = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+// ---- one token.  The channels of one head's q, k (and `nv` of its values from v0) through convolution and silu into shared
+// memory: q [dim] | k [dim] | v; the ring takes the step's projections (keys and queries once per group of heads).
+template <class TP>
+__device__ __forceinline__ void step_inputs(const DeltaArgs& a, const TP* x, float* ring, int pos, int h, int v0, int nv, bool store_qk, float* dst) {
   const int rep = a.heads / a.kv_heads, kh = h / rep, channels = a.channels();
-  pdl_wait();
-  const int pos = rows.prompt ? rows.pos[0] : rows.pos[r], seq = rows.prompt ? rows.seq0 : rows.seq0 + r;
-  const int cols = tid % kStepCols, group = tid / kStepCols;
-  float* state = a.state + ((int64_t)seq * a.heads + h) * a.dim * a.vdim;
-  // the state's first tile is on its way while the convolution runs
-  float S[RPT > 0 ? RPT : 1];
-  auto fetch = [&](int c) {
-#pragma unroll
-    for (int i = 0; i < RPT; ++i) {
-      const int row = group + i * kStepGroups;
-      S[i] = pos > 0 && row < a.dim && c < a.vdim ? state[(int64_t)row * a.vdim + c] : 0.0f;
-    }
-  };
-  if (RPT > 0) fetch(cols);
-
-  const TP* x = static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp;
-  float* ring = a.conv_state + (int64_t)seq * a.taps * channels;
-  for (int i = tid; i < 2 * a.dim + a.vdim; i += kStepThreads) {
-    const int c = i < a.dim ? kh * a.dim + i : i < 2 * a.dim ? (a.kv_heads + kh) * a.dim + i - a.dim : 2 * a.kv_heads * a.dim + h * a.vdim + i - 2 * a.dim;
+  for (int i = threadIdx.x; i < 2 * a.dim + nv; i += blockDim.x) {
+    const int c = i < a.dim ? kh * a.dim + i : i < 2 * a.dim ? (a.kv_heads + kh) * a.dim + i - a.dim : 2 * a.kv_heads * a.dim + h * a.vdim + v0 + i - 2 * a.dim;
     const float u = from(x[c]);
     float y = a.conv[(int64_t)(a.taps - 1) * channels + c] * u;
-    for (int b = 1; b < a.taps && b <= pos; ++b) y = fmaf(a.conv[(int64_t)(a.taps - 1 - b) * channels + c], ring[(int64_t)((pos - b) % a.taps) * channels + c], y);
+#pragma unroll 4
+    for (int b = 1; b < a.taps; ++b) {
+      const float past = b <= pos ? ring[(int64_t)((pos - b) % a.taps) * channels + c] : 0.0f;
+      y = fmaf(a.conv[(int64_t)(a.taps - 1 - b) * channels + c], past, y);
+    }
     // no block reads this entry in this step: its old token lies `taps` back
-    if (i >= 2 * a.dim || h % rep == 0) ring[(int64_t)(pos % a.taps) * channels + c] = u;
-    sm[i] = siluf_(y);
+    if (i >= 2 * a.dim || (store_qk && h % rep == 0)) ring[(int64_t)(pos % a.taps) * channels + c] = u;
+    dst[i] = siluf_(y);
   }
+}
+// after a barrier, by the first three warps: 1 / |q| / sqrt(dim), 1 / |k|, q . k (unscaled)
+__device__ __forceinline__ void step_scalars(const DeltaArgs& a, const float* q, const float* k, float* scal) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp >= 3) return;
+  const float *s0 = warp == 1 ? k : q, *s1 = warp == 0 ? q : k;
+  float s = 0.0f;
+  for (int i = lane; i < a.dim; i += 32) s = fmaf(s0[i], s1[i], s);
+  s = warp_sum(s);
+  if (lane == 0) scal[warp] = warp == 2 ? s : 1.0f / sqrtf(s + kUnitEps) * (warp == 0 ? 1.0f / sqrtf((float)a.dim) : 1.0f);
+}
+
+// A cluster = one head of one row, a block = 32 of its value columns; the state tile stays in registers between its two
+// uses, and the blocks add their squares through distributed shared memory.  Grid (column tiles, heads, rows).
+constexpr int kTileCols = 32, kTileGroups = 16, kTileThreads = kTileCols * kTileGroups, kTileRows = 8;   // dim <= 128
+constexpr int kMaxTiles = 8;
+
+template <class TP, class TO>
+__global__ void __launch_bounds__(kTileThreads) delta_step_kernel(const DeltaArgs a, const Rows rows, TO* __restrict__ out, int64_t ldo) {
+  namespace cg = cooperative_groups;
+  extern __shared__ float sm[];
+  float *q = sm, *k = q + a.dim, *v = k + a.dim;           // [dim], [dim], [kTileCols]
+  __shared__ float red[2][kTileGroups][kTileCols];
+  __shared__ float scal[3], squares;
+  pdl_trigger();
+  pdl_wait();
+  cg::cluster_group cluster = cg::this_cluster();
+  const int v0 = blockIdx.x * kTileCols, h = blockIdx.y, r = blockIdx.z, cols = threadIdx.x % kTileCols, group = threadIdx.x / kTileCols;
+  const int pos = rows.prompt ? rows.pos[0] : rows.pos[r], seq = rows.prompt ? rows.seq0 : rows.seq0 + r, c = v0 + cols;
+  const bool live = c < a.vdim;
+  float* state = a.state + ((int64_t)seq * a.heads + h) * a.dim * a.vdim;
+  float S[kTileRows];
+#pragma unroll
+  for (int i = 0; i < kTileRows; ++i) {
+    const int row = group + i * kTileGroups;
+    S[i] = pos > 0 && row < a.dim && live ? state[(int64_t)row * a.vdim + c] : 0.0f;
+  }
+  const float* gates = a.gates + (int64_t)r * a.ldg;
+  const float step = gates[h], decay = gates[a.heads + h];
+  const TP* x = static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp;
+  const float gate = live ? from(x[a.channels() + h * a.vdim + c]) : 0.0f;
+  step_inputs(a, x, a.conv_state + (int64_t)seq * a.taps * a.channels(), pos, h, v0, min(kTileCols, a.vdim - v0), blockIdx.x == 0, sm);
   __syncthreads();
-  if (warp < 3) {
-    const float *s0 = warp == 1 ? k : q, *s1 = warp == 0 ? q : k;
-    float s = 0.0f;
-    for (int i = lane; i < a.dim; i += 32) s = fmaf(s0[i], s1[i], s);
-    s = warp_sum(s);
-    if (lane == 0) scal[warp] = warp == 2 ? s : 1.0f / sqrtf(s + kUnitEps) * (warp == 0 ? 1.0f / sqrtf((float)a.dim) : 1.0f);
+  step_scalars(a, q, k, scal);
+  float sk = 0.0f, sq = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kTileRows; ++i) {
+    const int row = group + i * kTileGroups;
+    if (row < a.dim) {
+      sk = fmaf(S[i], k[row], sk);
+      sq = fmaf(S[i], q[row], sq);
+    }
   }
+  red[0][group][cols] = sk;
+  red[1][group][cols] = sq;
+  __syncthreads();
+  sk = sq = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kTileGroups; ++i) {
+    sk += red[0][i][cols];
+    sq += red[1][i][cols];
+  }
+  const float beta = sigmoidf_(step), g = expf(log_decay(a, h, decay)), rq = scal[0], rk = scal[1];
+  const float u = live ? beta * (v[cols] - g * rk * sk) : 0.0f, o = live ? g * rq * sq + scal[2] * rq * rk * u : 0.0f;
+  if (live) {
+#pragma unroll
+    for (int i = 0; i < kTileRows; ++i) {
+      const int row = group + i * kTileGroups;
+      if (row < a.dim) state[(int64_t)row * a.vdim + c] = fmaf(k[row], rk * u, g * S[i]);
+    }
+  }
+  if (group == 0) {
+    const float ss = warp_sum(o * o);
+    if (cols == 0) squares = ss;
+  }
+  cluster.sync();
+  if (group == 0) {
+    const float mine = cols < (int)gridDim.x ? *cluster.map_shared_rank(&squares, cols) : 0.0f;
+    const float inv = 1.0f / sqrtf(warp_sum(mine) / a.vdim + a.eps);
+    if (live) out[(int64_t)r * ldo + h * a.vdim + c] = to<TO>(o * inv * a.norm[c] * siluf_(gate));
+  }
+  cluster.sync();   // no block leaves while another reads its sum
+}
+
+// other sizes: one block per (head, row), the state read twice
+constexpr int kStepThreads = 512, kStepCols = 128, kStepGroups = kStepThreads / kStepCols;
+
+template <class TP, class TO>
+__global__ void __launch_bounds__(kStepThreads) delta_step_wide_kernel(const DeltaArgs a, const Rows rows, TO* __restrict__ out, int64_t ldo) {
+  extern __shared__ float sm[];
+  float *q = sm, *k = q + a.dim, *v = k + a.dim;          // [dim], [dim], [vdim] (later the outputs)
+  float* red = v + a.vdim;                                // [2][kStepGroups][kStepCols]
+  __shared__ float scal[3], total[kStepThreads / 32];
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.x, r = blockIdx.y, tid = threadIdx.x, cols = tid % kStepCols, group = tid / kStepCols;
+  const int pos = rows.prompt ? rows.pos[0] : rows.pos[r], seq = rows.prompt ? rows.seq0 : rows.seq0 + r;
+  float* state = a.state + ((int64_t)seq * a.heads + h) * a.dim * a.vdim;
+  const TP* x = static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp;
+  step_inputs(a, x, a.conv_state + (int64_t)seq * a.taps * a.channels(), pos, h, 0, a.vdim, true, sm);
+  __syncthreads();
+  step_scalars(a, q, k, scal);
   const float* gates = a.gates + (int64_t)r * a.ldg;
   const float beta = sigmoidf_(gates[h]), g = expf(log_decay(a, h, gates[a.heads + h]));
   __syncthreads();
   const float rq = scal[0], rk = scal[1], qk = scal[2] * rq * rk;
-
   float ss = 0.0f;
   for (int c0 = 0; c0 < a.vdim; c0 += kStepCols) {
     const int c = c0 + cols;
     const bool live = c < a.vdim;
-    if (RPT > 0 && c0 > 0) fetch(c);
     float sk = 0.0f, sq = 0.0f;
-    if (RPT > 0) {
-#pragma unroll
-      for (int i = 0; i < RPT; ++i) {
-        const int row = group + i * kStepGroups;
-        if (row < a.dim) {
-          sk = fmaf(S[i], k[row], sk);
-          sq = fmaf(S[i], q[row], sq);
-        }
-      }
-    } else if (live && pos > 0) {
+    if (live && pos > 0) {
 #pragma unroll 8
       for (int row = group; row < a.dim; row += kStepGroups) {
         const float s = state[(int64_t)row * a.vdim + c];
@@ -117,19 +177,10 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaArg
     const float o = g * rq * sq + qk * u;
     __syncthreads();
     if (live) {
-      const float ku = rk * u;
-      if (RPT > 0) {
-#pragma unroll
-        for (int i = 0; i < RPT; ++i) {
-          const int row = group + i * kStepGroups;
-          if (row < a.dim) state[(int64_t)row * a.vdim + c] = fmaf(k[row], ku, g * S[i]);
-        }
-      } else {
 #pragma unroll 8
-        for (int row = group; row < a.dim; row += kStepGroups) {
-          const float s = pos > 0 ? state[(int64_t)row * a.vdim + c] : 0.0f;
-          state[(int64_t)row * a.vdim + c] = fmaf(k[row], ku, g * s);
-        }
+      for (int row = group; row < a.dim; row += kStepGroups) {
+        const float s = pos > 0 ? state[(int64_t)row * a.vdim + c] : 0.0f;
+        state[(int64_t)row * a.vdim + c] = fmaf(k[row], rk * u, g * s);
       }
       if (group == 0) {
         v[c] = o;
@@ -138,13 +189,13 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaArg
     }
   }
   ss = warp_sum(ss);
-  if (lane == 0) total[warp] = ss;
+  if ((tid & 31) == 0) total[tid >> 5] = ss;
   __syncthreads();
   ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < kStepCols / 32; ++i) ss += total[i];   // the first group's warps
   const float inv = 1.0f / sqrtf(ss / a.vdim + a.eps);
-  const TP* gate = x + channels + h * a.vdim;
+  const TP* gate = x + a.channels() + h * a.vdim;
   for (int c = tid; c < a.vdim; c += kStepThreads) out[(int64_t)r * ldo + h * a.vdim + c] = to<TO>(v[c] * inv * a.norm[c] * siluf_(from(gate[c])));
 }
 
@@ -183,7 +234,7 @@ struct Vec<__nv_bfloat16, 4> {
 // warp per block row takes the rows' gates.  Rows before the batch come from the ring.
 // FEW: at most four taps, every input and weight of a turn requested at once
 template <class T, int V, bool FEW>
-__global__ void __launch_bounds__(kConvThreads) delta_conv_kernel(const DeltaArgs a, const Rows rows) {
+__global__ void __launch_bounds__(kConvThreads, 5) delta_conv_kernel(const DeltaArgs a, const Rows rows) {
   const int lane = threadIdx.x & 31, task = blockIdx.x * (kConvThreads / 32) + (threadIdx.x >> 5), r0 = blockIdx.y * kConvRows;
   const int vectors = 2 * a.kv_heads + a.heads, channels = a.channels(), pos0 = rows.pos[0], nr = min(kConvRows, rows.n - r0);
   const int ns = a.scalar_count();
@@ -717,8 +768,9 @@ cudaError_t launch_chunks(const DeltaArgs& a, const Rows& rows, int sm_count, cu
   return a.heads * ((a.vdim + 15) / 16) <= sm_count ? launch_scan<D, 16>(a, rows, st) : launch_scan<D, 32>(a, rows, st);
 }
 
-// a warp per (row, head)
-template <class T>
+// a warp per (row, head), V columns per lane and turn; the first kNormTurns turns stay in registers
+constexpr int kNormTurns = 4;
+template <class T, int V>
 __global__ void __launch_bounds__(kConvThreads) delta_norm_kernel(const DeltaArgs a, const Rows rows, T* __restrict__ out, int64_t ldo) {
   const int64_t task = (int64_t)blockIdx.x * (kConvThreads / 32) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -727,10 +779,43 @@ __global__ void __launch_bounds__(kConvThreads) delta_norm_kernel(const DeltaArg
   const int h = (int)(task % a.heads);
   const float* o = a.o + task * a.vdim;
   const T* gate = static_cast<const T*>(a.proj) + r * a.ldp + a.channels() + h * a.vdim;
-  float ss = 0.0f;
-  for (int c = lane; c < a.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
+  T* dst = out + r * ldo + h * a.vdim;
+  float x[kNormTurns][V], z[kNormTurns][V], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kNormTurns; ++i) {
+    const int c = V * (lane + 32 * i);
+    if (c >= a.vdim) break;
+    Vec<float, V>::load(o + c, x[i]);
+    Vec<T, V>::load(gate + c, z[i]);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(x[i][e], x[i][e], ss);
+  }
+  for (int c = V * (lane + 32 * kNormTurns); c < a.vdim; c += 32 * V) {
+    float y[V];
+    Vec<float, V>::load(o + c, y);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(y[e], y[e], ss);
+  }
   const float inv = 1.0f / sqrtf(warp_sum(ss) / a.vdim + a.eps);
-  for (int c = lane; c < a.vdim; c += 32) out[r * ldo + h * a.vdim + c] = to<T>(o[c] * inv * a.norm[c] * siluf_(from(gate[c])));
+  auto finish = [&](int c, float (&y)[V], const float (&g)[V]) {
+    float w[V];
+    Vec<float, V>::load(a.norm + c, w);
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[e] = y[e] * inv * w[e] * siluf_(g[e]);
+    Vec<T, V>::store(dst + c, y);
+  };
+#pragma unroll
+  for (int i = 0; i < kNormTurns; ++i) {
+    const int c = V * (lane + 32 * i);
+    if (c >= a.vdim) break;
+    finish(c, x[i], z[i]);
+  }
+  for (int c = V * (lane + 32 * kNormTurns); c < a.vdim; c += 32 * V) {
+    float y[V], g[V];
+    Vec<float, V>::load(o + c, y);
+    Vec<T, V>::load(gate + c, g);
+    finish(c, y, g);
+  }
 }
 
 }  // namespace
@@ -741,10 +826,26 @@ int delta_chunks(int rows) { return (rows + kChunk - 1) / kChunk; }
 
 template <class TP, class TO>
 cudaError_t launch_delta_step(const DeltaArgs& a, const Rows& rows, TO* out, int64_t ldo, bool pdl, cudaStream_t st) {
-  const size_t smem = 4 * (2 * (size_t)a.dim + a.vdim + 2 * kStepGroups * kStepCols);
-  if (smem > 48 * 1024) return cudaErrorInvalidValue;
-  auto kern = a.dim <= 32 * kStepGroups ? delta_step_kernel<TP, TO, 32> : delta_step_kernel<TP, TO, 0>;
-  return launch_kernel(kern, dim3(a.heads, rows.n), dim3(kStepThreads), smem, st, pdl, a, rows, out, ldo);
+  const int tiles = (a.vdim + kTileCols - 1) / kTileCols;
+  if (a.dim > kTileGroups * kTileRows || tiles > kMaxTiles) {
+    const size_t smem = 4 * (2 * (size_t)a.dim + a.vdim + 2 * kStepGroups * kStepCols);
+    if (smem > 48 * 1024) return cudaErrorInvalidValue;
+    return launch_kernel(delta_step_wide_kernel<TP, TO>, dim3(a.heads, rows.n), dim3(kStepThreads), smem, st, pdl, a, rows, out, ldo);
+  }
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3(tiles, a.heads, rows.n);
+  cfg.blockDim = dim3(kTileThreads);
+  cfg.dynamicSmemBytes = 4 * (2 * (size_t)a.dim + kTileCols);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = tiles;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl ? 2 : 1;
+  return cudaLaunchKernelEx(&cfg, delta_step_kernel<TP, TO>, a, rows, out, ldo);
 }
 template cudaError_t launch_delta_step<float, float>(const DeltaArgs&, const Rows&, float*, int64_t, bool, cudaStream_t);
 template cudaError_t launch_delta_step<__nv_bfloat16, __nv_bfloat16>(const DeltaArgs&, const Rows&, __nv_bfloat16*, int64_t, bool, cudaStream_t);
@@ -786,7 +887,9 @@ cudaError_t launch_delta_prompt(const DeltaArgs& a, const Rows& rows, T* out, in
     delta_rows_kernel<T><<<dim3(a.heads, (a.vdim + kCols - 1) / kCols), dim3(kCols, kGroups), smem, st>>>(a, rows);
     if ((e = cudaGetLastError()) != cudaSuccess) return e;
   }
-  delta_norm_kernel<T><<<(unsigned)(((int64_t)rows.n * a.heads + warps - 1) / warps), kConvThreads, 0, st>>>(a, rows, out, ldo);
+  const unsigned blocks = (unsigned)(((int64_t)rows.n * a.heads + warps - 1) / warps);
+  if (a.dim % 2 == 0 && a.vdim % 4 == 0 && a.ldp % 4 == 0 && ldo % 4 == 0) delta_norm_kernel<T, 4><<<blocks, kConvThreads, 0, st>>>(a, rows, out, ldo);
+  else delta_norm_kernel<T, 1><<<blocks, kConvThreads, 0, st>>>(a, rows, out, ldo);
   return cudaGetLastError();
 }
 template cudaError_t launch_delta_prompt<float>(const DeltaArgs&, const Rows&, float*, int64_t, int, cudaStream_t, int*);

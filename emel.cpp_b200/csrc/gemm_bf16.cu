@@ -80,9 +80,22 @@ __device__ __forceinline__ void mma_bf16(uint32_t tmem_d, uint64_t da, uint64_t 
 __device__ __forceinline__ void mma_commit(uint64_t* bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
 }
-__device__ __forceinline__ void tmem_ld8(uint32_t taddr, uint32_t (&v)[8]) {
-  asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
-               : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7])
+__device__ __forceinline__ void tmem_ld(uint32_t taddr, uint32_t (&v)[16]) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+               "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+               : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
+                 "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+               : "r"(taddr)
+               : "memory");
+}
+__device__ __forceinline__ void tmem_ld(uint32_t taddr, uint32_t (&v)[32]) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+               "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
+               "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+               : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
+                 "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]),
+                 "=r"(v[16]), "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]),
+                 "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
                : "r"(taddr)
                : "memory");
 }
@@ -191,26 +204,51 @@ __global__ void __launch_bounds__(kThreads) gemm_bf16_kernel(const __grid_consta
       const float b0 = live && p.bias ? p.bias[f] : 0.0f, b1 = GLU && live && p.bias ? p.bias[p.M + f] : 0.0f;
       const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
       const bool sigm = p.act == ACT_SILU_SIGMOID, gelu = p.act == ACT_GLU_GELU, cap = p.act == ACT_SOFTCAP, tail = f >= p.tail;
-      for (int c = 0; c < BN && t0 + c < p.rows; c += 8) {
-        uint32_t v[8], u[8];
-        tmem_ld8(lane_base + c, v);
-        if (GLU) tmem_ld8(lane_base + BN + c, u);
+      // bf16 outputs turn in shared memory (the stages are free: every copy has landed and been used), 32 features x kCh rows of
+      // a warp at a time, and leave as 16-byte stores
+      constexpr int kCh = BN < 32 ? BN : 32, kTileLd = 40;
+      __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(smem) + warp * 32 * kTileLd;
+      const int f_end = min(p.M, p.tail), fw = f0 + warp * 32;
+      for (int c = 0; c < BN && t0 + c < p.rows; c += kCh) {
+        uint32_t v[kCh], u[GLU ? kCh : 1];
+        tmem_ld(lane_base + c, v);
+        if constexpr (GLU) tmem_ld(lane_base + BN + c, u);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        float o[kCh];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          float o = __uint_as_float(v[j]) + b0;
-          if (GLU) {
-            o = (gelu ? gelu_tanhf_(o) : siluf_(o)) * (__uint_as_float(u[j]) + b1);
+        for (int j = 0; j < kCh; ++j) {
+          o[j] = __uint_as_float(v[j]) + b0;
+          if constexpr (GLU) {
+            o[j] = (gelu ? gelu_tanhf_(o[j]) : siluf_(o[j])) * (__uint_as_float(u[j]) + b1);
           } else if (sigm) {
-            const float sg = sigmoidf_(o);
-            o = f < p.act_split ? o * sg : sg;
+            const float sg = sigmoidf_(o[j]);
+            o[j] = f < p.act_split ? o[j] * sg : sg;
           } else if (cap) {
-            o = softcapf_(o * p.out_scale, p.softcap);
+            o[j] = softcapf_(o[j] * p.out_scale, p.softcap);
           }
-          if (live && t0 + c + j < p.rows) {
-            if (tail) p.tail_y[(int64_t)(t0 + c + j) * p.tail_ld + f - p.tail] = o;
-            else if (p.yb) p.yb[(int64_t)(t0 + c + j) * p.ldy + f] = __float2bfloat16_rn(o);
-            else p.y[(int64_t)(t0 + c + j) * p.ldy + f] = o;
+        }
+        if (live && (tail || !p.yb)) {
+          float* y = tail ? p.tail_y + f - p.tail : p.y + f;
+          const int64_t ld = tail ? p.tail_ld : p.ldy;
+#pragma unroll
+          for (int j = 0; j < kCh; ++j)
+            if (t0 + c + j < p.rows) y[(int64_t)(t0 + c + j) * ld] = o[j];
+        }
+        if (!p.yb) continue;
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < kCh; ++j) tile[j * kTileLd + lane] = __float2bfloat16_rn(o[j]);
+        __syncwarp();
+#pragma unroll
+        for (int i = lane; i < 4 * kCh; i += 32) {
+          const int j = i / 4, q = 8 * (i % 4), n = f_end - fw - q;   // n features of this piece are stored
+          if (t0 + c + j >= p.rows || n <= 0) continue;
+          const __nv_bfloat16* src = tile + j * kTileLd + q;
+          __nv_bfloat16* dst = p.yb + (int64_t)(t0 + c + j) * p.ldy + fw + q;
+          if (n >= 8) {
+            *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
+          } else {
+            for (int e = 0; e < n; ++e) dst[e] = src[e];
           }
         }
       }
@@ -258,6 +296,7 @@ bool encode_bf16_map(TmaMap* map, const __nv_bfloat16* base, int64_t rows, int64
 
 cudaError_t launch_gemm_bf16(const LinearArgs& a, const TmaMap& wmap, const XMaps& x, float* y, __nv_bfloat16* yb, int64_t ldy, int* status,
                              cudaStream_t st) {
+  if (yb && (ldy % 8 != 0 || reinterpret_cast<uintptr_t>(yb) % 16 != 0)) return cudaErrorInvalidValue;
   const bool glu = is_glu(a.act);
   GemmParams p{glu ? a.w.M / 2 : a.w.M, a.w.K, a.rows, a.bias, a.act, a.act_split, y, yb, ldy, status,
                a.out_scale, a.softcap, a.tail, a.tail_y, a.tail_ld};

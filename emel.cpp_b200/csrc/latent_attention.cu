@@ -21,7 +21,7 @@ namespace {
 
 constexpr int kThreads = 128;
 constexpr int kHG = 8;          // heads per block of the attention launch
-constexpr int kKeys = 64;       // keys per tile
+constexpr int kKeys = 64;       // most keys per tile
 constexpr int kCols = 512;      // latent columns per block of the attention launch
 constexpr int kSlice = 64;      // latent columns per block of the query launch
 constexpr int kOutTile = 32;    // values per block of the out launch
@@ -53,6 +53,8 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
   const float2 a = unpack2(v.x), b = unpack2(v.y);
   f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
 }
+
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 __device__ __forceinline__ int row_pos(const Rows& r, int i) { return r.prompt ? r.pos[0] + i : r.pos[i]; }
 __device__ __forceinline__ int row_seq(const Rows& r, int i) { return r.prompt ? r.seq0 : r.seq0 + i; }
@@ -111,8 +113,10 @@ template <class TC, class TP>
 __global__ void __launch_bounds__(kThreads) latent_in_kernel(const LatentArgs a, const Rows rows, int row0) {
   extern __shared__ float qs[];            // [dim], then the warps' partial columns
   pdl_trigger();
-  pdl_wait();
   const int h = blockIdx.y, r = row0 + blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (blockIdx.x < gridDim.x - 1)
+    for (int d = tid; d < a.dim; d += kThreads) prefetch_l2(a.up.w + (int64_t)(h * a.dim + d) * a.up.ld + blockIdx.x * kSlice);
+  pdl_wait();
   const TP* q = static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp + h * (a.dim + a.rot);
   float* out = a.qlat + ((int64_t)blockIdx.z * a.heads + h) * a.width;
   if (blockIdx.x == gridDim.x - 1) {
@@ -170,12 +174,13 @@ __device__ __forceinline__ float transpose_sum(float (&v)[32]) {
   return v[0];
 }
 
-// grid (ranges x column blocks, head groups, rows)
+// grid (ranges x column blocks, head groups, rows); tiles of `keys` cache rows pass through shared memory
 template <class TC>
-__global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs a, const Rows rows, int row0, int splits) {
+__global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs a, const Rows rows, int row0, int splits, int keys) {
   extern __shared__ __align__(16) float sm[];
   float* qs = sm;                          // [kHG][width]
   float* p = qs + kHG * a.width;           // [kHG][kKeys] scores, then weights
+  TC* tile = reinterpret_cast<TC*>(p + kHG * kKeys);   // [keys][width]
   __shared__ float m_run[kHG], l_run[kHG], fix[kHG];
   pdl_trigger();
   pdl_wait();
@@ -184,6 +189,13 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
   const int pos = row_pos(rows, r), lo = first_key(pos, a.window), n = pos - lo + 1;
   const int L = (n + splits - 1) / splits, k0 = min(n, split * L), k1 = min(n, k0 + L);
   const TC* cache = static_cast<const TC*>(a.cache) + ((int64_t)row_seq(rows, r) * a.capacity + lo) * a.width;
+  constexpr int kPer16 = 16 / sizeof(TC);
+  auto fetch = [&](int t0) {
+    const TC* src = cache + (int64_t)t0 * a.width;
+    for (int i = tid; i < min(keys, k1 - t0) * a.width / kPer16; i += kThreads) cp_async16(tile + i * kPer16, src + i * kPer16);
+    cp_async_commit();
+  };
+  if (k0 < k1) fetch(k0);
   const float* q = a.qlat + ((int64_t)blockIdx.z * a.heads + h0) * a.width;
   for (int i = tid; i < kHG * a.width; i += kThreads) qs[i] = h0 + i / a.width < a.heads ? q[i] : 0.0f;
   if (tid < kHG) {
@@ -193,14 +205,15 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
   const int col = col0 + 4 * tid;
   const bool mine = col < a.rank_pad;
   float acc[kHG][4] = {};
-  for (int t0 = k0; t0 < k1; t0 += kKeys) {
-    const int nt = min(kKeys, k1 - t0);
+  for (int t0 = k0; t0 < k1; t0 += keys) {
+    const int nt = min(keys, k1 - t0);
+    cp_async_wait<0>();
     __syncthreads();
     // scores: four keys of a warp at a time, lanes across the row
     for (int kb = 4 * warp; kb < nt; kb += 4 * (kThreads / 32)) {
       const TC* kp[4];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) kp[u] = cache + (int64_t)(t0 + min(kb + u, nt - 1)) * a.width;
+      for (int u = 0; u < 4; ++u) kp[u] = tile + min(kb + u, nt - 1) * a.width;
       float s[4 * kHG] = {};
       for (int c = 8 * lane; c < a.width; c += 256) {
         float kf[4][8];
@@ -246,7 +259,7 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
       for (int k = 0; k < nt; k += 4) {
         float v[4][4];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) load4(cache + (int64_t)(t0 + min(k + u, nt - 1)) * a.width + col, v[u]);   // weights past nt are 0
+        for (int u = 0; u < 4; ++u) load4(tile + min(k + u, nt - 1) * a.width + col, v[u]);   // weights past nt are 0
 #pragma unroll
         for (int h = 0; h < kHG; ++h) {
           const float4 w = *reinterpret_cast<const float4*>(p + h * kKeys + k);
@@ -255,6 +268,8 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
         }
       }
     }
+    __syncthreads();
+    if (t0 + keys < k1) fetch(t0 + keys);
   }
   __syncthreads();
   if (mine)
@@ -273,8 +288,11 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
   extern __shared__ __align__(16) float o[];    // [rank_pad]
   __shared__ float weight[kMaxSplits];
   pdl_trigger();
-  pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, r = row0 + blockIdx.z;
+  const int e0 = blockIdx.x * kOutTile, e1 = min(a.vdim, e0 + kOutTile);
+  const __nv_bfloat16* up = a.up.w + ((int64_t)a.heads * a.dim + (int64_t)h * a.vdim) * a.up.ld;
+  for (int64_t c = 64 * tid; c < (e1 - e0) * a.up.ld; c += 64 * kThreads) prefetch_l2(up + e0 * a.up.ld + c);
+  pdl_wait();
   if (warp == 0) {
     const float2 s = lane < splits ? reinterpret_cast<const float2*>(a.stats)[((int64_t)blockIdx.z * splits + lane) * a.heads + h] : make_float2(-INFINITY, 0.0f);
     float m = s.x;
@@ -287,9 +305,9 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
   const float* part = a.part + ((int64_t)blockIdx.z * splits * a.heads + h) * a.rank_pad;
   for (int c = 4 * tid; c < a.rank_pad; c += 4 * kThreads) {
     float4 t = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
     for (int s = 0; s < splits; ++s) {
       const float w = weight[s];
-      if (w == 0.0f) continue;
       const float4 v = *reinterpret_cast<const float4*>(part + (int64_t)s * a.heads * a.rank_pad + c);
       t.x = fmaf(w, v.x, t.x);
       t.y = fmaf(w, v.y, t.y);
@@ -300,9 +318,9 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
   }
   __syncthreads();
   const TP* gate = a.gate_at ? static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp + a.gate_at + h * a.vdim : nullptr;
-  const int e0 = blockIdx.x * kOutTile, e1 = min(a.vdim, e0 + kOutTile);
+#pragma unroll 2
   for (int e = e0 + warp; e < e1; e += kThreads / 32) {
-    const __nv_bfloat16* w = a.up.w + ((int64_t)a.heads * a.dim + (int64_t)h * a.vdim + e) * a.up.ld;
+    const __nv_bfloat16* w = up + (int64_t)e * a.up.ld;
     float s = 0.0f;
     for (int c = 8 * lane; c < a.rank_pad; c += 256) {
       float wf[8], of[8];
@@ -332,8 +350,14 @@ cudaError_t launch_latent_rows(const LatentArgs& a, const Rows& rows, TO* out, i
     splits = splits > fill ? fill : splits;
     splits = splits > kMaxSplits ? kMaxSplits : splits;
   }
-  const size_t s_in = 4 * ((size_t)a.dim + kThreads / 32 * kSlice), s_attn = 4 * (size_t)kHG * (a.width + kKeys), s_out = 4 * (size_t)a.rank_pad;
-  if (s_in > 48 * 1024 || s_attn > 200 * 1024 || s_out > 200 * 1024) return cudaErrorInvalidValue;
+  const size_t s_in = 4 * ((size_t)a.dim + kThreads / 32 * kSlice), s_q = 4 * (size_t)kHG * (a.width + kKeys), s_out = 4 * (size_t)a.rank_pad;
+  // two blocks per SM where a tile of 16 keys at least allows it
+  int keys = kKeys;
+  auto s_tile = [&](int k) { return s_q + sizeof(TC) * (size_t)k * a.width; };
+  while (keys > 16 && s_tile(keys) > 110 * 1024) keys /= 2;
+  while (keys > 1 && s_tile(keys) > 220 * 1024) keys /= 2;
+  const size_t s_attn = s_tile(keys);
+  if (s_in > 48 * 1024 || s_attn > 220 * 1024 || s_out > 200 * 1024) return cudaErrorInvalidValue;
   cudaError_t e = cudaSuccess;
   if (s_attn > 40 * 1024) e = cudaFuncSetAttribute(latent_attn_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s_attn);
   if (e == cudaSuccess && s_out > 40 * 1024) e = cudaFuncSetAttribute(latent_out_kernel<TP, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s_out);
@@ -346,7 +370,7 @@ cudaError_t launch_latent_rows(const LatentArgs& a, const Rows& rows, TO* out, i
   for (int r0 = 0; r0 < rows.n; r0 += (int)fit) {
     const int n = rows.n - r0 < (int)fit ? rows.n - r0 : (int)fit;
     e = launch_kernel(latent_in_kernel<TC, TP>, dim3((a.rank_pad + kSlice - 1) / kSlice + 1, a.heads, n), dim3(kThreads), s_in, st, pdl, a, rows, r0);
-    if (e == cudaSuccess) e = launch_kernel(latent_attn_kernel<TC>, dim3(splits * blocks, groups, n), dim3(kThreads), s_attn, st, pdl, a, rows, r0, splits);
+    if (e == cudaSuccess) e = launch_kernel(latent_attn_kernel<TC>, dim3(splits * blocks, groups, n), dim3(kThreads), s_attn, st, pdl, a, rows, r0, splits, keys);
     if (e == cudaSuccess)
       e = launch_kernel(latent_out_kernel<TP, TO>, dim3((a.vdim + kOutTile - 1) / kOutTile, a.heads, n), dim3(kThreads), s_out, st, pdl, a, rows, r0, splits, out, ldo);
     if (e != cudaSuccess) return e;
