@@ -25,6 +25,7 @@ constexpr int kKeys = 64;       // most keys per tile
 constexpr int kCols = 512;      // latent columns per block of the attention launch
 constexpr int kSlice = 64;      // latent columns per block of the query launch
 constexpr int kOutTile = 32;    // values per block of the out launch
+constexpr int kOutThreads = 512, kOutGroups = 4, kOutCols = 4 * kOutThreads / kOutGroups;   // a group adds up every fourth range
 constexpr int kMaxSplits = 32;
 
 __device__ __forceinline__ float from(float x) { return x; }
@@ -284,15 +285,26 @@ __global__ void __launch_bounds__(kThreads) latent_attn_kernel(const LatentArgs 
 
 // grid (value tiles, heads, rows)
 template <class TP, class TO>
-__global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a, const Rows rows, int row0, int splits, TO* __restrict__ out, int64_t ldo) {
+__global__ void __launch_bounds__(kOutThreads) latent_out_kernel(const LatentArgs a, const Rows rows, int row0, int splits, TO* __restrict__ out, int64_t ldo) {
   extern __shared__ __align__(16) float o[];    // [rank_pad]
+  __shared__ float4 sums[kOutGroups][kOutCols / 4];
   __shared__ float weight[kMaxSplits];
   pdl_trigger();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, r = row0 + blockIdx.z;
   const int e0 = blockIdx.x * kOutTile, e1 = min(a.vdim, e0 + kOutTile);
   const __nv_bfloat16* up = a.up.w + ((int64_t)a.heads * a.dim + (int64_t)h * a.vdim) * a.up.ld;
-  for (int64_t c = 64 * tid; c < (e1 - e0) * a.up.ld; c += 64 * kThreads) prefetch_l2(up + e0 * a.up.ld + c);
+  for (int64_t c = 64 * tid; c < (e1 - e0) * a.up.ld; c += 64 * kOutThreads) prefetch_l2(up + e0 * a.up.ld + c);
   pdl_wait();
+  const int group = tid / (kOutCols / 4), quad = tid % (kOutCols / 4);
+  const float* part = a.part + ((int64_t)blockIdx.z * splits * a.heads + h) * a.rank_pad;
+  const int64_t stride = (int64_t)a.heads * a.rank_pad;
+  // the first columns' sums are requested before the ranges' weights are known
+  float4 first[kMaxSplits / kOutGroups];
+#pragma unroll
+  for (int i = 0; i < kMaxSplits / kOutGroups; ++i) {
+    const int s = group + kOutGroups * i;
+    first[i] = s < splits && 4 * quad < a.rank_pad ? *reinterpret_cast<const float4*>(part + s * stride + 4 * quad) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
   if (warp == 0) {
     const float2 s = lane < splits ? reinterpret_cast<const float2*>(a.stats)[((int64_t)blockIdx.z * splits + lane) * a.heads + h] : make_float2(-INFINITY, 0.0f);
     float m = s.x;
@@ -302,24 +314,33 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
     weight[lane] = f / warp_sum(f * s.y);
   }
   __syncthreads();
-  const float* part = a.part + ((int64_t)blockIdx.z * splits * a.heads + h) * a.rank_pad;
-  for (int c = 4 * tid; c < a.rank_pad; c += 4 * kThreads) {
+  for (int c0 = 0; c0 < a.rank_pad; c0 += kOutCols) {
+    const int c = c0 + 4 * quad;
     float4 t = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 8
-    for (int s = 0; s < splits; ++s) {
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / kOutGroups; ++i) {
+      const int s = group + kOutGroups * i;
+      if (s >= splits || c >= a.rank_pad) break;
       const float w = weight[s];
-      const float4 v = *reinterpret_cast<const float4*>(part + (int64_t)s * a.heads * a.rank_pad + c);
+      const float4 v = c0 == 0 ? first[i] : *reinterpret_cast<const float4*>(part + s * stride + c);
       t.x = fmaf(w, v.x, t.x);
       t.y = fmaf(w, v.y, t.y);
       t.z = fmaf(w, v.z, t.z);
       t.w = fmaf(w, v.w, t.w);
     }
-    *reinterpret_cast<float4*>(o + c) = t;
+    sums[group][quad] = t;
+    __syncthreads();
+    for (int x = tid; x < min(kOutCols, a.rank_pad - c0); x += kOutThreads) {
+      float v = 0.0f;
+#pragma unroll
+      for (int g = 0; g < kOutGroups; ++g) v += reinterpret_cast<const float*>(sums[g])[x];
+      o[c0 + x] = v;
+    }
+    __syncthreads();
   }
-  __syncthreads();
   const TP* gate = a.gate_at ? static_cast<const TP*>(a.proj) + (int64_t)r * a.ldp + a.gate_at + h * a.vdim : nullptr;
 #pragma unroll 2
-  for (int e = e0 + warp; e < e1; e += kThreads / 32) {
+  for (int e = e0 + warp; e < e1; e += kOutThreads / 32) {
     const __nv_bfloat16* w = up + (int64_t)e * a.up.ld;
     float s = 0.0f;
     for (int c = 8 * lane; c < a.rank_pad; c += 256) {
@@ -337,11 +358,164 @@ __global__ void __launch_bounds__(kThreads) latent_out_kernel(const LatentArgs a
   }
 }
 
+// ---- the attention launch on the tensor cores (mma.sync bf16): bf16 caches with at most kMmaCols latent columns.  Sixteen
+// heads per block are the rows of both products; query and weights are fed as two bf16 operands, high part and remainder.
+constexpr int kMmaHeads = 16, kMmaThreads = 256, kMmaCols = 64 * kMmaThreads / 32;
+
+struct MmaShape {
+  int kw, row, smem;     // columns of the score product (a multiple of 16), elements between rows in shared memory
+};
+MmaShape mma_shape(const LatentArgs& a) {
+  MmaShape s;
+  s.kw = (a.width + 15) / 16 * 16;
+  s.row = s.kw + 8;
+  s.smem = 2 * (2 * kMmaHeads + kKeys) * s.row + 4 * kMmaHeads * (kKeys + 4) + 2 * 2 * kMmaHeads * (kKeys + 8) + 32;
+  return s;
+}
+
+// grid (ranges, head groups, rows)
+__global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentArgs a, const Rows rows, int row0, int splits, const MmaShape shape) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  constexpr int kPRow = kKeys + 8, kSRow = kKeys + 4;
+  const int R = shape.row;
+  __nv_bfloat16* q_hi = reinterpret_cast<__nv_bfloat16*>(raw);      // [kMmaHeads][R]
+  __nv_bfloat16* q_lo = q_hi + kMmaHeads * R;
+  __nv_bfloat16* tile = q_lo + kMmaHeads * R;                       // [kKeys][R]
+  __nv_bfloat16* p_hi = tile + kKeys * R + 16;                      // [kMmaHeads][kPRow]  (a load of two column blocks may look past the last row)
+  __nv_bfloat16* p_lo = p_hi + kMmaHeads * kPRow;
+  float* sc = reinterpret_cast<float*>(p_lo + kMmaHeads * kPRow);   // [kMmaHeads][kSRow]
+  __shared__ float m_run[kMmaHeads], l_run[kMmaHeads], fix[kMmaHeads];
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int split = blockIdx.x, h0 = blockIdx.y * kMmaHeads, r = row0 + blockIdx.z;
+  const int pos = row_pos(rows, r), lo = first_key(pos, a.window), n = pos - lo + 1;
+  const int L = (n + splits - 1) / splits, k0 = min(n, split * L), k1 = min(n, k0 + L);
+  const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(a.cache) + ((int64_t)row_seq(rows, r) * a.capacity + lo) * a.width;
+  const int chunks = shape.kw / 8, live_chunks = a.width / 8;
+  auto fetch = [&](int t0) {
+    for (int i = tid; i < kKeys * chunks; i += kMmaThreads) {
+      const int k = i / chunks, c = i - k * chunks;
+      const bool live = t0 + k < k1 && c < live_chunks;
+      cp16_zfill(tile + k * R + 8 * c, live ? cache + (int64_t)(t0 + k) * a.width + 8 * c : cache, live);
+    }
+    cp_async_commit();
+  };
+  if (k0 < k1) fetch(k0);
+  const float* q = a.qlat + ((int64_t)blockIdx.z * a.heads + h0) * a.width;
+  for (int i = tid; i < kMmaHeads * shape.kw / 2; i += kMmaThreads) {
+    const int h = i / (shape.kw / 2), c = i % (shape.kw / 2) * 2;
+    const float2 v = h0 + h < a.heads && c < a.width ? *reinterpret_cast<const float2*>(q + (int64_t)h * a.width + c) : make_float2(0.0f, 0.0f);
+    uint32_t hi, rest;
+    split2(v.x, v.y, hi, rest);
+    *reinterpret_cast<uint32_t*>(q_hi + h * R + c) = hi;
+    *reinterpret_cast<uint32_t*>(q_lo + h * R + c) = rest;
+  }
+  if (tid < kMmaHeads) {
+    m_run[tid] = -INFINITY;
+    l_run[tid] = 0.0f;
+  }
+  float acc[8][4] = {};
+  const int c0 = 64 * warp;
+  for (int t0 = k0; t0 < k1; t0 += kKeys) {
+    const int nt = min(kKeys, k1 - t0);
+    cp_async_wait<0>();
+    __syncthreads();
+    {
+      // eight keys per warp
+      float s[2][4] = {};
+      const __nv_bfloat16* kb = tile + (8 * warp + (lane & 7)) * R + 8 * (lane >> 3);
+      const int qa = (lane & 15) * R + (lane >> 4) * 8;
+#pragma unroll 3
+      for (int d = 0; d < shape.kw; d += 32) {
+        uint32_t b[4], x[4];
+        ldsm(b, kb + d);
+        ldsm(x, q_hi + qa + d);
+        mma_bf16_16816(s[0], x, b[0], b[1]);
+        ldsm(x, q_lo + qa + d);
+        mma_bf16_16816(s[1], x, b[0], b[1]);
+        if (d + 16 < shape.kw) {
+          ldsm(x, q_hi + qa + d + 16);
+          mma_bf16_16816(s[0], x, b[2], b[3]);
+          ldsm(x, q_lo + qa + d + 16);
+          mma_bf16_16816(s[1], x, b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[(g + 8 * (e >> 1)) * kSRow + 8 * warp + 2 * t + (e & 1)] = (s[0][e] + s[1][e]) * a.scale;
+    }
+    __syncthreads();
+    for (int h = warp; h < kMmaHeads; h += kMmaThreads / 32) {
+      const float s0 = 2 * lane < nt ? sc[h * kSRow + 2 * lane] : -INFINITY, s1 = 2 * lane + 1 < nt ? sc[h * kSRow + 2 * lane + 1] : -INFINITY;
+      float m = fmaxf(s0, s1);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      const float before = m_run[h];
+      m = fmaxf(m, before);
+      const float w0 = expf(s0 - m), w1 = expf(s1 - m);
+      uint32_t hi, rest;
+      split2(w0, w1, hi, rest);
+      *reinterpret_cast<uint32_t*>(p_hi + h * kPRow + 2 * lane) = hi;
+      *reinterpret_cast<uint32_t*>(p_lo + h * kPRow + 2 * lane) = rest;
+      const float l = warp_sum(w0 + w1), f = expf(before - m);
+      if (lane == 0) {
+        m_run[h] = m;
+        l_run[h] = l_run[h] * f + l;
+        fix[h] = f;
+      }
+    }
+    __syncthreads();
+    const float f0 = fix[g], f1 = fix[g + 8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      acc[i][0] *= f0;
+      acc[i][1] *= f0;
+      acc[i][2] *= f1;
+      acc[i][3] *= f1;
+    }
+#pragma unroll
+    for (int kk = 0; kk < kKeys / 16; ++kk) {
+      if (16 * kk >= nt) break;
+      uint32_t hi[4], rest[4];
+      ldsm(hi, p_hi + (lane & 15) * kPRow + 16 * kk + (lane >> 4) * 8);
+      ldsm(rest, p_lo + (lane & 15) * kPRow + 16 * kk + (lane >> 4) * 8);
+#pragma unroll
+      for (int np = 0; np < 4; ++np) {
+        if (c0 + 16 * np >= a.rank_pad) break;
+        uint32_t b[4];
+        ldsm_trans(b, tile + (16 * kk + (lane & 15)) * R + c0 + 16 * np + (lane >> 4) * 8);
+        mma_bf16_16816(acc[2 * np], hi, b[0], b[1]);
+        mma_bf16_16816(acc[2 * np + 1], hi, b[2], b[3]);
+        mma_bf16_16816(acc[2 * np], rest, b[0], b[1]);
+        mma_bf16_16816(acc[2 * np + 1], rest, b[2], b[3]);
+      }
+    }
+    __syncthreads();
+    if (t0 + kKeys < k1) fetch(t0 + kKeys);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int h = h0 + g + 8 * half;
+    if (h >= a.heads) continue;
+    float* dst = a.part + (((int64_t)blockIdx.z * splits + split) * a.heads + h) * a.rank_pad;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int c = c0 + 8 * i + 2 * t;
+      if (c < a.rank_pad) *reinterpret_cast<float2*>(dst + c) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
+    }
+  }
+  if (tid < kMmaHeads && h0 + tid < a.heads)
+    reinterpret_cast<float2*>(a.stats)[((int64_t)blockIdx.z * splits + split) * a.heads + h0 + tid] = make_float2(m_run[tid], l_run[tid]);
+}
+
 }  // namespace
 
 template <class TC, class TP, class TO>
 cudaError_t launch_latent_rows(const LatentArgs& a, const Rows& rows, TO* out, int64_t ldo, int sm_count, bool pdl, cudaStream_t st, int* launches) {
-  const int groups = (a.heads + kHG - 1) / kHG, blocks = (a.rank_pad + kCols - 1) / kCols;
+  const MmaShape shape = mma_shape(a);
+  const bool mma = sizeof(TC) == 2 && a.rank_pad <= kMmaCols && shape.smem <= 220 * 1024;
+  const int per_group = mma ? kMmaHeads : kHG, groups = (a.heads + per_group - 1) / per_group, blocks = mma ? 1 : (a.rank_pad + kCols - 1) / kCols;
   // about one tile of keys per range at least, two blocks per SM at most
   int splits = 1;
   if (rows.n <= kLatentRows) {
@@ -358,9 +532,10 @@ cudaError_t launch_latent_rows(const LatentArgs& a, const Rows& rows, TO* out, i
   while (keys > 1 && s_tile(keys) > 220 * 1024) keys /= 2;
   const size_t s_attn = s_tile(keys);
   if (s_in > 48 * 1024 || s_attn > 220 * 1024 || s_out > 200 * 1024) return cudaErrorInvalidValue;
-  cudaError_t e = cudaSuccess;
-  if (s_attn > 40 * 1024) e = cudaFuncSetAttribute(latent_attn_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s_attn);
-  if (e == cudaSuccess && s_out > 40 * 1024) e = cudaFuncSetAttribute(latent_out_kernel<TP, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s_out);
+  // the same limits for every size: launches of other sizes may already be in a captured step
+  cudaError_t e = cudaFuncSetAttribute(latent_attn_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_out_kernel<TP, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   if (e != cudaSuccess) return e;
   uint64_t fit = kLatentRows;
   const uint64_t per_part = (uint64_t)splits * a.heads * a.rank_pad, per_stats = 2ull * splits * a.heads;
@@ -370,9 +545,12 @@ cudaError_t launch_latent_rows(const LatentArgs& a, const Rows& rows, TO* out, i
   for (int r0 = 0; r0 < rows.n; r0 += (int)fit) {
     const int n = rows.n - r0 < (int)fit ? rows.n - r0 : (int)fit;
     e = launch_kernel(latent_in_kernel<TC, TP>, dim3((a.rank_pad + kSlice - 1) / kSlice + 1, a.heads, n), dim3(kThreads), s_in, st, pdl, a, rows, r0);
-    if (e == cudaSuccess) e = launch_kernel(latent_attn_kernel<TC>, dim3(splits * blocks, groups, n), dim3(kThreads), s_attn, st, pdl, a, rows, r0, splits, keys);
+    if (e == cudaSuccess) {
+      if (mma) e = launch_kernel(latent_attn_mma_kernel, dim3(splits, groups, n), dim3(kMmaThreads), (size_t)shape.smem, st, pdl, a, rows, r0, splits, shape);
+      else e = launch_kernel(latent_attn_kernel<TC>, dim3(splits * blocks, groups, n), dim3(kThreads), s_attn, st, pdl, a, rows, r0, splits, keys);
+    }
     if (e == cudaSuccess)
-      e = launch_kernel(latent_out_kernel<TP, TO>, dim3((a.vdim + kOutTile - 1) / kOutTile, a.heads, n), dim3(kThreads), s_out, st, pdl, a, rows, r0, splits, out, ldo);
+      e = launch_kernel(latent_out_kernel<TP, TO>, dim3((a.vdim + kOutTile - 1) / kOutTile, a.heads, n), dim3(kOutThreads), s_out, st, pdl, a, rows, r0, splits, out, ldo);
     if (e != cudaSuccess) return e;
     *launches += 3;
   }

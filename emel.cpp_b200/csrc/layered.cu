@@ -860,7 +860,7 @@ uint32_t layered_bind(Layered* m, int layer, int role, const emelb_view* t) {
   const void* dev = ctx_resolve_weights(m->c, t->data);
   if (!dev) return EMELB_INVALID_REQUEST;
   if (vec) {
-    if (t->type != EMELB_F32 || t->nb[0] != 4 || (M > 1 && (int64_t)t->nb[1] != 4 * K)) return EMELB_INVALID_REQUEST;
+    if (t->type != EMELB_F32 || t->nb[0] != 4 || (M > 1 && (int64_t)t->nb[1] != 4 * K) || reinterpret_cast<uintptr_t>(dev) % 16 != 0) return EMELB_INVALID_REQUEST;
     if (role == EMELB_T_MIX_CONV) {
       // kept tap by tap, so that neighbouring channels are read together
       float* taps = const_cast<float*>(l->w.conv);

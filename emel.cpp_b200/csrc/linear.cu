@@ -36,7 +36,13 @@ struct SplitVec {
   float* lo;
   float* hi;
   __device__ __forceinline__ float& at(int i) const { return ((i & 4) ? hi : lo)[(i >> 3) * 4 + (i & 3)]; }
+  __device__ __forceinline__ float4& quad(int j) const { return *reinterpret_cast<float4*>(((j & 1) ? hi : lo) + 4 * (j >> 1)); }   // elements 4j ..
 };
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float4 scale4(float4 x, float mean, float inv, float4 w) {
+  return make_float4((x.x - mean) * inv * w.x, (x.y - mean) * inv * w.y, (x.z - mean) * inv * w.z, (x.w - mean) * inv * w.w);
+}
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
 // A warp owns RW rows at a time (for a GLU a gate row and its up row) and walks them in 16-byte chunks, U per lane
 // in flight; the first chunks are requested before the wait for the kernel in front.  DUAL: the tasks of a second matrix,
@@ -75,6 +81,11 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
     }
   };
   if (task < tasks) load(task, 0);
+  if (v.pro == PRO_PRENORM)
+    for (int i = 32 * tid; i < K; i += 32 * kVecThreads) {
+      prefetch_l2(v.norm_w + i);
+      if (DUAL) prefetch_l2(v.norm2_w + i);
+    }
   pdl_wait();
 
   // ---- the input vector
@@ -82,8 +93,12 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
     xs.at(i) = 0.0f;
     if (DUAL) xs2.at(i) = 0.0f;
   }
+  const int quads = K / 4;
+  auto ld4 = [](const float* p, int j) { return reinterpret_cast<const float4*>(p)[j]; };
   if (v.pro == PRO_PLAIN) {
-    for (int i = tid; i < K; i += kVecThreads) xs.at(i) = v.x[i];
+#pragma unroll 8
+    for (int j = tid; j < quads; j += kVecThreads) xs.quad(j) = ld4(v.x, j);
+    for (int i = 4 * quads + tid; i < K; i += kVecThreads) xs.at(i) = v.x[i];
   } else if (v.pro == PRO_EMBED) {
     const __nv_bfloat16* row = v.table + (int64_t)*v.token * v.table_ld;
     for (int i = tid; i < K; i += kVecThreads) {
@@ -94,7 +109,23 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
   } else if (v.pro == PRO_PRENORM) {
     const __nv_bfloat16* row = v.table ? v.table + (int64_t)*v.token * v.table_ld : nullptr;
     float s = 0.0f, ss = 0.0f;
-    for (int i = tid; i < K; i += kVecThreads) {
+#pragma unroll 4
+    for (int j = tid; j < quads; j += kVecThreads) {
+      float4 x;
+      if (row) {
+        const uint2 t = reinterpret_cast<const uint2*>(row)[j];
+        x = make_float4(__uint_as_float(t.x << 16), __uint_as_float(t.x & 0xffff0000u), __uint_as_float(t.y << 16), __uint_as_float(t.y & 0xffff0000u));
+      } else {
+        x = ld4(v.x, j);
+      }
+      if (v.y) x = add4(x, ld4(v.y, j));
+      if (v.step) x = make_float4(x.x + v.step[4 * j], x.y + v.step[4 * j + 1], x.z + v.step[4 * j + 2], x.w + v.step[4 * j + 3]);
+      xs.quad(j) = x;
+      s += (x.x + x.y) + (x.z + x.w);
+      ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss))));
+      if (v.x_out && blockIdx.x == 0) reinterpret_cast<float4*>(v.x_out)[j] = x;
+    }
+    for (int i = 4 * quads + tid; i < K; i += kVecThreads) {
       float x = row ? __bfloat162float(row[i]) : v.x[i];
       if (v.y) x += v.y[i];
       if (v.step) x += v.step[i];
@@ -107,13 +138,20 @@ __global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArg
     if (!v.rms) {
       mean = block_sum(s, scratch) / K;
       ss = 0.0f;
-      for (int i = tid; i < K; i += kVecThreads) {
-        const float d = xs.at(i) - mean;
-        ss = fmaf(d, d, ss);
+      for (int j = tid; j < quads; j += kVecThreads) {
+        const float4 x = xs.quad(j);
+        ss = fmaf(x.x - mean, x.x - mean, fmaf(x.y - mean, x.y - mean, fmaf(x.z - mean, x.z - mean, fmaf(x.w - mean, x.w - mean, ss))));
       }
+      for (int i = 4 * quads + tid; i < K; i += kVecThreads) ss = fmaf(xs.at(i) - mean, xs.at(i) - mean, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / K + v.eps);
-    for (int i = tid; i < K; i += kVecThreads) {
+#pragma unroll 4
+    for (int j = tid; j < quads; j += kVecThreads) {
+      const float4 x = xs.quad(j);
+      xs.quad(j) = scale4(x, mean, inv, ld4(v.norm_w, j));
+      if (DUAL) xs2.quad(j) = scale4(x, mean, inv, ld4(v.norm2_w, j));
+    }
+    for (int i = 4 * quads + tid; i < K; i += kVecThreads) {
       const float n = (xs.at(i) - mean) * inv;
       xs.at(i) = n * v.norm_w[i];
       if (DUAL) xs2.at(i) = n * v.norm2_w[i];
@@ -307,8 +345,9 @@ cudaError_t launch_linear_vec(const LinearArgs& a, const VecArgs& v, int sm_coun
   // two rows per warp unless that leaves SMs without work
   const bool pair = dual || is_glu(a.act) || outs >= sm_count * kVecWarps * 2;
   auto kern = dual ? linear_vec_kernel<2, 4, true> : pair ? linear_vec_kernel<2, 4, false> : linear_vec_kernel<1, 8, false>;
-  if (smem > 48 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (smem > 40 * 1024) {
+    // the same limit for every size: launches of other sizes may already be in a captured step
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return e;
   }
   auto tasks_of = [&](int n, int act) { return pair && !is_glu(act) ? (n + 1) / 2 : n; };

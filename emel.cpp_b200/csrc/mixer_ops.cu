@@ -274,9 +274,10 @@ template cudaError_t launch_embed_rows_bf16<__nv_bfloat16>(const __nv_bfloat16*,
                                                            int64_t, cudaStream_t);
 
 namespace {
+// the same limit for every size: launches of other sizes may already be in a captured step
 template <class K>
 cudaError_t allow_smem(K kern, size_t bytes) {
-  return bytes > 48 * 1024 ? cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) : cudaSuccess;
+  return bytes > 48 * 1024 ? cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) : cudaSuccess;
 }
 }  // namespace
 

@@ -178,7 +178,7 @@ EMELB_API uint32_t emelb_llama_destroy(emelb_llama* s);
  * shard_count must be 1.  float32 = 1: activations, products and caches in f32 throughout (no reduced-precision
  * matrix mode); 0: matrix operands and the key / value cache in bf16 with f32 accumulation.
  * Matrices are bound as {K, M} views of type EMELB_BF16 whose row stride is a multiple of 16 bytes, with zeros
- * between K and the stride; vectors as EMELB_F32. */
+ * between K and the stride; vectors as EMELB_F32 at a 16-byte boundary. */
 EMELB_API uint32_t emelb_llama_check_layers(const emelb_llama_config* cfg, const emelb_layer_config* layers);
 EMELB_API uint32_t emelb_llama_create_layers(emelb_ctx* ctx, const emelb_llama_config* cfg,
                                              const emelb_layer_config* layers, int32_t float32, emelb_llama** out);
