@@ -768,9 +768,8 @@ cudaError_t launch_chunks(const DeltaArgs& a, const Rows& rows, int sm_count, cu
   return a.heads * ((a.vdim + 15) / 16) <= sm_count ? launch_scan<D, 16>(a, rows, st) : launch_scan<D, 32>(a, rows, st);
 }
 
-// a warp per (row, head), V columns per lane and turn; the first kNormTurns turns stay in registers
-constexpr int kNormTurns = 4;
-template <class T, int V>
+// a warp per (row, head)
+template <class T>
 __global__ void __launch_bounds__(kConvThreads) delta_norm_kernel(const DeltaArgs a, const Rows rows, T* __restrict__ out, int64_t ldo) {
   const int64_t task = (int64_t)blockIdx.x * (kConvThreads / 32) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -779,42 +778,39 @@ __global__ void __launch_bounds__(kConvThreads) delta_norm_kernel(const DeltaArg
   const int h = (int)(task % a.heads);
   const float* o = a.o + task * a.vdim;
   const T* gate = static_cast<const T*>(a.proj) + r * a.ldp + a.channels() + h * a.vdim;
-  T* dst = out + r * ldo + h * a.vdim;
-  float x[kNormTurns][V], z[kNormTurns][V], ss = 0.0f;
-#pragma unroll
-  for (int i = 0; i < kNormTurns; ++i) {
-    const int c = V * (lane + 32 * i);
-    if (c >= a.vdim) break;
-    Vec<float, V>::load(o + c, x[i]);
-    Vec<T, V>::load(gate + c, z[i]);
-#pragma unroll
-    for (int e = 0; e < V; ++e) ss = fmaf(x[i][e], x[i][e], ss);
-  }
-  for (int c = V * (lane + 32 * kNormTurns); c < a.vdim; c += 32 * V) {
-    float y[V];
-    Vec<float, V>::load(o + c, y);
-#pragma unroll
-    for (int e = 0; e < V; ++e) ss = fmaf(y[e], y[e], ss);
-  }
+  float ss = 0.0f;
+  for (int c = lane; c < a.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
   const float inv = 1.0f / sqrtf(warp_sum(ss) / a.vdim + a.eps);
-  auto finish = [&](int c, float (&y)[V], const float (&g)[V]) {
-    float w[V];
-    Vec<float, V>::load(a.norm + c, w);
+  for (int c = lane; c < a.vdim; c += 32) out[r * ldo + h * a.vdim + c] = to<T>(o[c] * inv * a.norm[c] * siluf_(from(gate[c])));
+}
+
+// heads of at most 128 values, a multiple of 4: four of them per warp, every load requested at once
+constexpr int kNormHeads = 4;
+template <class T>
+__global__ void __launch_bounds__(kConvThreads) delta_norm_small_kernel(const DeltaArgs a, const Rows rows, T* __restrict__ out, int64_t ldo) {
+  const int64_t tasks = (int64_t)rows.n * a.heads, first = ((int64_t)blockIdx.x * (kConvThreads / 32) + (threadIdx.x >> 5)) * kNormHeads;
+  const int c = 4 * (threadIdx.x & 31);
+  const bool live = c < a.vdim;
+  float x[kNormHeads][4] = {}, z[kNormHeads][4] = {}, w[4] = {};
+  if (live) Vec<float, 4>::load(a.norm + c, w);
 #pragma unroll
-    for (int e = 0; e < V; ++e) y[e] = y[e] * inv * w[e] * siluf_(g[e]);
-    Vec<T, V>::store(dst + c, y);
-  };
-#pragma unroll
-  for (int i = 0; i < kNormTurns; ++i) {
-    const int c = V * (lane + 32 * i);
-    if (c >= a.vdim) break;
-    finish(c, x[i], z[i]);
+  for (int i = 0; i < kNormHeads; ++i) {
+    const int64_t task = first + i;
+    if (task >= tasks || !live) continue;
+    Vec<float, 4>::load(a.o + task * a.vdim + c, x[i]);
+    Vec<T, 4>::load(static_cast<const T*>(a.proj) + task / a.heads * a.ldp + a.channels() + task % a.heads * a.vdim + c, z[i]);
   }
-  for (int c = V * (lane + 32 * kNormTurns); c < a.vdim; c += 32 * V) {
-    float y[V], g[V];
-    Vec<float, V>::load(o + c, y);
-    Vec<T, V>::load(gate + c, g);
-    finish(c, y, g);
+#pragma unroll
+  for (int i = 0; i < kNormHeads; ++i) {
+    const int64_t task = first + i;
+    float ss = 0.0f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss = fmaf(x[i][e], x[i][e], ss);
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / a.vdim + a.eps);
+    if (task >= tasks || !live) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[i][e] = x[i][e] * inv * w[e] * siluf_(z[i][e]);
+    Vec<T, 4>::store(out + task / a.heads * ldo + task % a.heads * a.vdim + c, x[i]);
   }
 }
 
@@ -887,9 +883,11 @@ cudaError_t launch_delta_prompt(const DeltaArgs& a, const Rows& rows, T* out, in
     delta_rows_kernel<T><<<dim3(a.heads, (a.vdim + kCols - 1) / kCols), dim3(kCols, kGroups), smem, st>>>(a, rows);
     if ((e = cudaGetLastError()) != cudaSuccess) return e;
   }
-  const unsigned blocks = (unsigned)(((int64_t)rows.n * a.heads + warps - 1) / warps);
-  if (a.dim % 2 == 0 && a.vdim % 4 == 0 && a.ldp % 4 == 0 && ldo % 4 == 0) delta_norm_kernel<T, 4><<<blocks, kConvThreads, 0, st>>>(a, rows, out, ldo);
-  else delta_norm_kernel<T, 1><<<blocks, kConvThreads, 0, st>>>(a, rows, out, ldo);
+  const bool small = a.dim % 2 == 0 && a.vdim % 4 == 0 && a.vdim <= 128 && a.ldp % 4 == 0 && ldo % 4 == 0;
+  const int64_t per_block = warps * (small ? kNormHeads : 1);
+  const unsigned blocks = (unsigned)(((int64_t)rows.n * a.heads + per_block - 1) / per_block);
+  if (small) delta_norm_small_kernel<T><<<blocks, kConvThreads, 0, st>>>(a, rows, out, ldo);
+  else delta_norm_kernel<T><<<blocks, kConvThreads, 0, st>>>(a, rows, out, ldo);
   return cudaGetLastError();
 }
 template cudaError_t launch_delta_prompt<float>(const DeltaArgs&, const Rows&, float*, int64_t, int, cudaStream_t, int*);

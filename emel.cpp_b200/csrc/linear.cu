@@ -48,7 +48,7 @@ __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefe
 // in flight; the first chunks are requested before the wait for the kernel in front.  DUAL: the tasks of a second matrix,
 // which meets the input with the other norm weight, follow those of the first.
 template <int RW, int U, bool DUAL>
-__global__ void __launch_bounds__(kVecThreads) linear_vec_kernel(const LinearArgs a, const VecArgs v) {
+__global__ void __launch_bounds__(kVecThreads, RW == 2 ? 4 : 3) linear_vec_kernel(const LinearArgs a, const VecArgs v) {
   extern __shared__ __align__(16) float xs_raw[];
   __shared__ float scratch[kVecWarps];
   pdl_trigger();

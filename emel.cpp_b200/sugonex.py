@@ -44,7 +44,7 @@ def layer_configs(cfg: dict):
 def stack_config(cfg: dict) -> ly.StackConfig:
     loop = cfg.get("loop")
     return ly.stack(ly.STACK_PARALLEL, ly.NORM_RMS, loop=(loop["start"], loop["stop"], loop["times"]) if loop else None, loop_step=bool(loop),
-                    logit_scale=cfg.get("logit_scale", 1.0), logit_softcap=cfg.get("logit_softcap") or 0.0)
+                    logit_scale=1.0 if cfg.get("logit_scale") is None else cfg["logit_scale"], logit_softcap=cfg.get("logit_softcap") or 0.0)
 
 
 def session_config(cfg: dict, n_ctx: int) -> el.Config:

@@ -51,14 +51,14 @@ TILED = model(256, 300, [
     delta(3, 3, 48, 80, 2, ff=128),
     latent(2, 128, 64, 128, 512, 0.15, base=1e4),
 ], loop=(3, 5, 2))
-# many heads, a wide latent, value rows wider than a tile, no loop
+# many heads, a wide latent, value rows wider than a tile, a loop of one pass
 HEADS = model(128, 90, [
     latent(20, 16, 8, 16, 24, 0.6, ff=40),
     delta(16, 4, 16, 24, 4, ff=56),
     windowed(9, 32, 136, 600, 0.4, 33),
     delta(2, 1, 144, 200, 3, ff=24),
     delta(4, 2, 64, 32, 4),
-])
+], loop=(2, 4, 1))
 MODELS = {"heads": HEADS, "odd": ODD, "plain": PLAIN, "tiled": TILED}
 
 
