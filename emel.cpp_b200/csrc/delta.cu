@@ -788,29 +788,30 @@ __global__ void __launch_bounds__(kConvThreads) delta_norm_kernel(const DeltaArg
 constexpr int kNormHeads = 4;
 template <class T>
 __global__ void __launch_bounds__(kConvThreads) delta_norm_small_kernel(const DeltaArgs a, const Rows rows, T* __restrict__ out, int64_t ldo) {
-  const int64_t tasks = (int64_t)rows.n * a.heads, first = ((int64_t)blockIdx.x * (kConvThreads / 32) + (threadIdx.x >> 5)) * kNormHeads;
+  const unsigned tasks = (unsigned)rows.n * a.heads, first = (blockIdx.x * (kConvThreads / 32) + (threadIdx.x >> 5)) * kNormHeads;
   const int c = 4 * (threadIdx.x & 31);
   const bool live = c < a.vdim;
   float x[kNormHeads][4] = {}, z[kNormHeads][4] = {}, w[4] = {};
+  int64_t dst[kNormHeads];
   if (live) Vec<float, 4>::load(a.norm + c, w);
 #pragma unroll
   for (int i = 0; i < kNormHeads; ++i) {
-    const int64_t task = first + i;
+    const unsigned task = first + i, r = task / (unsigned)a.heads, h = task - r * a.heads;
+    dst[i] = r * ldo + h * a.vdim + c;
     if (task >= tasks || !live) continue;
-    Vec<float, 4>::load(a.o + task * a.vdim + c, x[i]);
-    Vec<T, 4>::load(static_cast<const T*>(a.proj) + task / a.heads * a.ldp + a.channels() + task % a.heads * a.vdim + c, z[i]);
+    Vec<float, 4>::load(a.o + (int64_t)task * a.vdim + c, x[i]);
+    Vec<T, 4>::load(static_cast<const T*>(a.proj) + r * a.ldp + a.channels() + h * a.vdim + c, z[i]);
   }
 #pragma unroll
   for (int i = 0; i < kNormHeads; ++i) {
-    const int64_t task = first + i;
     float ss = 0.0f;
 #pragma unroll
     for (int e = 0; e < 4; ++e) ss = fmaf(x[i][e], x[i][e], ss);
     const float inv = 1.0f / sqrtf(warp_sum(ss) / a.vdim + a.eps);
-    if (task >= tasks || !live) continue;
+    if (first + i >= tasks || !live) continue;
 #pragma unroll
     for (int e = 0; e < 4; ++e) x[i][e] = x[i][e] * inv * w[e] * siluf_(z[i][e]);
-    Vec<T, 4>::store(out + task / a.heads * ldo + task % a.heads * a.vdim + c, x[i]);
+    Vec<T, 4>::store(out + dst[i], x[i]);
   }
 }
 

@@ -197,6 +197,25 @@ def test_state_remembers_a_far_token(be, tmp_path, f32):
 
 
 @BOTH
+def test_repeated_keys(be, tmp_path, f32):
+    """Long runs of the same few tokens with step sizes near 1 and hardly any decay: within a chunk every key meets itself
+    many times, so that the triangular systems of the chunked recurrence are far from the identity."""
+    cfg = sm.model(64, 30, [sm.delta(3, 1, 32, 40, 1), sm.delta(2, 2, 64, 32, 2)], loop=(0, 2, 2))
+
+    def near_one(t):
+        for i in (0, 1):
+            t[f"l{i}.mix.A_log"] = np.full_like(t[f"l{i}.mix.A_log"], -9.0)
+            t[f"l{i}.mix.b"] = sm.round_bf16(4.0 * t[f"l{i}.mix.b"])
+    c = Case(cfg, tmp_path / "m", 1, 12, change=near_one)
+    toks = [5] * 40 + [7, 5] * 40 + [9] * 70 + [5, 5, 7, 9] * 10
+    want = so.logits(cfg, c.w, toks)
+    s = models.load(be, str(c.folder), n_ctx=240, float32=f32)
+    for sizes in ([300], [1], [64, 3, 61]):
+        assert_close(sm.row_errors(feed(s, toks, sizes), want), f32, sizes)
+    s.close()
+
+
+@BOTH
 def test_first_tokens(be, cases, f32):
     c = cases["odd"]
     s = c.session(be, f32)
